@@ -77,7 +77,14 @@ class LayerSpec:
     weight vector shared by the heads); ``v_norm`` (values normed per head); ``softcap`` > 0 (``score <- cap tanh(score /
     cap)``); ``keep_first`` (with ``window``: the first keys stay visible); ``sink`` (a learned score per head joins the
     softmax denominator).  Latent attention: ``q_rank`` 0 = queries come straight from the layer input; ``out_gate``: the
-    concatenated heads are multiplied by ``sigmoid(W_g h)`` in front of the output projection."""
+    concatenated heads are multiplied by ``sigmoid(W_g h)`` in front of the output projection.
+    More softmax attention options: ``qk_norm`` "none" (q and k as projected); ``keys_as_values`` (there is no value
+    projection, the cached key rows are the values); ``proj_bias`` (q, k and output projections have biases);
+    ``distance_bias`` (head ``h`` of ``H`` loses ``2 ** (-8 (h + 1) / H)`` per token of distance); ``talk`` (a learned
+    ``[heads, heads]`` matrix mixes the heads' scores in front of the softmax); ``sink_one`` (a sink whose score is 0).
+    ``ff_act`` = "poly_norm": dense feed-forward without a gate whose activation is a weighted sum of the RMS-normed first
+    three powers and a constant.  ``route_kind`` = "sigmoid_topk": the ``top`` largest sigmoid scores, used as they are;
+    ``scale_input``: an expert's weight multiplies its input instead of its output."""
     mixer: str = "attention"
     heads: int = 1
     kv_heads: int = 1
@@ -113,6 +120,18 @@ class LayerSpec:
     keep_first: int = 0
     sink: bool = False
     out_gate: bool = False
+    keys_as_values: bool = False
+    proj_bias: bool = False
+    distance_bias: bool = False
+    talk: bool = False
+    sink_one: bool = False
+    ff_act: str = ""
+    scale_input: bool = False
+
+    @property
+    def head_slopes(self) -> Tuple[float, ...]:
+        """score lost per token of distance between query and key, one number per head (``distance_bias``)"""
+        return tuple(2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads))
 
     @property
     def leaves(self) -> Tuple["LayerSpec", ...]:
@@ -122,7 +141,7 @@ class LayerSpec:
 @dataclass
 class ModelConfig:
     name: str = "tiny-llama"
-    family: str = "llama"            # gpt2 | llama | mistral | gemma2 | kepovik | repudra | lonulix | fisopel
+    family: str = "llama"            # gpt2 | llama | mistral | gemma2 | kepovik | repudra | lonulix | fisopel | kazolorn
     vocab_size: int = 512
     hidden_size: int = 256
     n_layers: int = 2
@@ -169,6 +188,8 @@ class ModelConfig:
     loop_stop: int = 0
     loop_times: int = 1
     loop_in: bool = False
+    depth_average: bool = False      # parallel blocks: what leaves a layer is a learned weighted sum of its result, all earlier
+    #                                  layers' results and the embedding output
 
     # ------------------------------------------------------------------ derived
     @property
@@ -526,7 +547,65 @@ class ModelConfig:
         return d
 
     @staticmethod
+    def from_kazolorn_dict(d: Dict, name: str = "") -> "ModelConfig":
+        """``config.json`` of a Kazolorn checkpoint: ``layers`` lists {type, mixer sizes, mlp | null}; type ``attention``
+        (windowed, keys as values, mixed heads, distance bias); ``mlp.kind`` ``dense`` (PolyNorm) or ``moe`` (gated silu
+        experts chosen and weighted by sigmoid scores)."""
+        who = name or "kazolorn"
+        specs = []
+        for lay in d["layers"]:
+            m, mlp, kind = lay.get("mixer") or {}, lay.get("mlp"), lay["type"]
+            if kind != "attention":
+                raise ValueError(f"{who}: unknown layer type {kind!r}")
+            heads, dim = int(m["heads"]), int(m["dim"])
+            sp = LayerSpec(mixer="softmax_attention", heads=heads, kv_heads=int(m.get("kv_heads", heads)), dim=dim,
+                           vdim=int(m.get("vdim", dim)), scale=float(m.get("scale", dim ** -0.5)),
+                           window=int((m.get("mask") or {}).get("size", 0) or 0), qk_norm="none", v_norm=False,
+                           keys_as_values=True, proj_bias=True, distance_bias=True, talk=True, sink_one=True)
+            if sp.heads % sp.kv_heads:
+                raise ValueError(f"{who}: {sp.heads} heads cannot share {sp.kv_heads} key heads")
+            if sp.vdim != sp.dim:
+                raise ValueError(f"{who}: the keys are the values, but their widths differ ({sp.dim}, {sp.vdim})")
+            if mlp:
+                fk = mlp.get("kind", "dense")
+                if fk == "dense":
+                    sp.ff, sp.ff_act = int(mlp["ff"]), "poly_norm"
+                elif fk == "moe":
+                    r = mlp["router"]
+                    sp.ff_kind, sp.expert_ff, sp.experts, sp.top = "moe", int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"])
+                    sp.route_kind, sp.expert_gated, sp.scale_input = "sigmoid_topk", True, True
+                    sp.ff = sp.experts * sp.expert_ff
+                    if not 0 < sp.top <= sp.experts:
+                        raise ValueError(f"{who}: {sp.top} of {sp.experts} experts cannot be chosen")
+                else:
+                    raise ValueError(f"{who}: feed-forward kind {fk!r} is not implemented")
+            specs.append(sp)
+        return ModelConfig(
+            name=name or "kazolorn", family="kazolorn", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+            n_layers=len(specs), n_heads=max(sp.heads for sp in specs), n_kv_heads=max(sp.kv_heads for sp in specs),
+            head_dim=max(sp.dim for sp in specs), ffn_size=max([sp.ff for sp in specs] + [0]), max_position=1 << 30,
+            norm="rms", norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)), act="silu", glu=True, rope_theta=0.0,
+            layer_specs=tuple(specs), streams=0, block_layout="parallel", ff_norm=True, layer_scale=True,
+            depth_average=True)
+
+    def to_kazolorn_dict(self) -> Dict:
+        layers = []
+        for sp in self.layer_specs:
+            m = {"dim": sp.dim, "heads": sp.heads, "kv_heads": sp.kv_heads, "scale": sp.scale, "vdim": sp.vdim}
+            if sp.window:
+                m["mask"] = {"size": sp.window}
+            mlp = None
+            if sp.ff:
+                mlp = {"ff": sp.ff, "kind": "dense"} if sp.ff_kind == "dense" else \
+                    {"expert": {"ff": sp.expert_ff}, "kind": "moe", "router": {"experts": sp.experts, "top": sp.top}}
+            layers.append({"type": "attention", "mixer": m, "mlp": mlp})
+        return {"architecture": "Kazolorn", "layers": layers, "norm": {"eps": self.norm_eps}, "vocab": self.vocab_size,
+                "width": self.hidden_size}
+
+    @staticmethod
     def from_hf_dict(d: Dict, name: str = "") -> "ModelConfig":
+        if str(d.get("architecture", "")).lower() == "kazolorn":
+            return ModelConfig.from_kazolorn_dict(d, name)
         if str(d.get("architecture", "")).lower() == "fisopel":
             return ModelConfig.from_fisopel_dict(d, name)
         if str(d.get("architecture", "")).lower() == "lonulix":
@@ -584,6 +663,8 @@ class ModelConfig:
             return self.to_lonulix_dict()
         if self.family == "fisopel":
             return self.to_fisopel_dict()
+        if self.family == "kazolorn":
+            return self.to_kazolorn_dict()
         if self.family == "gpt2":
             return {"model_type": "gpt2", "architectures": ["GPT2LMHeadModel"], "vocab_size": self.vocab_size,
                     "n_embd": self.hidden_size, "n_layer": self.n_layers, "n_head": self.n_heads,
@@ -783,6 +864,33 @@ def _fisopel(name, width, vocab, layers, loop=None, embed_scale=2.0):
 PRESETS["tiny-fisopel"] = _fisopel("tiny-fisopel", 128, 512, [
     ("attention", 4, 2, 32, 16, 40, 6, 30.0, (6, 32, 2, 48)), ("latent_attention", 3, 16, 16, 24, 48, 4.0, (5, 32, 3, 0)),
     ("latent_attention", 2, 32, 8, 32, 40, 0.0, 0)], loop=(0, 2, 2))
+
+
+def _kazolorn(name, width, vocab, layers):
+    """layers: (H, G, dim, window, mlp); mlp: 0 (none) | ff (dense) | (experts, expert_ff, top)"""
+    specs = []
+    for h, g, d, win, mlp in layers:
+        sp = LayerSpec(mixer="softmax_attention", heads=h, kv_heads=g, dim=d, vdim=d, scale=d ** -0.5, window=win, qk_norm="none",
+                       v_norm=False, keys_as_values=True, proj_bias=True, distance_bias=True, talk=True, sink_one=True)
+        if isinstance(mlp, tuple):
+            e, eff, top = mlp
+            sp.ff_kind, sp.experts, sp.expert_ff, sp.top, sp.ff = "moe", e, eff, top, e * eff
+            sp.route_kind, sp.expert_gated, sp.scale_input = "sigmoid_topk", True, True
+        elif mlp:
+            sp.ff, sp.ff_act = int(mlp), "poly_norm"
+        specs.append(sp)
+    return ModelConfig(name=name, family="kazolorn", vocab_size=vocab, hidden_size=width, n_layers=len(specs),
+                       n_heads=max(sp.heads for sp in specs), n_kv_heads=max(sp.kv_heads for sp in specs),
+                       head_dim=max(sp.dim for sp in specs), ffn_size=max(sp.ff for sp in specs), max_position=1 << 30,
+                       norm="rms", norm_eps=1e-5, act="silu", glu=True, rope_theta=0.0, layer_specs=tuple(specs),
+                       block_layout="parallel", ff_norm=True, layer_scale=True, depth_average=True, eos_token_id=-1,
+                       bos_token_id=-1)
+
+
+# parallel blocks with depth averages, test preset: grouped heads with a dense feed-forward, one key head with experts, all
+# heads with keys of their own and no feed-forward, experts again
+PRESETS["tiny-kazolorn"] = _kazolorn("tiny-kazolorn", 128, 512, [
+    (4, 2, 32, 40, 192), (4, 1, 16, 72, (5, 32, 2)), (2, 2, 32, 100, 0), (6, 3, 16, 40, (4, 48, 1))])
 PRESETS["tiny-gpt2"].vocab_size = 384
 PRESETS["tiny-gpt2"].eos_token_id = 1
 PRESETS["tiny-gpt2"].bos_token_id = 0

@@ -25,6 +25,13 @@ norm, capped scores, a window that keeps the first keys in sight and a sink in t
 absorbed into the queries, values up-projected per head behind the attention, rotary part in the half-split pairing with
 YaRN frequencies).  Feed-forward: gated silu experts chosen by their router logits beside a shared expert.
 
+Family ``kazolorn``: parallel blocks with a norm each and layer scale, whose results are averaged over depth (what enters a
+layer is a learned weighted sum of the embedding output and every earlier layer's result, kept in fp32).  Mixer: windowed
+softmax attention whose values are the cached keys, with a linear distance bias, a learned matrix that mixes the heads' scores
+in front of the softmax, and a one in the denominator.  The score mix is served in absorbed form: ``sum_g T[h, g] (q_g . k_g')``
+is ONE dot product of a mixed query row over all key heads with the cached key row, so every head attends on its own.
+Feed-forward: PolyNorm, or gated silu experts chosen by sigmoid scores that multiply the expert's input.
+
 Same interface as ``native.NativePiece`` (the runner drives both through ``forward(BatchMeta)``): a flat batch of spans
 (prompt portions of any length beside single decoded tokens), physical KV slots and block tables from the page allocator,
 logits for the rows named by ``last_idx``.  What is new here and lives next to the shared machinery:
@@ -66,6 +73,7 @@ class _Mix:
     idx: int = 0                        # position among the mixers of its layer (scratch buffers are per position)
     off: Dict[str, int] = field(default_factory=dict)       # column of each projection in the fused output
     w_o: torch.Tensor = None
+    b_o: Optional[torch.Tensor] = None  # bias of the output projection
     w2: Optional[torch.Tensor] = None   # second level of the low-rank gate projections
     rank: int = 0
     f: Dict[str, torch.Tensor] = field(default_factory=dict)
@@ -87,6 +95,7 @@ class _Layer:
     w_down: Optional[torch.Tensor] = None
     w_glu: Optional[torch.Tensor] = None   # post-norm dense feed-forward, bf16: [gate | up] interleaved for the gated GEMM epilogue
     ff_off: Dict[str, int] = field(default_factory=dict)    # routed experts: columns of router / gate block / up block
+    b_cat: Optional[torch.Tensor] = None   # bias of the fused projection (padded to its rows)
     mix: tuple = ()                     # parallel blocks: the mixers that read the layer's input side by side
     act_params: tuple = (0.0, 0.0)      # xIELU: softplus(p), 1/2 + softplus(q)
 
@@ -205,6 +214,8 @@ class HybridPiece:
         self._bufs: Dict[tuple, torch.Tensor] = {}
         self.h = self._buf("h", dtype, self.Wp)
         self.h2 = self._buf("h2", dtype, self.Wp) if cfg.ff_norm else None
+        # depth averages: the embedding output and every layer's result of the step's tokens, fp32
+        self.past = torch.zeros((cfg.n_layers + 1, max_tokens, W), device=dev, dtype=f32) if cfg.depth_average else None
         self.last_x = torch.zeros((self.max_out_rows, self.Wp), device=dev, dtype=dtype)
         self.logits = torch.zeros((self.max_out_rows, self.vocab_pad), device=dev, dtype=f32)
         self._ones = torch.ones(self.ns, device=dev, dtype=f32)
@@ -262,7 +273,7 @@ class HybridPiece:
             for l, _, first in self.runs:
                 L = self.L[l]
                 n += 2 + sum(per[mx.spec.mixer] for mx in L.mix)                             # join + fused projection
-                n += (4 if L.spec.ff_kind == "moe" else 2) if L.spec.ff else 0
+                n += (4 if L.spec.ff_kind == "moe" else (3 if L.spec.ff_act == "poly_norm" else 2)) if L.spec.ff else 0
                 n += 2 if (first and self.w_loop is not None) else 0
             return n
         n = 3          # embedding, final stream sum + norm, previous-token commit (+ the head GEMM counted by the runner)
@@ -331,6 +342,7 @@ class HybridPiece:
         ls1 = vec(p + "ls1") if self.cfg.layer_scale else torch.ones(W, device=dev)
         col, mixes = 0, []
         blocks = []                       # row blocks of the fused projection, in float64
+        biases = []                       # (first row, vector) of the projections that have one
         for j, leaf in enumerate(sp.leaves):
             q = p + "mix." + (("left.", "right.")[j] if sp.mixer == "parallel" else "")
             mx = _Mix(spec=leaf, key=f"{l}.{j}", idx=j)
@@ -340,7 +352,7 @@ class HybridPiece:
                     col += w.shape[0]
                     blocks.append(w)
             else:
-                for n in _PROJ[leaf.mixer]:
+                for n in ("q", "k") if leaf.keys_as_values else _PROJ[leaf.mixer]:
                     mx.off[n] = col
                     col += tensors[q + n].shape[0]
                     blocks.append(tensors[q + n].to(device=dev, dtype=torch.float64))
@@ -348,7 +360,20 @@ class HybridPiece:
             if leaf.mixer == "latent_attention":
                 pass
             elif leaf.mixer == "softmax_attention":
-                mx.f["q.norm"], mx.f["k.norm"] = vec(q + "q.norm"), vec(q + "k.norm")
+                if leaf.qk_norm != "none":
+                    mx.f["q.norm"], mx.f["k.norm"] = vec(q + "q.norm"), vec(q + "k.norm")
+                if leaf.proj_bias:
+                    biases += [(mx.off[n], vec(q + n + ".b")) for n in (("q", "k") if leaf.keys_as_values else ("q", "k", "v"))]
+                    mx.b_o = torch.zeros(mx.w_o.shape[0], device=dev)
+                    mx.b_o[:W] = vec(q + "o.b")
+                slopes = torch.tensor(leaf.head_slopes, dtype=torch.float64, device=dev)
+                if leaf.talk:           # mixing scores mixes their distance biases too: one slope per mixed head
+                    mx.f["talk"] = vec(q + "talk")
+                    slopes = mx.f["talk"].to(torch.float64) @ slopes
+                if leaf.distance_bias:
+                    mx.f["slopes"] = slopes.to(torch.float32).contiguous()
+                if leaf.sink_one:
+                    mx.f["sink"] = torch.zeros(leaf.heads, device=dev)
                 if leaf.sink:
                     mx.f["sink"] = vec(q + "sink")
                 rot = leaf.rot
@@ -379,12 +404,21 @@ class HybridPiece:
             mixes.append(mx)
         L.mix = tuple(mixes)
         L.w_cat = ops.pad_weight(torch.cat(blocks, 0).to(torch.float32), 128, 64).to(self.dtype).contiguous()
+        if biases:
+            L.b_cat = torch.zeros(L.w_cat.shape[0], device=dev)
+            for row, b in biases:
+                L.b_cat[row:row + b.numel()] = b
+        if self.cfg.depth_average:
+            L.f["dwa"] = vec(p + "dwa")
         if sp.ff:
             if self.cfg.ff_norm:
                 L.f["norm2"] = vec(p + "norm2")
             L.f["ls2"] = vec(p + "ls2") if self.cfg.layer_scale else None
             if sp.ff_kind == "moe":
                 self._build_routed_ff(L, p, tensors)
+                return L
+            if sp.ff_act == "poly_norm":
+                L.w_up, L.w_down, L.f["act"] = mat(p + "mlp.up"), mat(p + "mlp.down"), vec(p + "mlp.act")
                 return L
             L.w_up, L.w_down = mat(p + "mlp.up"), mat(p + "mlp.down", k_mult=128)
             a = vec(p + "mlp.act")
@@ -452,7 +486,8 @@ class HybridPiece:
             return
         if sp.mixer == "softmax_attention":
             self.k_cache[key] = torch.zeros((num_pages, ops.PAGE, sp.kv_heads, sp.dim), device=dev, dtype=self.dtype)
-            self.v_cache[key] = torch.zeros((num_pages, ops.PAGE, sp.kv_heads, sp.vdim), device=dev, dtype=self.dtype)
+            self.v_cache[key] = self.k_cache[key] if sp.keys_as_values else \
+                torch.zeros((num_pages, ops.PAGE, sp.kv_heads, sp.vdim), device=dev, dtype=self.dtype)
             return
         self.state[key] = torch.zeros((self.state_slots, sp.heads, sp.dim, sp.vdim), device=dev, dtype=f32)
         if sp.mixer == "mlstm":
@@ -469,9 +504,12 @@ class HybridPiece:
         T, S, mq = m.n_tokens, m.n_seqs, m.max_q
         eps, W = c.norm_eps, c.hidden_size
         x = self.streams[:T].view(T, W)
+        past = self.past
+        first = self.streams[:T] if past is None else past[0, :T].unsqueeze(1)
         ops.hyb_embed(m.ids, m.positions, m.q_start, m.q_len, m.seq_slot, self.prev_tok, self.embed, None, 0, 0, 0,
-                      self.streams[:T], S, mq, scale=c.embed_scale)
+                      first, S, mq, scale=c.embed_scale)
         h = self.h[:T]
+        depth, n_past = None, 0          # depth average that the next join takes
         pend: list = []
         hcat = None
         if self.w_loop is not None:                  # operand of the loop's input matrix: [residual | embedding output]
@@ -488,9 +526,10 @@ class HybridPiece:
                 replace = True
             two = self.cfg.ff_norm and L.spec.ff > 0
             hf = self.h2[:T] if two else h           # what the feed-forward reads
-            ops.ls_join(x, m.q_start, m.q_len, S, mq, terms=pend, gamma=L.f["norm1"], eps=eps, h=h, replace=replace,
-                        gamma2=L.f["norm2"] if two else None, h2=hf if two else None)
-            proj = ops.linear(L.w_cat, h, self._buf("proj", torch.float32, L.w_cat.shape[0])[:T])
+            ops.ls_join(past[0, :T] if past is not None and n_past == 0 else x, m.q_start, m.q_len, S, mq, terms=pend,
+                        gamma=L.f["norm1"], eps=eps, h=h, replace=replace, gamma2=L.f["norm2"] if two else None,
+                        h2=hf if two else None, depth=depth)
+            proj = ops.linear(L.w_cat, h, self._buf("proj", torch.float32, L.w_cat.shape[0])[:T], bias=L.b_cat)
             pend = []
             joins = []
             main = torch.cuda.current_stream()
@@ -523,13 +562,17 @@ class HybridPiece:
                 pend.append((yff if yff is not None else self._ff(L, hf, T), L.f["ls2"], False))
             for done in joins:
                 main.wait_event(done)
+            if past is not None:
+                n_past += 1
+                depth = (past, L.f["dwa"], n_past, past[0, :T] if n_past == 1 else x)
             if self.debug_layers is not None:
-                self.debug_layers.append(self._debug_join(x, pend, T))
+                self.debug_layers.append(self._debug_join(x, pend, T, depth))
         self._pass = 0
         R = m.n_out or S
         rows = m.last_idx if m.last_idx is not None else m.q_start
         xl = self.last_x[:R]
-        ops.ls_join(x, m.q_start, m.q_len, S, mq, terms=pend, gamma=self.final_norm, eps=eps, h=xl, rows=rows, n_rows=R)
+        ops.ls_join(x, m.q_start, m.q_len, S, mq, terms=pend, gamma=self.final_norm, eps=eps, h=xl, rows=rows, n_rows=R,
+                    depth=depth)
         logits = ops.linear(self.w_head, xl, self.logits[:R])
         if self.caps_logits:
             ops.act_cols(logits, 0, logits, logits.shape[1], ops.COLS_SOFTCAP, R, p0=c.final_softcap)
@@ -692,42 +735,53 @@ class HybridPiece:
         return ops.linear(mx.w_o, do, y)
 
     def _ff(self, L: _Layer, h: torch.Tensor, T: int) -> torch.Tensor:
-        """down(xIELU(up(h))): the activation is the epilogue of the up-projection; routed experts: see ``_ff_routed``"""
+        """down(xIELU(up(h))): the activation is the epilogue of the up-projection; PolyNorm needs whole rows and has a kernel
+        of its own behind it; routed experts: see ``_ff_routed``"""
         if L.spec.ff_kind == "moe":
             return self._ff_routed(L, h, T)
+        if L.spec.ff_act == "poly_norm":
+            z = ops.linear(L.w_up, h, self._buf("proj2", torch.float32, L.w_up.shape[0])[:T])
+            hid = self._buf(f"ff{L.spec.ff}", self.dtype, L.w_down.shape[1])[:T]
+            ops.poly_norm(z, 0, L.f["act"], hid, L.spec.ff, self.cfg.norm_eps, T)
+            return ops.linear(L.w_down, hid, self._buf("yff", torch.float32, L.w_down.shape[0])[:T])
         hid = self._buf("ff", self.dtype, L.w_up.shape[0])[:T]
         ops.linear(L.w_up, h, hid, act=ops.ACT_XIELU, act_params=L.act_params)
         return ops.linear(L.w_down, hid, self._buf("yff", torch.float32, L.w_down.shape[0])[:T])
 
     def _ff_routed(self, L: _Layer, h: torch.Tensor, T: int) -> torch.Tensor:
-        """shared expert + the ``top`` experts with the largest router logits, weighted by the softmax over those logits:
-        one GEMM (router logits, all gate rows, all up rows), the router, ``silu(gate) * up * weight`` per hidden column,
+        """shared expert + the ``top`` experts with the largest router logits, weighted by the softmax over those logits or by
+        their sigmoids (then on the expert's input): one GEMM (router logits, all gate rows, all up rows), the router, ``silu(gate) * up * weight`` per hidden column,
         one GEMM over the down-projections side by side"""
         sp, o, f32 = L.spec, L.ff_off, torch.float32
         p2 = ops.linear(L.w_up, h, self._buf("proj2", f32, L.w_up.shape[0])[:T])
         wt = self._buf("route", f32, max(1, sp.experts))[:T]
         idw = self._buf("keep", f32, 1)[:T]
-        ops.moe_route(p2, o["router"], None, sp.experts, 1, 1, sp.top, 1.0, wt, idw, T)
+        ops.moe_route(p2, o["router"], None, sp.experts, 1, 1, sp.top, 1.0, wt, idw, T, sigmoid=sp.route_kind == "sigmoid_topk")
         hid = self._buf("ff", self.dtype, L.w_down.shape[1])[:T]
         ops.gated_cols(p2, o["gate"], o["up"], hid, o["hidden"], ops.GATE_SILU, T, wt=wt, per=sp.expert_ff, both=True,
-                       lead=sp.shared_ff)
+                       lead=sp.shared_ff, scale_input=sp.scale_input)
         return ops.linear(L.w_down, hid, self._buf("yff", f32, L.w_down.shape[0])[:T])
 
-    def _debug_join(self, x: torch.Tensor, terms, T: int) -> torch.Tensor:
+    def _debug_join(self, x: torch.Tensor, terms, T: int, depth=None) -> torch.Tensor:
         """the residual after the pending outputs have joined it (plain torch, tests only)"""
         W, eps = self.cfg.hidden_size, self.cfg.norm_eps
-        v = x[:T].clone()
+        v = (x if depth is None else depth[3])[:T].clone()
         for y, w, normed in terms:
             y = y[:T, :W]
             if normed:
                 y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps)
             v += y * w if w is not None else y
+        if depth is not None:
+            past, wts, k, _ = depth
+            v = wts[k] * v + torch.einsum("j,jtw->tw", wts[:k], past[:k, :T])
         return v
 
     def _mix_softmax_attention(self, mx: _Mix, proj: torch.Tensor, m, y: torch.Tensor) -> torch.Tensor:
         sp, T = mx.spec, m.n_tokens
         H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
         kc, vc = self.k_cache[self._key(mx)], self.v_cache[self._key(mx)]
+        if sp.talk:
+            return self._mixed_heads(mx, proj, m, y)
         q = self._buf(f"q{mx.idx}", torch.float32, H * D)[:T]
         if sp.qk_norm == "head":        # a norm per head (one weight vector for all heads), no rotation, values as they are
             assert sp.rot is None and not sp.v_norm and mx.off["k"] == mx.off["q"] + H * D and mx.off["v"] == mx.off["k"] + G * D
@@ -741,6 +795,21 @@ class HybridPiece:
         ops.softmax_attention(q, kc, vc, ao, m.block_table, m.q_start, m.q_len, m.kv_len, m.n_seqs, m.max_q, H, G, D, V,
                               sp.window, sp.scale, softcap=sp.softcap, keep_first=sp.keep_first, sink=mx.f.get("sink"))
         return ops.linear(mx.w_o, ao, y)
+
+    def _mixed_heads(self, mx: _Mix, proj: torch.Tensor, m, y: torch.Tensor) -> torch.Tensor:
+        """softmax attention whose scores are mixed across the heads: a mixed query row per head over the whole key row (all
+        key heads), so the attention kernel sees one key head of ``kv_heads * dim`` channels; values per value head"""
+        sp, T = mx.spec, m.n_tokens
+        H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
+        assert sp.qk_norm == "none" and sp.keys_as_values and sp.rot is None and not sp.softcap and not sp.keep_first
+        kc, vc = self.k_cache[self._key(mx)], self.v_cache[self._key(mx)]
+        q = self._buf(f"q{mx.idx}", torch.float32, H * G * D)[:T]
+        ops.talk_prep(proj, mx.off["q"], mx.off["k"], mx.f["talk"], sp.scale, m.slots, q, kc, T, H, G, D)
+        ao = self._buf(f"mix{mx.idx}.{H * V}", self.dtype, mx.w_o.shape[1])[:T]
+        ops.softmax_attention(q, kc.view(kc.shape[0], kc.shape[1], 1, G * D), vc, ao, m.block_table, m.q_start, m.q_len, m.kv_len,
+                              m.n_seqs, m.max_q, H, 1, G * D, V, sp.window, 1.0, sink=mx.f.get("sink"), v_heads=G,
+                              slopes=mx.f.get("slopes"))
+        return ops.linear(mx.w_o, ao, y, bias=mx.b_o)
 
     def _scan_out(self, mx: _Mix, o, gate, off_g, act, aux, m, y) -> torch.Tensor:
         sp, T = mx.spec, m.n_tokens

@@ -220,10 +220,39 @@ def fisopel_tensor_specs(cfg: ModelConfig, layers: Iterable[int], first: bool, l
     return specs
 
 
+def kazolorn_tensor_specs(cfg: ModelConfig, layers: Iterable[int], first: bool, last: bool):
+    """(checkpoint name, shape, kind) of a Kazolorn model; matrices are kept as [out, in].  Kinds as above, plus "depth" (the
+    weights of a depth average: one per earlier result, the layer's own last)."""
+    W = cfg.hidden_size
+    specs = [("embed", (cfg.vocab_size, W), "w")] if first else []
+    for l in layers:
+        sp, p = cfg.layer_specs[l], f"l{l}."
+        m = p + "mix."
+        if sp.mixer != "softmax_attention":
+            raise ValueError(f"{cfg.name}: layer {l} has mixer {sp.mixer!r}, which is not part of this family")
+        H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
+        specs += [(p + "norm1", (W,), "one"), (m + "q", (H * D, W), "w"), (m + "q.b", (H * D,), "bias"),
+                  (m + "k", (G * D, W), "w"), (m + "k.b", (G * D,), "bias"), (m + "talk", (H, H), "hc_mix"),
+                  (m + "o", (W, H * V), "w"), (m + "o.b", (W,), "bias"), (p + "ls1", (W,), "small")]
+        if sp.ff:
+            specs += [(p + "norm2", (W,), "one"), (p + "ls2", (W,), "small")]
+            if sp.ff_kind == "moe":
+                for e in range(sp.experts):
+                    specs += [(f"{p}mlp.e{e}.gate", (sp.expert_ff, W), "w"), (f"{p}mlp.e{e}.up", (sp.expert_ff, W), "w"),
+                              (f"{p}mlp.e{e}.down", (W, sp.expert_ff), "w")]
+                specs.append((p + "mlp.router", (sp.experts, W), "w"))
+            else:
+                specs += [(p + "mlp.up", (sp.ff, W), "w"), (p + "mlp.down", (W, sp.ff), "w"), (p + "mlp.act", (4,), "small")]
+        specs.append((p + "dwa", (l + 2,), "depth"))
+    if last:
+        specs += [("final.norm", (W,), "one"), ("head", (cfg.vocab_size, W), "w")]
+    return specs
+
+
 def hybrid_tensor_specs(cfg: ModelConfig, layers: Iterable[int], first: bool, last: bool):
     """tensor list of a hybrid family (configs with per-layer mixer specs)"""
     fn = {"repudra": repudra_tensor_specs, "lonulix": lonulix_tensor_specs,
-          "fisopel": fisopel_tensor_specs}.get(cfg.family, kepovik_tensor_specs)
+          "fisopel": fisopel_tensor_specs, "kazolorn": kazolorn_tensor_specs}.get(cfg.family, kepovik_tensor_specs)
     return fn(cfg, layers, first, last)
 
 
@@ -252,6 +281,8 @@ def _init_random_hybrid(cfg: ModelConfig, layers, first, last, device, dtype, se
             noise = noise + 1.0
         elif kind == "hc_in":
             noise = noise + 1.0 / shape[0]
+        elif kind == "depth":
+            noise[-1] += 1.0
         elif kind == "hc_mix":
             noise = noise + torch.eye(shape[0], device=noise.device)
         t[name] = noise.to(dtype)

@@ -35,7 +35,7 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "set_decode_state", "hyb_embed", "hyb_commit_prev", "hc_step", "act_cols", "attn_prep",
                         "sig_attention", "delta_scan", "delta_post", "ls_join", "rot_attn_prep", "softmax_attention",
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
-                        "moe_route", "gated_cols", "head_up_gate")
+                        "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm")
 
 
 class _CountedModule:
@@ -464,12 +464,16 @@ def pad_weight(w: torch.Tensor, n_mult: int = 128, k_mult: int = 64) -> torch.Te
     return out
 
 
-def linear(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, act: int = -1, act_params=(0.0, 0.0)) -> torch.Tensor:
-    """out[t, :] = x[t, :] . w^T for padded operands: bf16 on the tcgen05 GEMM (fp32 or bf16 output, optional fused
+def linear(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, act: int = -1, act_params=(0.0, 0.0),
+           bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t, :] = x[t, :] . w^T (+ ``bias``, fp32 of the padded output width) for padded operands: bf16 on the tcgen05 GEMM (fp32 or bf16 output, optional fused
     activation ``act`` = ACT_RELU_SQ / ACT_GELU / ACT_XIELU (with its two numbers ``act_params``) on a bf16 output);
     float32 operands through cuBLAS in true fp32."""
     if w.dtype == torch.float32:
-        torch.mm(x, w.t(), out=out)
+        if bias is not None:
+            torch.addmm(bias, x, w.t(), out=out)
+        else:
+            torch.mm(x, w.t(), out=out)
         if act in (ACT_RELU_SQ, ACT_XIELU):
             native().act_cols(out, 0, out, out.shape[1], COLS_RELU_SQ if act == ACT_RELU_SQ else COLS_XIELU, out.shape[0],
                               float(act_params[0]), float(act_params[1]))
@@ -478,9 +482,9 @@ def linear(w: torch.Tensor, x: torch.Tensor, out: torch.Tensor, act: int = -1, a
         return out
     if act >= 0:
         assert out.dtype == torch.bfloat16
-        gemm(w, x, out=out, epi=EPI_GELU, act_gelu=act, act_p0=float(act_params[0]), act_p1=float(act_params[1]))
+        gemm(w, x, out=out, epi=EPI_GELU, act_gelu=act, bias=bias, act_p0=float(act_params[0]), act_p1=float(act_params[1]))
     else:
-        gemm(w, x, out=out, epi=EPI_PLAIN, out_fp32=out.dtype == torch.float32)
+        gemm(w, x, out=out, epi=EPI_PLAIN, bias=bias, out_fp32=out.dtype == torch.float32)
     return out
 
 
@@ -529,20 +533,24 @@ def delta_post(o, gate, off_g, weight, out, T, H, dv, eps):
 
 # ------------------------------------------------------- parallel-block hybrids (one residual, layer scale, recurrences)
 def ls_join(x, q_start, q_len, n_seqs, max_q, *, terms=(), gamma=None, eps=1e-6, plus_one=False, h=None, rows=None,
-            n_rows=0, gamma2=None, h2=None, replace=False):
+            n_rows=0, gamma2=None, h2=None, replace=False, depth=None):
     """Residual join and next norm in one pass: ``x += sum_k w_k * y_k`` for up to three ``terms = (y, w, normed)``
     (``normed``: y is divided by its root mean square over the width first; ``w`` None = 1), then
     ``h = x / rms(x) * gamma`` (``gamma``: one gain or one per coordinate) as the GEMM operand.  ``rows`` gathers token
     rows (logit rows) instead of walking the spans; the residual is then left as it is.  ``replace``: the new residual
     is the sum of the terms alone.  ``gamma`` None with ``h``: the operand is the residual itself.  ``gamma2`` / ``h2``: a
-    second normed operand of the same rows with its own weight vector (two sublayers side by side, a norm each)."""
+    second normed operand of the same rows with its own weight vector (two sublayers side by side, a norm each).
+    ``depth`` = (past [layers + 1, tokens, W], weights [k + 1], k, entry): the joined row (``entry`` + terms; ``entry`` is the
+    residual that entered the layer, usually ``x`` itself) is kept as ``past[k]`` and ``x`` becomes
+    ``sum_j weights[j] * past[j]`` over ``j <= k``."""
     assert len(terms) <= 3
     t = list(terms) + [(None, None, False)] * (3 - len(terms))
     flat = []
     for y, w, normed in t:
         flat += [y, w, int(bool(normed))]
+    past, wts, k, entry = depth if depth is not None else (None, None, 0, None)
     native().ls_join(x, q_start, q_len, rows, n_rows, n_seqs, max_q, *flat, eps, gamma, int(plus_one), h, gamma2, h2,
-                     int(bool(replace)))
+                     int(bool(replace)), past, wts, int(k), entry)
 
 
 def rot_attn_prep(proj, off_q, off_k, off_v, qn, kn, freq, rdims, amp, positions, slots, q_out, k_cache, v_cache, T, H, G,
@@ -552,11 +560,13 @@ def rot_attn_prep(proj, off_q, off_k, off_v, qn, kn, freq, rdims, amp, positions
 
 
 def softmax_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, V, window,
-                      scale, softcap=0.0, keep_first=0, sink=None):
+                      scale, softcap=0.0, keep_first=0, sink=None, v_heads=0, slopes=None):
     """causal softmax attention over the paged cache; ``window`` > 0: the last ``window`` keys and the first ``keep_first``
-    ones; ``softcap`` > 0: ``score <- softcap * tanh(score / softcap)``; ``sink`` [H]: ``exp(sink_h)`` joins the denominator"""
+    ones; ``softcap`` > 0: ``score <- softcap * tanh(score / softcap)``; ``sink`` [H]: ``exp(sink_h)`` joins the denominator;
+    ``slopes`` [H]: ``score -= slopes[h] * (query position - key position)``; ``v_heads``: value heads per cache row when they
+    differ from the ``G`` key heads (head ``h`` reads value head ``h // (H / v_heads)``)"""
     native().softmax_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, V,
-                               window, float(scale), float(softcap), int(keep_first), sink)
+                               window, float(scale), float(softcap), int(keep_first), sink, int(v_heads), slopes)
 
 
 def short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q):
@@ -619,18 +629,32 @@ def rot_heads(src, off, dst, H, Dh, freq, rdims, positions, T, slots=None, roff=
     native().rot_heads(src, off, dst, H, Dh, freq, rdims, positions, slots, T, int(roff), float(amp), freq_lo)
 
 
-def moe_route(proj, off, corr, n_real, count, keep, top, scale, wt, idw, T, sel_idx=None, sel_w=None):
+def talk_prep(proj, off_q, off_k, talk, scale, slots, q_out, k_cache, T, H, G, D):
+    """Mixed heads (``score_h <- sum_g talk[h, g] score_g``) in absorbed form: one query row per head over ALL key heads of a
+    cache row, ``q_out[t, h, c] = scale * sum over the heads g that read key head c of talk[h, g] q[t, g]`` ([T, H * G * D],
+    float or bf16), and the key rows (``proj`` columns ``off_k`` ..) into the paged cache."""
+    native().talk_prep(proj, off_q, off_k, talk, float(scale), slots, q_out, k_cache, T, H, G, D)
+
+
+def poly_norm(x, off, w, out, n, eps, T):
+    """``out[t, c] = w0 N(z) + w1 N(z^2) + w2 N(z^3) + w3`` for ``z = x[t, off : off + n]``, powers element by element, ``N``
+    divides a row by its root mean square"""
+    native().poly_norm(x, off, w, out, n, float(eps), T)
+
+
+def moe_route(proj, off, corr, n_real, count, keep, top, scale, wt, idw, T, sel_idx=None, sel_w=None, sigmoid=False):
     """softmax router over ``corr.numel()`` outputs (the last ones beyond ``n_real`` are identity experts): dense weight
     rows ``wt`` [T, n_real] and the summed identity weight ``idw`` [T]; optionally the choices in order.  ``corr`` None:
-    ``n_real`` outputs, the largest logits are chosen and the weights are the softmax over the chosen logits alone"""
+    ``n_real`` outputs, the largest logits are chosen and the weights are the softmax over the chosen logits alone; ``sigmoid``: their sigmoids times ``scale``"""
     native().moe_route(proj, off, corr, corr.numel() if corr is not None else n_real, n_real, count, keep, top,
-                       float(scale), wt, idw, sel_idx, sel_w, T)
+                       float(scale), wt, idw, sel_idx, sel_w, T, int(bool(sigmoid)))
 
 
-def gated_cols(x, off_a, off_b, out, n, act, T, wt=None, per=0, both=False, lead=0):
+def gated_cols(x, off_a, off_b, out, n, act, T, wt=None, per=0, both=False, lead=0, scale_input=False):
     """``out[t, c] = act(x[t, off_a + c]) * x[t, off_b + c]``, or ``* wt[t, c // per]`` with per-expert weights, or
-    (``both``) times the two of them, the first ``lead`` columns having weight 1 (a shared expert in front of the routed ones)"""
-    native().gated_cols(x, off_a, off_b, wt, per, out, n, act, T, int(bool(both)), int(lead))
+    (``both``) times the two of them, the first ``lead`` columns having weight 1 (a shared expert in front of the routed ones);
+    ``scale_input`` (with ``both``): ``act(w a) * (w b)``, the expert's input carries the weight"""
+    native().gated_cols(x, off_a, off_b, wt, per, out, n, act, T, 2 if scale_input else int(bool(both)), int(lead))
 
 
 def head_up_gate(a, U, out, T, H, V, C, gate=None, off_g=0):

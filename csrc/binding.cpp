@@ -539,7 +539,8 @@ void delta_post(const Tensor& o, const Tensor& gate, int64_t off_g, const Tensor
 void ls_join(const Tensor& x, const Tensor& q_start, const Tensor& q_len, const OptT& rows, int64_t n_rows, int64_t n_seqs,
              int64_t max_q, const OptT& y0, const OptT& w0, int64_t norm0, const OptT& y1, const OptT& w1, int64_t norm1,
              const OptT& y2, const OptT& w2, int64_t norm2, double eps, const OptT& gamma, int64_t plus_one,
-             const OptT& h, const OptT& gamma2, const OptT& h2, int64_t replace) {
+             const OptT& h, const OptT& gamma2, const OptT& h2, int64_t replace, const OptT& past, const OptT& dw, int64_t k,
+             const OptT& xin) {
   c10::cuda::CUDAGuard guard(x.device());
   const bool has_h = h.has_value() && h->defined();
   const bool has_g = gamma.has_value() && gamma->defined();
@@ -550,6 +551,10 @@ void ls_join(const Tensor& x, const Tensor& q_start, const Tensor& q_len, const 
               "ls_join: the second operand needs the first one and a weight vector of its own");
   auto ld = [](const OptT& t) { return (t.has_value() && t->defined()) ? static_cast<int>(t->stride(0)) : 0; };
   const int W = static_cast<int>(x.size(-1));
+  const bool has_past = past.has_value() && past->defined();
+  TORCH_CHECK(!has_past || (dw.has_value() && dw->numel() > k && past->dim() == 3 && past->size(0) > k &&
+                            past->size(-1) == W && past->stride(1) == W && k >= 0),
+              "ls_join: a depth average needs [layers + 1, tokens, W] rows and k + 1 weights");
   check(b2b::launch_ls_join(const_cast<float*>(fp(x)), ip(q_start), ip(q_len),
                             (rows.has_value() && rows->defined()) ? ip(*rows) : nullptr, static_cast<int>(n_rows),
                             static_cast<int>(n_seqs), static_cast<int>(max_q), fp_or_null(y0), ld(y0), fp_or_null(w0),
@@ -558,7 +563,9 @@ void ls_join(const Tensor& x, const Tensor& q_start, const Tensor& q_len, const 
                             fp_or_null(gamma), (has_g && gamma->numel() > 1) ? 1 : 0, static_cast<int>(plus_one),
                             has_h ? h->data_ptr() : nullptr, has_h ? static_cast<int>(h->stride(0)) : 0, W,
                             has_h ? is_f32(*h) : 1, has_h2 ? fp(*gamma2) : nullptr, has_h2 ? h2->data_ptr() : nullptr,
-                            has_h2 ? static_cast<int>(h2->stride(0)) : 0, static_cast<int>(replace), cur_stream()),
+                            has_h2 ? static_cast<int>(h2->stride(0)) : 0, static_cast<int>(replace), fp_or_null(xin),
+                            has_past ? const_cast<float*>(fp(*past)) : nullptr, fp_or_null(dw),
+                            has_past ? static_cast<size_t>(past->stride(0)) : 0, static_cast<int>(k), cur_stream()),
         "ls_join");
 }
 
@@ -581,9 +588,11 @@ void rot_attn_prep(const Tensor& proj, int64_t off_q, int64_t off_k, int64_t off
 void softmax_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& out,
                        const Tensor& block_table, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len,
                        int64_t n_seqs, int64_t max_q, int64_t H, int64_t G, int64_t D, int64_t V, int64_t window,
-                       double scale, double softcap, int64_t keep_first, const OptT& sink) {
+                       double scale, double softcap, int64_t keep_first, const OptT& sink, int64_t v_heads,
+                       const OptT& slopes) {
   c10::cuda::CUDAGuard guard(q.device());
   TORCH_CHECK(!(sink.has_value() && sink->defined()) || sink->numel() >= H, "softmax_attention: one sink per head");
+  TORCH_CHECK(!(slopes.has_value() && slopes->defined()) || slopes->numel() >= H, "softmax_attention: one slope per head");
   TORCH_CHECK(k_cache.scalar_type() == out.scalar_type() && v_cache.scalar_type() == out.scalar_type(),
               "softmax_attention: cache and output dtypes must match");
   check(b2b::launch_softmax_attention(fp(q), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
@@ -593,8 +602,21 @@ void softmax_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
                                       static_cast<int>(G), static_cast<int>(D), static_cast<int>(V),
                                       static_cast<int>(window), static_cast<float>(scale),
                                       static_cast<int>(v_cache.stride(1)), is_f32(out), static_cast<float>(softcap),
-                                      static_cast<int>(keep_first), fp_or_null(sink), cur_stream()),
+                                      static_cast<int>(keep_first), fp_or_null(sink), static_cast<int>(v_heads),
+                                      fp_or_null(slopes), cur_stream()),
         "softmax_attention");
+}
+
+// proj [T, >= ...] fp32: q (H * D columns at off_q), k (G * D at off_k); q_out [T, H * G * D] float or bf16; cache rows [G, D]
+void talk_prep(const Tensor& proj, int64_t off_q, int64_t off_k, const Tensor& talk, double scale, const Tensor& slots,
+               const Tensor& q_out, const Tensor& k_cache, int64_t T, int64_t H, int64_t G, int64_t D) {
+  c10::cuda::CUDAGuard guard(proj.device());
+  TORCH_CHECK(talk.numel() == H * H && q_out.stride(0) == H * G * D && q_out.size(0) >= T, "talk_prep: sizes");
+  check(b2b::launch_talk_prep(fp(proj), static_cast<int>(proj.stride(0)), static_cast<int>(off_q), static_cast<int>(off_k),
+                              fp(talk), static_cast<float>(scale), ip(slots), q_out.data_ptr(), k_cache.data_ptr(),
+                              static_cast<int>(T), static_cast<int>(H), static_cast<int>(G), static_cast<int>(D),
+                              is_f32(q_out), is_f32(k_cache), cur_stream()),
+        "talk_prep");
 }
 
 void short_conv(const Tensor& x, int64_t off, const Tensor& w, const Tensor& tail, const Tensor& y, const Tensor& q_start,
@@ -704,7 +726,7 @@ void rot_heads(const Tensor& src, int64_t off, const Tensor& dst, int64_t H, int
 
 void moe_route(const Tensor& proj, int64_t off, const OptT& corr, int64_t E, int64_t n_real, int64_t count, int64_t keep,
                int64_t top, double scale, const Tensor& wt, const Tensor& idw, const OptT& sel_idx, const OptT& sel_w,
-               int64_t T) {
+               int64_t T, int64_t sigmoid) {
   c10::cuda::CUDAGuard guard(proj.device());
   const bool has_sel = sel_idx.has_value() && sel_idx->defined();
   TORCH_CHECK(!(corr.has_value() && corr->defined()) || corr->numel() == E, "moe_route: one correction per router output");
@@ -713,8 +735,18 @@ void moe_route(const Tensor& proj, int64_t off, const OptT& corr, int64_t E, int
                               static_cast<int>(keep), static_cast<int>(top), static_cast<float>(scale),
                               const_cast<float*>(fp(wt)), static_cast<int>(wt.stride(0)), const_cast<float*>(fp(idw)),
                               has_sel ? const_cast<int*>(ip(*sel_idx)) : nullptr,
-                              const_cast<float*>(fp_or_null(sel_w)), static_cast<int>(T), cur_stream()),
+                              const_cast<float*>(fp_or_null(sel_w)), static_cast<int>(T), static_cast<int>(sigmoid),
+                              cur_stream()),
         "moe_route");
+}
+
+void poly_norm(const Tensor& in, int64_t off, const Tensor& w, const Tensor& out, int64_t n, double eps, int64_t T) {
+  c10::cuda::CUDAGuard guard(in.device());
+  TORCH_CHECK(w.numel() == 4, "poly_norm: four numbers");
+  check(b2b::launch_poly_norm(fp(in), static_cast<int>(in.stride(0)), static_cast<int>(off), fp(w), out.data_ptr(),
+                              static_cast<int>(out.stride(0)), static_cast<int>(n), static_cast<float>(eps),
+                              static_cast<int>(T), is_f32(out), cur_stream()),
+        "poly_norm");
 }
 
 void gated_cols(const Tensor& in, int64_t off_a, int64_t off_b, const OptT& wt, int64_t per, const Tensor& out, int64_t n,
@@ -793,6 +825,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("ls_join", &ls_join);
   m.def("rot_attn_prep", &rot_attn_prep);
   m.def("softmax_attention", &softmax_attention);
+  m.def("talk_prep", &talk_prep);
   m.def("short_conv", &short_conv);
   m.def("mlstm_gates", &mlstm_gates);
   m.def("lin_scan", &lin_scan);
@@ -801,6 +834,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("latent_prep", &latent_prep);
   m.def("rot_heads", &rot_heads);
   m.def("moe_route", &moe_route);
+  m.def("poly_norm", &poly_norm);
   m.def("gated_cols", &gated_cols);
   m.def("head_up_gate", &head_up_gate);
 }

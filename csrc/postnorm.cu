@@ -7,7 +7,8 @@
 //   * latent_prep      latent attention: RMS norm of the query latent (-> operand of the query up-projection), RMS norm of
 //                      the key/value latent and rotation of the shared rotary key part -> one cache row [rotary | latent]
 //   * rot_heads        rotary positions on the first channels of every head of a projection -> dense query rows
-//   * moe_route        softmax router with a selection-only correction, group-limited top-k and identity experts
+//   * poly_norm        a N(z) + b N(z^2) + c N(z^3) + e over whole rows of a projection (N: division by the root mean square)
+//   * moe_route        softmax router with a selection-only correction, group-limited top-k and identity experts; top-k sigmoid scores
 //   * gated_cols       out = act(a) * b for two column blocks, or act(a) * per-expert weight (routed experts run as one
 //                      stacked up-projection whose hidden columns are scaled by the token's weight for their expert), or both
 //   * head_up_gate     a [V, C] matrix per head applied to per-head latent rows, times a sigmoid output gate
@@ -263,6 +264,72 @@ __global__ void rot_heads_kernel(const float* __restrict__ src, int ld, int off,
   dst[static_cast<size_t>(t) * n + c] = v;
 }
 
+// ------------------------------------------------------------------------------------------- PolyNorm
+// out[t, c] = w0 z / rms(z) + w1 z^2 / rms(z^2) + w2 z^3 / rms(z^3) + w3, z = in[t, off + c], c < n; rms over the row's n
+// values, eps inside the root.  One block per row; NV > 0: the row stays in registers (NV float4 per thread), NV = 0: it is
+// read twice.
+constexpr int PN_THREADS = 256;
+template <typename OT, int NV>
+__global__ void __launch_bounds__(PN_THREADS)
+    poly_norm_kernel(const float* __restrict__ in, int ld_in, int off, const float* __restrict__ w, OT* __restrict__ out,
+                     int ld_out, int n, float eps) {
+  pdl_begin();
+  __shared__ float part[3][PN_THREADS / 32];
+  const size_t t = blockIdx.x;
+  const float* zr = in + t * ld_in + off;
+  OT* orow = out + t * ld_out;
+  float4 v[NV > 0 ? NV : 1];
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto add = [&](float z) {
+    const float q = z * z;
+    s2 += q;
+    s4 += q * q;
+    s6 += q * q * q;
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = (k * PN_THREADS + threadIdx.x) * 4;
+      v[k] = c < n ? *reinterpret_cast<const float4*>(zr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      add(v[k].x); add(v[k].y); add(v[k].z); add(v[k].w);
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += PN_THREADS) add(zr[c]);
+  }
+  s2 = warp_sum_(s2);
+  s4 = warp_sum_(s4);
+  s6 = warp_sum_(s6);
+  const int warp = threadIdx.x >> 5;
+  if ((threadIdx.x & 31) == 0) {
+    part[0][warp] = s2;
+    part[1][warp] = s4;
+    part[2][warp] = s6;
+  }
+  __syncthreads();
+  s2 = s4 = s6 = 0.f;
+#pragma unroll
+  for (int k = 0; k < PN_THREADS / 32; ++k) {
+    s2 += part[0][k];
+    s4 += part[1][k];
+    s6 += part[2][k];
+  }
+  const float fn = static_cast<float>(n);
+  const float a = w[0] / sqrtf(s2 / fn + eps), b = w[1] / sqrtf(s4 / fn + eps), c3 = w[2] / sqrtf(s6 / fn + eps), e = w[3];
+  auto val = [&](float z) { return ((c3 * z + b) * z + a) * z + e; };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = (k * PN_THREADS + threadIdx.x) * 4;
+      if (c < n) st4(orow + c, make_float4(val(v[k].x), val(v[k].y), val(v[k].z), val(v[k].w)));
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += PN_THREADS) stf(orow, c, val(zr[c]));
+  }
+}
+
 // ------------------------------------------------------------------------------------------- router
 // One warp per token.  z = logits [E] (fp32, column off of proj), s = softmax(z); choice = s + corr; consecutive experts
 // are bundled into `count` equal groups, a group's score is its largest choice, only experts of the `keep` best groups stay
@@ -270,11 +337,12 @@ __global__ void rot_heads_kernel(const float* __restrict__ src, int ld, int off,
 // s / (sum of the chosen s + 1e-20) * scale (= the softmax over the chosen logits alone when scale = 1).  corr == nullptr:
 // the choice is made on the logits themselves.  Experts n_real .. E - 1 are identity experts: their weights are summed into
 // idw[t]; wt [T, ld_wt] receives the dense weight row of the real experts (0 = not chosen).  sel_idx / sel_w [T, top]
-// (optional) list the choices in order.
+// (optional) list the choices in order.  sigmoid != 0 (with corr == nullptr): the weights are sigmoid(z) * scale of the chosen
+// logits, not renormalised (the largest logits have the largest sigmoids).
 __global__ void __launch_bounds__(128)
     moe_route_kernel(const float* __restrict__ proj, int ld, int off, const float* __restrict__ corr, int E, int n_real,
                      int count, int keep, int top, float scale, float* __restrict__ wt, int ld_wt,
-                     float* __restrict__ idw, int* __restrict__ sel_idx, float* __restrict__ sel_w, int T) {
+                     float* __restrict__ idw, int* __restrict__ sel_idx, float* __restrict__ sel_w, int T, int sigmoid) {
   pdl_begin();
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -297,7 +365,7 @@ __global__ void __launch_bounds__(128)
   }
   den = warp_sum_(den);
   for (int j = lane; j < E; j += 32) {
-    const float p = s[j] / den;
+    const float p = sigmoid ? sigmoid_(z[j]) : s[j] / den;
     s[j] = p;
     ch[j] = corr != nullptr ? p + corr[j] : z[j];      // no correction: the largest logits themselves are chosen
   }
@@ -362,7 +430,7 @@ __global__ void __launch_bounds__(128)
   float keep_w = 0.f;
   for (int k = lane; k < top; k += 32) {
     const int j = k < n_sel ? sel[k] : -1;
-    const float wgt = j >= 0 ? s[j] / (tot + 1e-20f) * scale : 0.f;
+    const float wgt = j >= 0 ? (sigmoid ? s[j] : s[j] / (tot + 1e-20f)) * scale : 0.f;
     if (j >= 0 && j < n_real) wt[static_cast<size_t>(t) * ld_wt + j] = wgt;
     if (j >= n_real) keep_w += wgt;
     if (sel_idx != nullptr) sel_idx[static_cast<size_t>(t) * top + k] = j;
@@ -375,7 +443,8 @@ __global__ void __launch_bounds__(128)
 // ------------------------------------------------------------------------------------------- gated columns
 // out[t, c] = act(in[t, off_a + c]) * (wt == nullptr ? in[t, off_b + c] : wt[t, c / per]) for c < n.  both != 0 (with wt):
 // act(a) * in[t, off_b + c] * weight, where the first `lead` columns have weight 1 and column c >= lead has
-// wt[t, (c - lead) / per] (gated experts side by side behind a shared one).
+// wt[t, (c - lead) / per] (gated experts side by side behind a shared one).  both == 2: act(w a) * (w b), the weight scales what
+// goes into the expert.
 // act: 0 silu, 1 exact (erf) gelu, 2 tanh gelu.  Four columns per thread when every offset allows 16-byte accesses.
 __device__ __forceinline__ float act_(float z, int act) {
   if (act == 0) return z / (1.f + expf(-z));
@@ -391,8 +460,8 @@ __global__ void __launch_bounds__(256)
   if (e >= static_cast<long long>(T) * n) return;
   const int c = static_cast<int>(e % n);
   const size_t t = static_cast<size_t>(e / n);
-  const float a = act_(in[t * ld_in + off_a + c], act);
   float b = wt != nullptr ? (c < lead ? 1.f : wt[t * ld_wt + (c - lead) / per]) : in[t * ld_in + off_b + c];
+  const float a = act_(in[t * ld_in + off_a + c] * (both == 2 ? b : 1.f), act);
   if (both && wt != nullptr) b *= in[t * ld_in + off_b + c];
   stf(out, t * ld_out + c, a * b);
 }
@@ -406,11 +475,12 @@ __global__ void __launch_bounds__(256)
   const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
   if (c >= n) return;
   const size_t t = blockIdx.y;
-  const float4 a = *reinterpret_cast<const float4*>(in + t * ld_in + off_a + c);
+  float4 a = *reinterpret_cast<const float4*>(in + t * ld_in + off_a + c);
   float4 b;
   if (wt != nullptr) {
     const float wv = c < lead ? 1.f : wt[t * ld_wt + (c - lead) / per];      // per and lead are multiples of four: one expert for the four columns
     b = make_float4(wv, wv, wv, wv);
+    if (both == 2) a = make_float4(wv * a.x, wv * a.y, wv * a.z, wv * a.w);
     if (both) {
       const float4 u = *reinterpret_cast<const float4*>(in + t * ld_in + off_b + c);
       b = make_float4(wv * u.x, wv * u.y, wv * u.z, wv * u.w);
@@ -672,8 +742,9 @@ int launch_rot_heads(const float* src, int ld, int off, float* dst, int H, int D
 
 int launch_moe_route(const float* proj, int ld, int off, const float* corr, int E, int n_real, int count, int keep,
                      int top, float scale, float* wt, int ld_wt, float* idw, int* sel_idx, float* sel_w, int T,
-                     cudaStream_t s) {
+                     int sigmoid, cudaStream_t s) {
   if (T <= 0) return 0;
+  if (sigmoid && corr != nullptr) return -2;
   if (E <= 0 || n_real < 0 || n_real > E || count <= 0 || E % count != 0 || top <= 0 || top > E) return -2;
   if (corr == nullptr && count > 1 && keep < count) return -2;      // group-limited choice is defined on corrected scores
   int warps = 4;
@@ -681,7 +752,32 @@ int launch_moe_route(const float* proj, int ld, int off, const float* corr, int 
   const size_t smem = static_cast<size_t>(warps) * 4 * E * sizeof(float);
   if (smem > 48 * 1024) return -2;
   launch_kernel(moe_route_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, s, 1u, proj, ld, off, corr, E,
-                n_real, count, keep, top, scale, wt, ld_wt, idw, sel_idx, sel_w, T);
+                n_real, count, keep, top, scale, wt, ld_wt, idw, sel_idx, sel_w, T, sigmoid);
+  return last_error();
+}
+
+int launch_poly_norm(const float* in, int ld_in, int off, const float* w, void* out, int ld_out, int n, float eps, int T,
+                     int f32, cudaStream_t s) {
+  if (T <= 0 || n <= 0) return 0;
+  const bool vec = n % 4 == 0 && ld_in % 4 == 0 && off % 4 == 0 && ld_out % 4 == 0 &&
+                   reinterpret_cast<uintptr_t>(in) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0;
+  const int nv = vec ? (n + 4 * PN_THREADS - 1) / (4 * PN_THREADS) : 0;
+#define B2B_PN(OT, NV)                                                                                                  \
+  launch_kernel(poly_norm_kernel<OT, NV>, dim3(T), dim3(PN_THREADS), 0, s, 1u, in, ld_in, off, w, static_cast<OT*>(out), \
+                ld_out, n, eps)
+#define B2B_PN_T(OT)                                                                                                    \
+  do {                                                                                                                  \
+    if (nv == 1) B2B_PN(OT, 1);                                                                                         \
+    else if (nv == 2) B2B_PN(OT, 2);                                                                                    \
+    else if (nv > 2 && nv <= 4) B2B_PN(OT, 4);                                                                          \
+    else if (nv > 4 && nv <= 8) B2B_PN(OT, 8);                                                                          \
+    else if (nv > 8 && nv <= 16) B2B_PN(OT, 16);                                                                        \
+    else B2B_PN(OT, 0);                                                                                                 \
+  } while (0)
+  if (f32) B2B_PN_T(float);
+  else B2B_PN_T(bf16);
+#undef B2B_PN_T
+#undef B2B_PN
   return last_error();
 }
 

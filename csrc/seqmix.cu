@@ -3,12 +3,15 @@
 //   * ls_join            one residual stream: x += sum_k w_k * (optionally width-normed) y_k, then the RMS norm of the
 //                        next block (one gain for all coordinates, or a vector) written as the GEMM operand; optionally a
 //                        second normed operand with its own weights (a norm per sublayer of a parallel block), a replace
-//                        mode (the residual entering a pass of a looped range of layers) and a plain operand copy
+//                        mode (the residual entering a pass of a looped range of layers), a plain operand copy, and a
+//                        depth average (the row becomes a weighted sum of itself and earlier layers' kept rows)
+//   * talk_prep          softmax attention with mixed heads, absorbed form: per head one query row over all key heads
 //   * rot_attn_prep      softmax attention: RMS norm over the WHOLE q / k projection, rotary positions on the first
 //                        `rdims` channels of every head (pairs 2i, 2i+1; frequencies from a table, so any scaling rule
 //                        is a host matter), per-head value norm, K / V rows into the paged cache
 //   * softmax_attention  causal softmax attention over the paged cache, key width != value width, grouped heads, optional
-//                        window with kept first keys, optional score cap, optional sink in the denominator; an
+//                        window with kept first keys, optional score cap, optional sink in the denominator, optional
+//                        linear distance bias, value heads counted apart from key heads; an
 //                        exact CUDA-core kernel (one warp per query and head, online softmax) and a tensor-core kernel
 //                        for spans in the bf16 mode
 //   * short_conv         causal per-channel convolution over time + silu, with the last taps-1 inputs per sequence slot
@@ -87,8 +90,17 @@ struct JoinTerm {
 // of squares, pass 3 writes the operand.  VEC: 16-byte accesses (W and every row stride multiples of 4).
 // replace: the new residual row is the sum of the terms alone (the old row is not read).  gamma == nullptr: the operand is
 // the residual row itself.  gamma2 / h2: a second normed operand of the same row (blocks whose two sublayers have a norm each).
+// past (depth averages): the joined row is kept as past[k] ([entry of stride `dstride` floats][token][W]) and the residual
+// row becomes sum_j dw[j] past[j] over j <= k; xin: the row that entered the layer (x itself, or past[0] in the first layer).
 // grid (groups of LSJ_WARPS / WPT tokens, sequences) or (groups of rows); dynamic smem LSJ_WARPS / WPT * W floats.
 constexpr int LSJ_WARPS = 4;
+
+struct DepthTerm {
+  float* past;             // null: no depth average
+  const float* dw;         // [k + 1]
+  size_t dstride;
+  int k;
+};
 
 template <bool VEC> struct Ld4;
 template <> struct Ld4<true> {
@@ -120,7 +132,8 @@ __global__ void __launch_bounds__(32 * LSJ_WARPS)
     ls_join_kernel(float* __restrict__ x, const int* __restrict__ q_start, const int* __restrict__ q_len,
                    const int* __restrict__ rows, int n_rows, JoinTerm a, JoinTerm b, JoinTerm c, float eps,
                    const float* __restrict__ gamma, int gstride, int plus_one, OT* __restrict__ h, int ld_h, int W,
-                   const float* __restrict__ gamma2, OT* __restrict__ h2, int ld_h2, int replace) {
+                   const float* __restrict__ gamma2, OT* __restrict__ h2, int ld_h2, int replace,
+                   const float* __restrict__ xin, DepthTerm dep) {
   pdl_begin();
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
@@ -156,9 +169,10 @@ __global__ void __launch_bounds__(32 * LSJ_WARPS)
     r[k] = 1.f / sqrtf(total(ss) * inv_w + eps);
   }
   float* xr = x + static_cast<size_t>(t) * W;
+  const float* xi = xin + static_cast<size_t>(t) * W;
   float ss = 0.f;
   for (int i = lane; i < nv; i += NL) {
-    float4 v = replace ? make_float4(0.f, 0.f, 0.f, 0.f) : Ld4<VEC>::ld(xr, i);
+    float4 v = replace ? make_float4(0.f, 0.f, 0.f, 0.f) : Ld4<VEC>::ld(xi, i);
 #pragma unroll
     for (int k = 0; k < 3; ++k) {
       if (terms[k].y == nullptr) continue;
@@ -170,6 +184,23 @@ __global__ void __launch_bounds__(32 * LSJ_WARPS)
         v.y += yv.y * r[k] * wv.y;
         v.z += yv.z * r[k] * wv.z;
         v.w += yv.w * r[k] * wv.w;
+      }
+    }
+    if (dep.past != nullptr) {
+      float* pr = dep.past + static_cast<size_t>(t) * W;
+      if (rows == nullptr) Ld4<VEC>::st(pr + dep.k * dep.dstride, i, v);
+      const float wk = dep.dw[dep.k];
+      v.x *= wk; v.y *= wk; v.z *= wk; v.w *= wk;
+#pragma unroll 4
+      for (int j = 0; j < dep.k; ++j) {
+        const float4 pv = Ld4<VEC>::ld(pr + j * dep.dstride, i);
+        const float wj = dep.dw[j];
+        v.x += wj * pv.x;
+        if (VEC) {
+          v.y += wj * pv.y;
+          v.z += wj * pv.z;
+          v.w += wj * pv.w;
+        }
       }
     }
     ss += v.x * v.x + (VEC ? v.y * v.y + v.z * v.z + v.w * v.w : 0.f);
@@ -292,6 +323,72 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// ------------------------------------------------------------------- softmax attention: mixed heads, absorbed form
+// score_h = sum_g talk[h, g] scale (q_g . k_(g's key head)) = qm_h . [k_0 | k_1 | ...] with, per key head c,
+//     qm[h, c, :] = scale * sum over the heads g of key head c of talk[h, g] q_g
+// so a head needs ONE dot product with the whole cached key row (G * D channels) and no exchange with other heads.
+// proj [T, ld] fp32 holds q (H*D) at off_q, k (G*D) at off_k.  One block per token: the query row and the matrix (transposed,
+// rows padded to a multiple of 4) in shared memory; a thread owns E adjacent channels of one key head and writes them for
+// every head.  qm -> q_out [T, H*G*D], key row -> cache.
+template <typename CT, int E> __device__ __forceinline__ void st_run(CT* p, const float (&v)[E]) {
+  if constexpr (E == 1) stf(p, 0, v[0]);
+  else if constexpr (sizeof(CT) == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *reinterpret_cast<uint2*>(p) = [&] {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    return make_uint2(*reinterpret_cast<unsigned*>(&a), *reinterpret_cast<unsigned*>(&b));
+  }();
+}
+template <typename QT, typename CT, int E>
+__global__ void __launch_bounds__(256)
+    talk_prep_kernel(const float* __restrict__ proj, int ld, int off_q, int off_k, const float* __restrict__ talk,
+                     float scale, const int* __restrict__ slots, QT* __restrict__ q_out, CT* __restrict__ k_cache, int H,
+                     int G, int D) {
+  pdl_begin();
+  extern __shared__ __align__(16) float tp[];
+  const int t = blockIdx.x, slot = slots[t];
+  if (slot < 0) return;                               // padding row of a bucketed chunk (block-uniform)
+  const int Hp = (H + 3) & ~3, nq = H * D, nk = G * D, per = H / G;
+  float* qs = tp;                                     // [H * D]
+  float* tt = tp + ((nq + 3) & ~3);                   // [H (mixed from)][Hp (mixed into)]
+  const float* row = proj + static_cast<size_t>(t) * ld;
+  for (int i = threadIdx.x; i < nq; i += blockDim.x) qs[i] = row[off_q + i] * scale;
+  for (int i = threadIdx.x; i < H * Hp; i += blockDim.x) {
+    const int g = i / Hp, h = i % Hp;
+    tt[i] = h < H ? talk[h * H + g] : 0.f;
+  }
+  for (int i = threadIdx.x; i < nk; i += blockDim.x) stf(k_cache, static_cast<size_t>(slot) * nk + i, row[off_k + i]);
+  __syncthreads();
+  QT* qo = q_out + static_cast<size_t>(t) * H * nk;
+  for (int c = threadIdx.x * E; c < nk; c += blockDim.x * E) {
+    const int kv = c / D, d = c % D;                  // (E divides D: the run stays inside one key head)
+    for (int h0 = 0; h0 < H; h0 += 4) {
+      float acc[4][E];
+#pragma unroll
+      for (int a = 0; a < 4; ++a)
+#pragma unroll
+        for (int e = 0; e < E; ++e) acc[a][e] = 0.f;
+      for (int g = kv * per; g < (kv + 1) * per; ++g) {
+        const float4 w = *reinterpret_cast<const float4*>(tt + g * Hp + h0);
+        const float wa[4] = {w.x, w.y, w.z, w.w};
+        float qv[E];
+        if constexpr (E == 4) {
+          const float4 v = *reinterpret_cast<const float4*>(qs + g * D + d);
+          qv[0] = v.x; qv[1] = v.y; qv[2] = v.z; qv[3] = v.w;
+        } else {
+          qv[0] = qs[g * D + d];
+        }
+#pragma unroll
+        for (int a = 0; a < 4; ++a)
+#pragma unroll
+          for (int e = 0; e < E; ++e) acc[a][e] += wa[a] * qv[e];
+      }
+#pragma unroll
+      for (int a = 0; a < 4; ++a)
+        if (h0 + a < H) st_run<QT, E>(qo + static_cast<size_t>(h0 + a) * nk + c, acc[a]);
+    }
+  }
+}
+
 // dot product of a shared-memory fp32 vector with a cache row, 128-bit loads when the row allows it
 template <typename T> __device__ __forceinline__ float dot_row(const float* q, const T* k, int n, bool vec);
 template <> __device__ __forceinline__ float dot_row<float>(const float* q, const float* k, int n, bool vec) {
@@ -330,6 +427,8 @@ template <> __device__ __forceinline__ float dot_row<bf16>(const float* q, const
 // out[t, h, :] = sum_j softmax_j(q_t . k_j * scale) v_j over the keys j <= i, and j > i - window when window > 0
 // (the first keep_first keys stay visible whatever the window).  softcap > 0: score <- softcap * tanh(score / softcap).
 // sink [H] (optional): exp(sink_h) joins the denominator of head h; it has no key and no value.
+// slope [H] (optional): slope_h * (i - j) is taken off the score of head h.  Gv value heads: head h reads value head
+// h / (H / Gv) (Gv = G unless the key row of all heads is one vector, see talk_prep).
 // Positions count from the start of the sequence: i = kv_len - q_len + index in span.  One warp per (query, head): a
 // pass over 32 keys computes one score per lane, rescales the running sums, then the lanes own value channels.
 // grid (query tiles of 4, heads, sequences), 128 threads, dynamic smem 4 * D floats.
@@ -350,7 +449,8 @@ __global__ void __launch_bounds__(32 * (WPQ > 1 ? WPQ : SMX_WARPS))
                              OT* __restrict__ out, int ld_out, const int* __restrict__ block_table, int max_pages,
                              const int* __restrict__ q_start, const int* __restrict__ q_len,
                              const int* __restrict__ kv_len, int H, int G, int D, int V, int window, float scale, int ldv,
-                             float softcap, int keep_first, const float* __restrict__ sink) {
+                             float softcap, int keep_first, const float* __restrict__ sink, int Gv,
+                             const float* __restrict__ slope) {
   pdl_begin();
   extern __shared__ float qs_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -361,7 +461,8 @@ __global__ void __launch_bounds__(32 * (WPQ > 1 ? WPQ : SMX_WARPS))
   const int t = q_start[s] + i;
   const int pi = kv_len[s] - n + i;
   const int lo = window > 0 ? max(0, pi - window + 1) : 0;
-  const int g = hd / (H / G);
+  const int g = hd / (H / G), gv = hd / (H / Gv);
+  const float sl = slope != nullptr ? slope[hd] : 0.f;
   float* qs = qs_all + (WPQ > 1 ? 0 : warp * D);
   const float* qrow = q + (static_cast<size_t>(t) * H + hd) * D;
   if (WPQ > 1) {
@@ -396,6 +497,7 @@ __global__ void __launch_bounds__(32 * (WPQ > 1 ? WPQ : SMX_WARPS))
         slot = static_cast<long long>(bt[j >> 6]) * 64 + (j & 63);
         sc = dot_row<CT>(qs, k_cache + (static_cast<size_t>(slot) * G + g) * D, D, kvec);
         if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
+        sc -= sl * static_cast<float>(pi - j);
       }
       const float nmx = fmaxf(mx, warp_max_(sc));        // finite: key j0 is always visible
       const float corr = expf(mx - nmx);                 // first pass: exp(-inf) = 0
@@ -407,8 +509,8 @@ __global__ void __launch_bounds__(32 * (WPQ > 1 ? WPQ : SMX_WARPS))
       const int cnt = min(32, jend - j0 + 1);
       for (int jj = 0; jj < cnt; ++jj) {
         const float w = __shfl_sync(0xffffffffu, p, jj);
-        const long long sl = __shfl_sync(0xffffffffu, slot, jj);
-        const CT* vrow = v_cache + static_cast<size_t>(sl) * ldv + g * V;
+        const long long vs = __shfl_sync(0xffffffffu, slot, jj);
+        const CT* vrow = v_cache + static_cast<size_t>(vs) * ldv + gv * V;
 #pragma unroll
         for (int r = 0; r < VR; ++r) {
           const int d = lane + 32 * r;
@@ -1191,7 +1293,10 @@ int launch_ls_join(float* x, const int* q_start, const int* q_len, const int* ro
                    const float* y0, int ld0, const float* w0, int norm0, const float* y1, int ld1, const float* w1,
                    int norm1, const float* y2, int ld2, const float* w2, int norm2, float eps, const float* gamma,
                    int gstride, int plus_one, void* h, int ld_h, int W, int f32, const float* gamma2, void* h2, int ld_h2,
-                   int replace, cudaStream_t s) {
+                   int replace, const float* xin, float* past, const float* dw, size_t dstride, int k,
+                   cudaStream_t s) {
+  if (xin == nullptr) xin = x;
+  const DepthTerm dep{past, dw, dstride, k};
   const bool wide = W > 512;                 // wide rows: the whole block works on one token
   const int tpb = wide ? 1 : LSJ_WARPS;
   dim3 grid;
@@ -1207,7 +1312,7 @@ int launch_ls_join(float* x, const int* q_start, const int* q_len, const int* ro
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool vec = W % 4 == 0 && al16(x) && (y0 == nullptr || (ld0 % 4 == 0 && al16(y0))) &&
                    (y1 == nullptr || (ld1 % 4 == 0 && al16(y1))) && (y2 == nullptr || (ld2 % 4 == 0 && al16(y2))) &&
-                   al16(w0) && al16(w1) && al16(w2) && (h == nullptr || (ld_h % 4 == 0 && al16(h))) &&
+                   al16(w0) && al16(w1) && al16(w2) && al16(xin) && al16(past) && dstride % 4 == 0 && (h == nullptr || (ld_h % 4 == 0 && al16(h))) &&
                    (gstride == 0 || al16(gamma)) && (h2 == nullptr || (ld_h2 % 4 == 0 && al16(h2) && al16(gamma2)));
 #define B2B_LSJ1(OT, VEC, WPT)                                                                                          \
   do {                                                                                                                  \
@@ -1216,7 +1321,7 @@ int launch_ls_join(float* x, const int* q_start, const int* q_len, const int* ro
                            static_cast<int>(smem));                                                                     \
     launch_kernel(ls_join_kernel<OT, VEC, WPT>, grid, dim3(32 * LSJ_WARPS), smem, s, 1u, x, q_start, q_len, rows, n_rows, \
                   a, b, c, eps, gamma, gstride, plus_one, static_cast<OT*>(h), ld_h, W, gamma2, static_cast<OT*>(h2),    \
-                  ld_h2, replace);                                                                                      \
+                  ld_h2, replace, xin, dep);                                                                            \
   } while (0)
 #define B2B_LSJ(OT, VEC)                                                                                                \
   do {                                                                                                                  \
@@ -1259,22 +1364,54 @@ int launch_rot_attn_prep(const float* proj, int ld, int off_q, int off_k, int of
   return last_error();
 }
 
+int launch_talk_prep(const float* proj, int ld, int off_q, int off_k, const float* talk, float scale, const int* slots,
+                     void* q_out, void* k_cache, int T, int H, int G, int D, int q_f32, int f32, cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G != 0 || D <= 0 || (f32 && !q_f32)) return -2;
+  const size_t smem = (static_cast<size_t>((H * D + 3) & ~3) + static_cast<size_t>(H) * ((H + 3) & ~3)) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+  const bool vec = D % 4 == 0 && reinterpret_cast<uintptr_t>(q_out) % 16 == 0;
+  const dim3 block(vec && G * D <= 512 ? 128 : 256);
+#define B2B_TALK(QT, CT, E)                                                                                             \
+  do {                                                                                                                  \
+    if (smem > 48 * 1024)                                                                                               \
+      cudaFuncSetAttribute(talk_prep_kernel<QT, CT, E>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)); \
+    launch_kernel(talk_prep_kernel<QT, CT, E>, dim3(T), block, smem, s, 1u, proj, ld, off_q, off_k, talk, scale, slots,  \
+                  static_cast<QT*>(q_out), static_cast<CT*>(k_cache), H, G, D);                                         \
+  } while (0)
+  if (f32) {
+    if (vec) B2B_TALK(float, float, 4);
+    else B2B_TALK(float, float, 1);
+  } else if (q_f32) {
+    if (vec) B2B_TALK(float, bf16, 4);
+    else B2B_TALK(float, bf16, 1);
+  } else {
+    if (vec) B2B_TALK(bf16, bf16, 4);
+    else B2B_TALK(bf16, bf16, 1);
+  }
+#undef B2B_TALK
+  return last_error();
+}
+
 int launch_softmax_attention(const float* q, const void* k_cache, const void* v_cache, void* out, int ld_out,
                              const int* block_table, int max_pages, const int* q_start, const int* q_len,
                              const int* kv_len, int n_seqs, int max_q, int H, int G, int D, int V, int window,
-                             float scale, int ldv, int f32, float softcap, int keep_first, const float* sink,
-                             cudaStream_t s) {
+                             float scale, int ldv, int f32, float softcap, int keep_first, const float* sink, int Gv,
+                             const float* slope, cudaStream_t s) {
   if (n_seqs <= 0 || max_q <= 0) return 0;
+  if (Gv <= 0) Gv = G;
+  if (Gv > H || H % Gv != 0) return -2;
+  const bool plain = Gv == G && slope == nullptr;      // (the tensor-core variant has neither option)
   if (window <= 0) keep_first = 0;          // every earlier key is visible anyway
   if (V > 64 * SMX_VR || G <= 0 || H % G != 0) return -2;
   const bool wide_v = V > 32 * SMX_VR;      // values of 257 .. 512 channels: 16 channels per lane
-  if (ldv <= 0) ldv = G * V;               // values in a cache of their own; otherwise a view into wider rows
+  if (ldv <= 0) ldv = Gv * V;               // values in a cache of their own; otherwise a view into wider rows
   // short spans and decode steps of grouped heads: the heads that share a key/value head become rows of the tile
   const int hg = (H / G > 1 && max_q < 16 * SMX_MMA_WARPS) ? H / G : 1;
   // (decode steps of 4 or more grouped heads too when sequences x key/value heads fill the machine: a page is staged once
   // per key/value head instead of once per query head -- 32 sequences x 8 key/value heads of 128 channels at 512 keys: 6 %
   // off the decode step; with 2 key/value heads the 64 blocks that walk their pages one by one lose to the 8-warp kernel)
-  if (!f32 && (max_q * hg >= SMX_MMA_MIN_Q || (hg >= 4 && max_q <= SMX_DEC_MAX_Q && n_seqs * G >= 256)) && D % 8 == 0 && V % 8 == 0 && D <= 128 && V <= 128 && ld_out % 2 == 0 &&
+  if (!f32 && plain && (max_q * hg >= SMX_MMA_MIN_Q || (hg >= 4 && max_q <= SMX_DEC_MAX_Q && n_seqs * G >= 256)) && D % 8 == 0 && V % 8 == 0 && D <= 128 && V <= 128 && ld_out % 2 == 0 &&
       ldv % 8 == 0 && reinterpret_cast<uintptr_t>(v_cache) % 16 == 0) {
     dim3 mgrid((max_q * hg + 16 * SMX_MMA_WARPS - 1) / (16 * SMX_MMA_WARPS), hg > 1 ? G : H, n_seqs);
     const int dt = (D + 15) / 16, vt = (V + 15) / 16;
@@ -1294,7 +1431,7 @@ int launch_softmax_attention(const float* q, const void* k_cache, const void* v_
 #define B2B_SMX(CT, WPQ, VR_, GRID, BLOCK, SMEM)                                                                         \
   launch_kernel(softmax_attention_kernel<CT, CT, WPQ, VR_>, dim3(GRID), dim3(BLOCK), SMEM, s, 1u, q,                     \
                 static_cast<const CT*>(k_cache), static_cast<const CT*>(v_cache), static_cast<CT*>(out), ld_out,        \
-                block_table, max_pages, q_start, q_len, kv_len, H, G, D, V, window, scale, ldv, softcap, keep_first, sink)
+                block_table, max_pages, q_start, q_len, kv_len, H, G, D, V, window, scale, ldv, softcap, keep_first, sink, Gv, slope)
 #define B2B_SMX_T(WPQ, GRID, BLOCK, SMEM)                                                                               \
   if (f32) {                                                                                                            \
     if (wide_v) B2B_SMX(float, WPQ, 2 * SMX_VR, GRID, BLOCK, SMEM);                                                     \
