@@ -803,9 +803,15 @@ class HybridPiece:
         H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
         assert sp.qk_norm == "none" and sp.keys_as_values and sp.rot is None and not sp.softcap and not sp.keep_first
         kc, vc = self.k_cache[self._key(mx)], self.v_cache[self._key(mx)]
-        q = self._buf(f"q{mx.idx}", torch.float32, H * G * D)[:T]
+        fast = self.dtype == torch.bfloat16 and ops.mixed_attention_supported(H, G, D)
+        qb = self._buf(f"q{mx.idx}", torch.bfloat16 if fast else torch.float32, H * G * D)
+        q = qb[:T]
         ops.talk_prep(proj, mx.off["q"], mx.off["k"], mx.f["talk"], sp.scale, m.slots, q, kc, T, H, G, D)
         ao = self._buf(f"mix{mx.idx}.{H * V}", self.dtype, mx.w_o.shape[1])[:T]
+        if fast:
+            ops.mixed_attention(qb, kc, ao, m.block_table, m.q_start, m.q_len, m.kv_len, m.n_seqs, m.max_q, H, G, D, sp.window,
+                                slopes=mx.f.get("slopes"), sink=mx.f.get("sink"))
+            return ops.linear(mx.w_o, ao, y, bias=mx.b_o)
         ops.softmax_attention(q, kc.view(kc.shape[0], kc.shape[1], 1, G * D), vc, ao, m.block_table, m.q_start, m.q_len, m.kv_len,
                               m.n_seqs, m.max_q, H, 1, G * D, V, sp.window, 1.0, sink=mx.f.get("sink"), v_heads=G,
                               slopes=mx.f.get("slopes"))

@@ -35,7 +35,7 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "set_decode_state", "hyb_embed", "hyb_commit_prev", "hc_step", "act_cols", "attn_prep",
                         "sig_attention", "delta_scan", "delta_post", "ls_join", "rot_attn_prep", "softmax_attention",
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
-                        "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm")
+                        "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention")
 
 
 class _CountedModule:
@@ -634,6 +634,17 @@ def talk_prep(proj, off_q, off_k, talk, scale, slots, q_out, k_cache, T, H, G, D
     cache row, ``q_out[t, h, c] = scale * sum over the heads g that read key head c of talk[h, g] q[t, g]`` ([T, H * G * D],
     float or bf16), and the key rows (``proj`` columns ``off_k`` ..) into the paged cache."""
     native().talk_prep(proj, off_q, off_k, talk, float(scale), slots, q_out, k_cache, T, H, G, D)
+
+
+def mixed_attention_supported(H, G, D):
+    """whether ``mixed_attention`` has a kernel for ``H`` heads over ``G`` key heads of ``D`` channels (else: ``softmax_attention``)"""
+    return bool(native().mixed_attention_supported(int(H), int(G), int(G) * int(D), int(D)))
+
+
+def mixed_attention(q, k_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, window, slopes=None, sink=None):
+    """softmax attention with mixed heads behind ``talk_prep`` (bf16 query rows [rows, H * G * D], bf16 cache whose key rows are
+    the values): spans on tcgen05, single tokens on a cluster of CTAs per query; options as in ``softmax_attention``"""
+    native().mixed_attention(q, k_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, window, slopes, sink)
 
 
 def poly_norm(x, off, w, out, n, eps, T):

@@ -2,7 +2,8 @@
 next to the closest uniform decoder (Llama), or (``--family repudra``) the parallel-block Repudra graph next to the
 closest hybrid (Kepovik), or (``--family lonulix``) the post-norm Lonulix graph next to Repudra (the other family whose
 attention and recurrences run on the kernels of ``csrc/seqmix.cu``), or (``--family fisopel``) the looped Fisopel graph next
-to Lonulix (the other family with latent attention and routed experts); random weights, layer shapes of real models.
+to Lonulix (the other family with latent attention and routed experts), or (``--family kazolorn``) the depth-averaged Kazolorn
+graph next to Fisopel (the other family of parallel blocks with two norms, windowed attention and gated experts); random weights, layer shapes of real models.
 
 Per width it reports (1) prefill and decode tokens/s through the same ``GpuRunner`` calls that serving uses (chunked
 graph prefill, CUDA-graph decode steps), timed with CUDA events, and (2) a per-kernel breakdown of one eager prefill
@@ -134,6 +135,32 @@ def fisopel_sized(width: int, vocab: int = 32000) -> ModelConfig:
                        block_layout="parallel", ff_norm=True, loop_start=1, loop_stop=3, loop_times=2, loop_in=True)
 
 
+def kazolorn_sized(width: int, vocab: int = 32000) -> ModelConfig:
+    """six parallel-block layers with depth averages: attention (width / 128 heads of 128 channels, grouped 4:1, keys as values,
+    distance bias, mixed heads, window 1024) in every layer, beside a PolyNorm feed-forward of 29 width / 8 hidden channels
+    or 8 gated experts of width / 4 (2 per token), alternating.  The layer matrices hold about 53 width^2 parameters, as
+    ``fisopel_sized(width)`` does."""
+    H = width // 128
+
+    def att(ff=0):
+        sp = LayerSpec(mixer="softmax_attention", heads=H, kv_heads=max(1, H // 4), dim=128, vdim=128, scale=128 ** -0.5,
+                       window=1024, qk_norm="none", v_norm=False, keys_as_values=True, proj_bias=True, distance_bias=True,
+                       talk=True, sink_one=True)
+        if ff:
+            sp.ff, sp.ff_act = ff, "poly_norm"
+        else:
+            sp.ff_kind, sp.experts, sp.expert_ff, sp.top, sp.ff = "moe", 8, width // 4, 2, 2 * width
+            sp.route_kind, sp.expert_gated, sp.scale_input = "sigmoid_topk", True, True
+        return sp
+
+    specs = tuple(att(0 if l % 2 else 29 * width // 8) for l in range(6))
+    return ModelConfig(name=f"mini-kazolorn-{width}", family="kazolorn", vocab_size=vocab, hidden_size=width,
+                       n_layers=len(specs), n_heads=H, n_kv_heads=max(1, H // 4), head_dim=128,
+                       ffn_size=max(sp.ff for sp in specs), max_position=1 << 30, norm="rms", norm_eps=1e-5, act="silu",
+                       glu=True, rope_theta=0.0, layer_specs=specs, block_layout="parallel", ff_norm=True, layer_scale=True,
+                       depth_average=True)
+
+
 def llama_sized(width: int, layer_params: int, n_layers: int = 4, vocab: int = 32000) -> ModelConfig:
     """Llama layers (GQA 4:1, SwiGLU) whose matrices hold about ``layer_params`` parameters in ``n_layers`` layers"""
     H = width // 128
@@ -205,6 +232,15 @@ def _nb(t) -> int:
     return t.numel() * t.element_size()
 
 
+def visible_keys(hint: Dict, window: int, keep_first: int):
+    """((query, key) pairs a windowed causal attention evaluates, keys it has to read per sequence)"""
+    S, q, ctx = hint["S"], hint["q"], hint["ctx"]
+    if window <= 0:
+        return S * (q * ctx + q * (q + 1) / 2), ctx + q
+    per = sum(min(ctx + i + 1, window + max(0, min(keep_first, ctx + i + 1 - window))) for i in range(q))
+    return S * float(per), min(ctx + q, window + q - 1 + keep_first)
+
+
 def cost(name: str, a, hint: Dict):
     """(algorithmic FLOPs, bytes, runs on tensor cores) of one kernel call; ``hint``: tokens T, sequences S, span q,
     context ctx (keys before the span), and for attention the visible keys per query."""
@@ -253,16 +289,28 @@ def cost(name: str, a, hint: Dict):
         W = a[0].shape[-1]
         rows = a[4] if a[3] is not None else T
         n_terms = sum(1 for i in (7, 10, 13) if a[i] is not None)
-        return 0.0, rows * W * 4 * ((1 if a[3] is not None else 2) + n_terms) + (rows * W * a[19].element_size()
-                                                                                   if a[19] is not None else 0), False
+        depth = 0
+        if a[23] is not None:                   # depth average: k kept rows are read and the joined one is written
+            depth = a[25] + (1 if a[3] is None else 0)
+        ops_out = sum(rows * W * t.element_size() for t in (a[19], a[21]) if t is not None)
+        return 0.0, rows * W * 4 * ((1 if a[3] is not None else 2) + n_terms + depth) + ops_out, False
     if name == "rot_attn_prep":
         H, G, D, V = a[15], a[16], a[17], a[18]
         return 0.0, T * ((H + G) * D + G * V) * 4 + T * H * D * 4 + T * G * (D + V) * a[12].element_size(), False
     if name == "softmax_attention":
         H, G, D, V = a[10], a[11], a[12], a[13]
-        keys = S * (q * ctx + q * (q + 1) / 2)                       # causal
-        kv_bytes = S * (ctx + q) * G * (D + V) * a[1].element_size()
+        keys, span = visible_keys(hint, a[14], a[17])
+        kv_bytes = S * span * (G * D + (0 if a[1].data_ptr() <= a[2].data_ptr() < a[1].data_ptr() + _nb(a[1]) else G * V)) * a[1].element_size()
         return 2.0 * H * (D + V) * keys, kv_bytes + T * H * D * 4 + T * H * V * a[3].element_size(), q >= 16
+    if name == "mixed_attention":               # products and mix of the plain form: q.k per head, H x H mix, p.v per head
+        H, G, D = a[9], a[10], a[11]
+        keys, span = visible_keys(hint, a[12], 0)
+        return 2.0 * H * (2 * D + H) * keys, S * span * G * D * 2 + T * H * D * 4 + T * H * D * 2, q >= 16
+    if name == "talk_prep":
+        H, G, D = a[9], a[10], a[11]
+        return 0.0, T * (H + G) * D * 4 + T * H * G * D * a[6].element_size() + T * G * D * a[7].element_size(), False
+    if name == "poly_norm":
+        return 0.0, T * a[4] * (4 + a[3].element_size()), False
     if name == "short_conv":
         return 0.0, 2 * T * a[2].shape[0] * 4, False
     if name == "mlstm_gates":
@@ -422,7 +470,9 @@ def run(widths, prompt_len=2048, batch=32, steps=32, warmup=3, ctx=512, device="
     out = []
     for w in widths:
         kep = kepovik_sized(w)
-        if family == "fisopel":
+        if family == "kazolorn":
+            pair = (kazolorn_sized(w), fisopel_sized(w))
+        elif family == "fisopel":
             pair = (fisopel_sized(w), lonulix_sized(w))
         elif family == "lonulix":
             pair = (lonulix_sized(w), repudra_sized(w))

@@ -142,6 +142,7 @@ void set_wait_policy(int64_t abort_word, double limit_ms) {
   const auto ns = static_cast<unsigned long long>(limit_ms * 1e6);
   check(b2b::set_wait_policy_gemm(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(gemm)");
   check(b2b::set_wait_policy_elementwise(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(elementwise)");
+  check(b2b::set_wait_policy_mixed(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(mixed)");
 }
 
 void set_pdl(bool on) { b2b::g_pdl_mode = on ? 1 : 0; }
@@ -607,6 +608,28 @@ void softmax_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
         "softmax_attention");
 }
 
+// q [rows, H * GD] bf16 (talk_prep), k_cache [pages, 64, G, D] bf16 with GD = G * D channels per token, out [T, >= H * V] bf16
+void mixed_attention(const Tensor& q, const Tensor& k_cache, const Tensor& out, const Tensor& block_table,
+                     const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int64_t n_seqs, int64_t max_q, int64_t H,
+                     int64_t Gv, int64_t V, int64_t window, const OptT& slopes, const OptT& sink) {
+  c10::cuda::CUDAGuard guard(q.device());
+  check_bf16(q, "q");
+  check_bf16(k_cache, "k_cache");
+  check_bf16(out, "out");
+  const int64_t GD = k_cache.size(2) * k_cache.size(3);
+  TORCH_CHECK(k_cache.is_contiguous() && k_cache.size(1) == 64 && q.stride(0) == H * GD && q.stride(1) == 1 &&
+                  GD == Gv * V && out.size(1) >= H * V, "mixed_attention: sizes");
+  TORCH_CHECK(!(sink.has_value() && sink->defined()) || sink->numel() >= H, "mixed_attention: one sink per head");
+  TORCH_CHECK(!(slopes.has_value() && slopes->defined()) || slopes->numel() >= H, "mixed_attention: one slope per head");
+  check(b2b::launch_mixed_attention(q.data_ptr(), static_cast<int>(q.size(0)), k_cache.data_ptr(),
+                                    static_cast<int>(k_cache.size(0)), out.data_ptr(), static_cast<int>(out.stride(0)),
+                                    ip(block_table), static_cast<int>(block_table.stride(0)), ip(q_start), ip(q_len),
+                                    ip(kv_len), static_cast<int>(n_seqs), static_cast<int>(max_q), static_cast<int>(H),
+                                    static_cast<int>(Gv), static_cast<int>(GD), static_cast<int>(V),
+                                    static_cast<int>(window), fp_or_null(slopes), fp_or_null(sink), cur_stream()),
+        "mixed_attention");
+}
+
 // proj [T, >= ...] fp32: q (H * D columns at off_q), k (G * D at off_k); q_out [T, H * G * D] float or bf16; cache rows [G, D]
 void talk_prep(const Tensor& proj, int64_t off_q, int64_t off_k, const Tensor& talk, double scale, const Tensor& slots,
                const Tensor& q_out, const Tensor& k_cache, int64_t T, int64_t H, int64_t G, int64_t D) {
@@ -826,6 +849,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rot_attn_prep", &rot_attn_prep);
   m.def("softmax_attention", &softmax_attention);
   m.def("talk_prep", &talk_prep);
+  m.def("mixed_attention", &mixed_attention);
+  m.def("mixed_attention_supported", &b2b::mixed_attention_supported);
+  m.def("mixed_attention_gave_up", &b2b::mixed_attention_gave_up);
   m.def("short_conv", &short_conv);
   m.def("mlstm_gates", &mlstm_gates);
   m.def("lin_scan", &lin_scan);

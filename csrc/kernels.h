@@ -98,6 +98,14 @@ int launch_ls_join(float* x, const int* q_start, const int* q_len, const int* ro
                    int replace, const float* xin, float* past, const float* dw, size_t dstride, int k,
                    cudaStream_t s);
 // mixed heads (score_h <- sum_g talk[h, g] score_g) as one query row per head over the whole key row; keys into the cache
+//   (mixed_attention.cu: the attention behind it for bf16 caches, q [rows, H * GD] bf16, values = channels of the key rows;
+//   mixed_attention_gave_up: CTAs whose bounded waits ran out so far, 0 unless there is a bug)
+bool mixed_attention_supported(int H, int Gv, int GD, int V);
+unsigned mixed_attention_gave_up();
+int launch_mixed_attention(const void* q, int q_rows, const void* k_cache, int n_pages, void* out, int ld_out,
+                           const int* block_table, int max_pages, const int* q_start, const int* q_len, const int* kv_len,
+                           int n_seqs, int max_q, int H, int Gv, int GD, int V, int window, const float* slope,
+                           const float* sink, cudaStream_t s);
 int launch_talk_prep(const float* proj, int ld, int off_q, int off_k, const float* talk, float scale, const int* slots,
                      void* q_out, void* k_cache, int T, int H, int G, int D, int q_f32, int f32, cudaStream_t s);
 int launch_rot_attn_prep(const float* proj, int ld, int off_q, int off_k, int off_v, const float* qn, const float* kn,
@@ -156,6 +164,7 @@ int launch_head_up_gate(const void* a, int ld_a, const void* U, const float* gat
 
 // bounded handoff waits: device abort word + time limit for the waits of each translation unit (0 / null = trap policy)
 int set_wait_policy_gemm(uint32_t* abort_word, unsigned long long limit_ns);
+int set_wait_policy_mixed(uint32_t* abort_word, unsigned long long limit_ns);
 int set_wait_policy_elementwise(uint32_t* abort_word, unsigned long long limit_ns);
 
 // gemm_tc.cu

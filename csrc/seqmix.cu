@@ -352,10 +352,9 @@ __global__ void __launch_bounds__(256)
   float* tt = tp + ((nq + 3) & ~3);                   // [H (mixed from)][Hp (mixed into)]
   const float* row = proj + static_cast<size_t>(t) * ld;
   for (int i = threadIdx.x; i < nq; i += blockDim.x) qs[i] = row[off_q + i] * scale;
-  for (int i = threadIdx.x; i < H * Hp; i += blockDim.x) {
-    const int g = i / Hp, h = i % Hp;
-    tt[i] = h < H ? talk[h * H + g] : 0.f;
-  }
+  for (int i = threadIdx.x; i < H * H; i += blockDim.x) tt[i % H * Hp + i / H] = talk[i];
+  if (Hp != H)
+    for (int i = threadIdx.x; i < H * (Hp - H); i += blockDim.x) tt[i / (Hp - H) * Hp + H + i % (Hp - H)] = 0.f;
   for (int i = threadIdx.x; i < nk; i += blockDim.x) stf(k_cache, static_cast<size_t>(slot) * nk + i, row[off_k + i]);
   __syncthreads();
   QT* qo = q_out + static_cast<size_t>(t) * H * nk;

@@ -1,0 +1,810 @@
+"""Kazolorn (parallel blocks with a norm each and layer scale, averaged over depth; windowed attention whose values are the
+cached keys, with a distance bias, scores mixed across the heads and a one in the denominator; PolyNorm or sigmoid-chosen
+gated experts with scaled input) against the plain oracle in ``kazolorn_oracle.py``.  Every test builds its own small
+configuration and random checkpoint on disk, so the config reader, the loader, the page allocator, the batch slots and the
+chunk path of the runner are all on the tested path.  The GPU tests run the float32 mode at tight tolerance and the bf16
+serving mode at rounding tolerance.
+"""
+from __future__ import annotations
+
+import json
+import math
+import os
+
+import numpy as np
+import pytest
+import torch
+
+import kazolorn_oracle as O
+
+from bee2bee_b200.models.config import ModelConfig, resolve_config
+
+gpu = pytest.mark.gpu
+
+
+# ----------------------------------------------------------------------------------------------- model builders
+def dense(ff=40):
+    return {"ff": ff, "kind": "dense"}
+
+
+def moe(experts=5, ff=24, top=2):
+    return {"expert": {"ff": ff}, "kind": "moe", "router": {"experts": experts, "top": top}}
+
+
+def att(heads=4, kv=2, dim=16, window=30, scale=None, mlp=None):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"dim": dim, "heads": heads, "kv_heads": kv, "mask": {"size": window},
+                      "scale": scale if scale is not None else dim ** -0.5, "vdim": dim}}
+
+
+def make_cfg(layers, width=64, vocab=200, eps=1e-5):
+    return {"architecture": "Kazolorn", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def make_tensors(cfg, seed=0, tweak=None):
+    """random checkpoint (values exactly representable in bf16, kept as float32)"""
+    g = torch.Generator().manual_seed(seed)
+    W, t = cfg["width"], {}
+
+    def rn(*shape, std=1.0, mean=0.0):
+        return (torch.randn(*shape, generator=g) * std + mean).bfloat16().float()
+
+    def lin(n_out, n_in, gain=1.0):
+        return rn(n_out, n_in, std=gain * n_in ** -0.5)
+
+    t["embed"], t["head"] = rn(cfg["vocab"], W), lin(cfg["vocab"], W)
+    for i, lay in enumerate(cfg["layers"]):
+        p, m, q = f"l{i}.", lay["mixer"], f"l{i}.mix."
+        H, G, D = m["heads"], m["kv_heads"], m["dim"]
+        t[p + "norm1"] = rn(W, std=0.1, mean=1.0)
+        t[q + "q"], t[q + "q.b"] = lin(H * D, W, 1.5), rn(H * D, std=0.5)
+        t[q + "k"], t[q + "k.b"] = lin(G * D, W, 1.5), rn(G * D, std=0.5)
+        t[q + "talk"] = (torch.eye(H) + torch.randn(H, H, generator=g) * 0.6 * H ** -0.5).bfloat16().float()
+        t[q + "o"], t[q + "o.b"] = lin(W, H * D, 1.5), rn(W, std=0.3)
+        t[p + "ls1"] = rn(W, std=0.2, mean=0.7)
+        mlp = lay["mlp"]
+        if mlp:
+            t[p + "norm2"], t[p + "ls2"] = rn(W, std=0.1, mean=1.0), rn(W, std=0.2, mean=0.7)
+            if mlp["kind"] == "dense":
+                t[p + "mlp.up"], t[p + "mlp.down"] = lin(mlp["ff"], W, 1.5), lin(W, mlp["ff"])
+                t[p + "mlp.act"] = rn(4, std=0.4, mean=0.5)
+            else:
+                f = mlp["expert"]["ff"]
+                for e in range(mlp["router"]["experts"]):
+                    n = f"{p}mlp.e{e}."
+                    t[n + "gate"], t[n + "up"], t[n + "down"] = lin(f, W, 1.5), lin(f, W, 1.5), lin(W, f, 1.5)
+                t[p + "mlp.router"] = lin(mlp["router"]["experts"], W, 3.0)
+        t[p + "dwa"] = torch.cat([torch.randn(i + 1, generator=g) * 0.3, torch.randn(1, generator=g) * 0.1 + 0.9]).bfloat16().float()
+    t["final.norm"] = rn(W, std=0.1, mean=1.0)
+    if tweak:
+        tweak(t)
+    return t
+
+
+def save_model(path, cfg, t):
+    from safetensors.torch import save_file
+
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    save_file({k: v.bfloat16().contiguous() for k, v in t.items()}, os.path.join(path, "model.safetensors"))
+    return str(path)
+
+
+def oracle_logits(tokens, t, cfg):
+    with torch.no_grad():
+        return O.forward(cfg, t, list(tokens))[0].float().numpy()
+
+
+def rel_err(got, want):
+    """per-row error: difference with its mean removed, as a root mean square relative to the spread of the logits"""
+    d = got - want
+    d = d - d.mean(-1, keepdims=True)
+    return np.sqrt((d ** 2).mean(-1)) / want.std()
+
+
+TOL = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
+
+
+def routed(cfg):
+    return any(lay["mlp"] and lay["mlp"]["kind"] == "moe" for lay in cfg["layers"])
+
+
+def assert_close(got, want, dtype, cfg, tol=None, what=""):
+    """Every row within the tolerance of its number format -- except bf16 with routed experts: rounding turns the near tie of
+    a router the other way now and then, which moves that token's row (and, through the caches, later rows a little) by far
+    more than rounding does elsewhere.  Those runs are judged as a population; the same schedules run strictly in float32
+    and, in bf16, on a model without a router."""
+    err = rel_err(got, want)
+    tol = tol if tol is not None else TOL[dtype]
+    if dtype == torch.float32 or not routed(cfg):
+        assert err.max() < tol, (what, float(err.max()))
+    else:
+        assert np.median(err) < tol / 3 and (err > tol).mean() <= 0.25 and err.max() < 0.7, \
+            (what, float(err.max()), float(np.median(err)), float((err > tol).mean()))
+
+
+def engine(path, dtype, max_tokens=512, slots=4, chunk_tokens=256):
+    from bee2bee_b200.engine.core import Engine
+
+    return Engine(path, device="cuda:0", max_batch=slots, max_seq_len=max_tokens, max_prefill_tokens=chunk_tokens,
+                  num_pages=max_tokens // 64 + 1, dtype=dtype, max_logit_rows=chunk_tokens, prefix_cache=False)
+
+
+def replay(eng, key, tokens, cuts, end=True):
+    """feed ``tokens`` in portions ``cuts`` (then single tokens), asking for every position -> [T, V]"""
+    out, pos, k = [], 0, 0
+    while pos < len(tokens):
+        n = min(cuts[k] if k < len(cuts) else 1, len(tokens) - pos)
+        k += 1
+        last = pos + n == len(tokens)
+        out.append(eng.replay_step([(key, tokens[pos:pos + n], list(range(n)))], [key] if (last and end) else []))
+        pos += n
+    return np.concatenate(out)
+
+
+def toks(n, vocab, seed):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+# ------------------------------------------------------------------------------------------------- CPU tests
+def test_config_reader_roundtrip_and_registry():
+    d = make_cfg([att(heads=6, kv=3, dim=24, window=9, scale=0.3, mlp=dense(56)), att(mlp=moe(experts=6, top=3)), att(kv=4),
+                  att(heads=2, kv=1, window=1, mlp=moe(top=1))], eps=1e-4)
+    c = ModelConfig.from_hf_dict(d, "x")
+    assert c.family == "kazolorn" and c.hybrid and not c.recurrent and c.n_layers == 4 and not c.tie_embeddings
+    assert c.block_layout == "parallel" and c.ff_norm and c.layer_scale and c.depth_average and not c.scalar_norm
+    assert c.norm_eps == 1e-4 and c.embed_scale == 1.0 and c.final_softcap == 0.0
+    a, b, e = c.layer_specs[:3]
+    assert (a.mixer, a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.scale) == ("softmax_attention", 6, 3, 24, 24, 9, 0.3)
+    assert a.keys_as_values and a.proj_bias and a.distance_bias and a.talk and a.sink_one and not a.sink and a.qk_norm == "none"
+    assert a.ff == 56 and a.ff_act == "poly_norm" and a.ff_kind == "dense"
+    assert (b.ff_kind, b.experts, b.expert_ff, b.top, b.shared_ff, b.route_kind, b.expert_gated, b.scale_input) == \
+        ("moe", 6, 24, 3, 0, "sigmoid_topk", True, True) and b.ff == 6 * 24
+    assert e.ff == 0 and e.kv_heads == 4
+    assert np.allclose(a.head_slopes, O.head_slopes(6)) and a.head_slopes[5] == 2.0 ** -8
+    assert ModelConfig.from_hf_dict(c.to_hf_dict(), "x") == c
+    from bee2bee_b200.models import piece_class
+    from bee2bee_b200.models.hybrid import HybridPiece
+    assert piece_class(c) is HybridPiece
+    wide = att()
+    wide["mixer"]["vdim"] = 8
+    for bad in (make_cfg([{"type": "nope", "mixer": {"heads": 1, "dim": 8}, "mlp": None}]), make_cfg([att(heads=3, kv=2)]),
+                make_cfg([att(mlp=moe(experts=2, top=3))]), make_cfg([att(mlp={"kind": "odd"})]), make_cfg([wide])):
+        with pytest.raises(ValueError):
+            ModelConfig.from_hf_dict(bad, "x")
+
+
+def test_checkpoint_loader_names_and_shapes(tmp_path):
+    from bee2bee_b200.models.weights import hybrid_tensor_specs, init_random, load_or_init
+
+    d = make_cfg([att(mlp=dense()), att(heads=3, kv=3, mlp=moe()), att()], width=48)
+    t = make_tensors(d)
+    path = save_model(tmp_path / "m", d, t)
+    c = resolve_config(path)
+    got = load_or_init(path, c, range(3), True, True)
+    assert set(got) == set(t)
+    for k in t:
+        assert torch.equal(got[k], t[k]), k
+    assert got["l1.mix.talk"].shape == (3, 3) and got["l2.dwa"].shape == (4,) and got["l0.mlp.act"].shape == (4,)
+    assert "l2.norm2" not in got and "l2.ls2" not in got and got["l1.mlp.router"].shape == (5, 48)
+    preset = resolve_config("tiny-kazolorn")
+    rnd = init_random(preset, range(preset.n_layers), True, True)
+    specs = hybrid_tensor_specs(preset, range(preset.n_layers), True, True)
+    assert {n for n, _, _ in specs} == set(rnd) and all(tuple(rnd[n].shape) == tuple(s) for n, s, _ in specs)
+    assert ModelConfig.from_hf_dict(preset.to_hf_dict(), "tiny-kazolorn") == preset
+
+
+def test_oracle_mechanisms_by_hand():
+    f64 = torch.float64
+    assert O.in_window(4, 2).tolist() == [[True, False, False, False], [True, True, False, False], [False, True, True, False],
+                                          [False, False, True, True]]
+    assert O.in_window(3, 0).tolist() == torch.ones(3, 3).tril().bool().tolist()
+    # one visible key of score s: e^s / (1 + e^s); a very negative score leaves nothing, a very large one everything
+    p = O.softmax_plus_one(torch.tensor([[1.0, 9.0], [-800.0, 0.0], [800.0, 0.0]], dtype=f64),
+                           torch.tensor([[True, False], [True, False], [True, False]]))
+    assert np.allclose(p.numpy(), [[math.e / (1 + math.e), 0.0], [0.0, 0.0], [1.0, 0.0]])
+    assert O.head_slopes(2) == [2.0 ** -4, 2.0 ** -8]
+    # two heads, one key head, distance 1: the products minus the slopes; then head 0 takes 2 s_0 - s_1
+    q = torch.tensor([[[0.0], [0.0]], [[1.0], [3.0]]], dtype=f64)
+    s = O.biased_scores(q, torch.tensor([[[5.0]], [[7.0]]], dtype=f64), 0.5)
+    assert np.allclose(s[:, 1, 0].numpy(), [2.5 - 2.0 ** -4, 7.5 - 2.0 ** -8])
+    mixed = O.mix_heads(s, torch.tensor([[2.0, -1.0], [0.0, 1.0]], dtype=f64))
+    assert np.allclose(mixed[:, 1, 0].numpy(), [2 * (2.5 - 2.0 ** -4) - (7.5 - 2.0 ** -8), 7.5 - 2.0 ** -8])
+    # PolyNorm of (1, -2): roots of the mean second, fourth and sixth powers
+    y = O.poly_norm(torch.tensor([[1.0, -2.0]], dtype=f64), torch.tensor([1.0, 10.0, 100.0, 0.5], dtype=f64), 0.0)
+    r2, r4, r6 = 2.5 ** 0.5, 8.5 ** 0.5, 32.5 ** 0.5
+    assert np.allclose(y.numpy(), [[1 / r2 + 10 / r4 + 100 / r6 + 0.5, -2 / r2 + 40 / r4 - 800 / r6 + 0.5]])
+    idx, w = O.choose(torch.tensor([[0.0, 2.0, -1.0, 1.0]], dtype=f64), 2)
+    assert idx == [[1, 3]] and np.allclose(w[0], [1 / (1 + math.exp(-2)), 1 / (1 + math.exp(-1))])
+    # the weight scales the input: down(silu(w g) * w u), not w down(silu(g) * u)
+    P = {"e0.gate": torch.tensor([[2.0]], dtype=f64), "e0.up": torch.tensor([[3.0]], dtype=f64),
+         "e0.down": torch.tensor([[1.0]], dtype=f64), "router": torch.tensor([[0.5]], dtype=f64)}
+    y = O.routed_ff(torch.tensor([[1.0]], dtype=f64), P, "", 1)
+    w = 1 / (1 + math.exp(-0.5))
+    assert np.allclose(y.numpy(), (2 * w) / (1 + math.exp(-2 * w)) * 3 * w)
+    assert O.depth_average([torch.tensor([1.0], dtype=f64), torch.tensor([10.0], dtype=f64)], torch.tensor([3.0, 0.5])).tolist() == [8.0]
+
+
+def test_cpu_engine_refuses_hybrid_models():
+    from bee2bee_b200.engine.core import Engine
+
+    with pytest.raises(ValueError):
+        Engine("tiny-kazolorn", device="cpu")
+
+
+# ------------------------------------------------------------------------------------------- kernels alone (GPU)
+@gpu
+@pytest.mark.parametrize("W,k", [(64, 1), (70, 3), (192, 2), (1040, 5), (2304, 7)])
+def test_join_kernel_depth_average(W, k):
+    """the joined row is kept as entry k, the residual becomes the weighted sum of the entries 0 .. k, both norms read that;
+    logit rows (gathered) see the same average without writing anything"""
+    from bee2bee_b200 import ops
+
+    dev, eps = "cuda", 1e-5
+    g = torch.Generator().manual_seed(W)
+    q_len = [5, 0, 3]
+    T, cap = sum(q_len), 11
+    ld = (W + 63) // 64 * 64 + 64
+    x, y0, y1 = torch.randn(T, W, generator=g), torch.randn(T, ld, generator=g), torch.randn(T, ld, generator=g)
+    past = torch.randn(k + 2, cap, W, generator=g)
+    w0, w1, g1, g2 = (torch.randn(W, generator=g) for _ in range(4))
+    wts = torch.randn(k + 1, generator=g)
+    qs = torch.tensor([0, 5, 5], dtype=torch.int32, device=dev)
+    ql = torch.tensor(q_len, dtype=torch.int32, device=dev)
+    for own in (True, False):                  # the entering row is x itself, or (first layer) entry 0
+        entry = x if own else past[0, :T]
+        new = entry.double() + y0[:, :W].double() * w0.double() + y1[:, :W].double() * w1.double()
+        avg = O.depth_average([past[j, :T].double() for j in range(k)] + [new], wts.double())
+        n = O.rms(avg, eps)
+        for odt, tol in ((torch.float32, 5e-5), (torch.bfloat16, 3e-2)):
+            xd, pd = x.to(dev).contiguous(), past.to(dev).contiguous()
+            h1, h2 = torch.zeros(T, ld, device=dev, dtype=odt), torch.zeros(T, ld, device=dev, dtype=odt)
+            kw = dict(terms=[(y0.to(dev), w0.to(dev), False), (y1.to(dev), w1.to(dev), False)], eps=eps,
+                      depth=(pd, wts.to(dev), k, xd if own else pd[0, :T]))
+            rows = torch.tensor([6, 0, 3], dtype=torch.int32, device=dev)
+            hr = torch.zeros(3, ld, device=dev, dtype=odt)
+            ops.ls_join(xd, qs, ql, 3, 5, gamma=g1.to(dev), h=hr, rows=rows, n_rows=3, **kw)
+            assert torch.equal(xd.cpu(), x) and torch.equal(pd.cpu(), past)
+            assert torch.allclose(hr[:, :W].float().cpu().double(), (n * g1.double())[[6, 0, 3]], atol=tol, rtol=1e-2)
+            ops.ls_join(xd, qs, ql, 3, 5, gamma=g1.to(dev), h=h1, gamma2=g2.to(dev), h2=h2, **kw)
+            assert torch.allclose(pd[k, :T].cpu().double(), new, atol=2e-5)
+            assert torch.allclose(xd.cpu().double(), avg, atol=5e-5)
+            assert torch.allclose(h1[:, :W].float().cpu().double(), n * g1.double(), atol=tol, rtol=1e-2)
+            assert torch.allclose(h2[:, :W].float().cpu().double(), n * g2.double(), atol=tol, rtol=1e-2)
+            keep = [j for j in range(k + 2) if j != k]
+            assert torch.equal(pd[keep].cpu(), past[keep]) and torch.equal(pd[k, T:].cpu(), past[k, T:])
+
+
+def _paged(rows, page_ids, dtype):
+    """rows [n, G, D] of one sequence -> cache [pages, 64, G, D] with the sequence's pages at ``page_ids``"""
+    cache = torch.full((max(page_ids) + 2, 64) + tuple(rows.shape[1:]), 3.0)      # other pages hold junk, not zeros
+    for j in range(rows.shape[0]):
+        cache[page_ids[j // 64], j % 64] = rows[j]
+    return cache.to("cuda", dtype)
+
+
+def mixed_reference(q, k, talk, scale, slopes, window, sink):
+    """the plain order: every head's biased scores, then the mix, then the softmax (float64) -> [T, H, D]"""
+    H, G = q.shape[1], k.shape[1]
+    n = k.shape[0]
+    dist = (torch.arange(n)[:, None] - torch.arange(n)[None, :]).double()
+    s = torch.stack([(q[:, h].double() @ k[:, h // (H // G)].double().T) * scale - slopes[h] * dist for h in range(H)])
+    s = O.mix_heads(s, talk.double())
+    ok = O.in_window(n, window)
+    s = s.masked_fill(~ok, -float("inf"))
+    top = s.max(-1, keepdim=True).values
+    if sink is not None:
+        top = torch.maximum(top, sink.double().view(H, 1, 1))
+    e = torch.exp(s - top)
+    den = e.sum(-1, keepdim=True) + (torch.exp(sink.double().view(H, 1, 1) - top) if sink is not None else 0.0)
+    p = e / den
+    return torch.stack([p[h] @ k[:, h // (H // G)].double() for h in range(H)], 1)
+
+
+SHAPES = [(4, 2, 16), (8, 2, 40), (6, 3, 24), (3, 3, 8), (4, 1, 64), (2, 1, 120), (12, 4, 32), (16, 4, 128), (5, 5, 56), (40, 8, 16),
+          (32, 8, 128), (9, 3, 88), (8, 8, 72), (1, 1, 128), (4, 2, 20), (2, 2, 7)]
+
+
+@gpu
+@pytest.mark.parametrize("H,G,D", SHAPES)
+@pytest.mark.parametrize("nq,window", [(300, 0), (300, 70), (300, 129), (2, 1), (1, 0), (1, 65), (7, 33), (129, 128), (2, 190)])
+def test_mixed_heads_attention_kernels(H, G, D, nq, window):
+    """prep (mixed query rows, keys into the cache) + attention for the last ``nq`` of 300 positions on scattered pages, beside
+    an idle sequence and a sequence of its own length: bf16 on the tensor-core kernels (where the sizes allow), float32 on the
+    exact kernel.  Random mixing matrices with entries of both signs."""
+    from bee2bee_b200 import ops
+
+    n, n2, dev = 300, 45, "cuda"
+    g = torch.Generator().manual_seed(H * 100 + D + nq)
+    scale = 1.3 * D ** -0.5
+    talk = torch.eye(H) + torch.randn(H, H, generator=g) * 0.7 * H ** -0.5
+    slopes0 = torch.tensor(O.head_slopes(H), dtype=torch.float64)
+    slopes = (talk.double() @ slopes0).float().to(dev)
+    sink = torch.randn(H, generator=g)
+    pages = {0: [4, 1, 6, 9, 2], 1: [7]}
+    data, want = {}, {}
+    for s, m in ((0, n), (1, n2)):
+        q = (torch.randn(m, H, D, generator=g)).bfloat16().float()
+        k = (torch.randn(m, G, D, generator=g)).bfloat16().float()
+        data[s] = (q, k)
+        want[s] = mixed_reference(q, k, talk, scale, slopes0, window, sink)
+    lens = [nq, 0, min(nq, n2)]
+    T = sum(lens)
+    bt = torch.tensor([pages[0] + [0] * 3, [0] * 8, pages[1] + [0] * 7], dtype=torch.int32, device=dev)
+    qs = torch.tensor([0, lens[0], lens[0]], dtype=torch.int32, device=dev)
+    ql = torch.tensor(lens, dtype=torch.int32, device=dev)
+    kvl = torch.tensor([n, 0, n2], dtype=torch.int32, device=dev)
+    off_q, off_k = 4, 4 + H * D + 3
+    proj = torch.randn(T + 2, off_k + G * D + 5, generator=g)
+    proj[:lens[0], off_q:off_q + H * D] = data[0][0][n - lens[0]:].reshape(lens[0], -1)
+    proj[lens[0]:T, off_q:off_q + H * D] = data[1][0][n2 - lens[2]:].reshape(lens[2], -1)
+    proj[:lens[0], off_k:off_k + G * D] = data[0][1][n - lens[0]:].reshape(lens[0], -1)
+    proj[lens[0]:T, off_k:off_k + G * D] = data[1][1][n2 - lens[2]:].reshape(lens[2], -1)
+    slot = [pages[0][j // 64] * 64 + j % 64 for j in range(n - lens[0], n)] + \
+           [pages[1][j // 64] * 64 + j % 64 for j in range(n2 - lens[2], n2)] + [-1, -1]          # two padding rows
+    slot = torch.tensor(slot, dtype=torch.int32, device=dev)
+    ref = torch.cat([want[0][n - lens[0]:], want[1][n2 - lens[2]:]], 0)
+    vec = D % 8 == 0
+    assert ops.mixed_attention_supported(H, G, D) == vec
+    for dtype, tol in ((torch.float32, 3e-5), (torch.bfloat16, 4e-2)):
+        kc = _paged(data[0][1], pages[0], dtype)
+        kc[7, :n2] = data[1][1].to(dev, dtype)
+        for s, m, l in ((0, n, lens[0]), (1, n2, lens[2])):                 # the new tokens' keys come from the prep kernel
+            for j in range(m - l, m):
+                kc[pages[s][j // 64], j % 64] = 5.0
+        fast = dtype == torch.bfloat16 and vec
+        qm = torch.zeros(T + 2, H * G * D, device=dev, dtype=torch.bfloat16 if fast else torch.float32)
+        ops.talk_prep(proj.to(dev), off_q, off_k, talk.to(dev), scale, slot, qm, kc, T + 2, H, G, D)
+        assert torch.equal(kc[4, 0].float().cpu(), data[0][1][0].to(dtype).float()) and float(qm[T:].float().abs().max()) == 0.0
+        assert torch.equal(kc[pages[0][4], (n - 1) % 64].float().cpu(), data[0][1][n - 1].to(dtype).float())
+        out = torch.zeros(T, (H * D + 7) // 8 * 8 + 8, device=dev, dtype=dtype)
+        if fast:
+            ops.mixed_attention(qm, kc, out, bt, qs, ql, kvl, 3, nq, H, G, D, window, slopes=slopes, sink=sink.to(dev))
+        else:
+            ops.softmax_attention(qm, kc.view(kc.shape[0], 64, 1, G * D), kc, out, bt, qs, ql, kvl, 3, nq, H, 1, G * D, D, window,
+                                  1.0, sink=sink.to(dev), v_heads=G, slopes=slopes)
+        got = out[:, :H * D].float().cpu().double().view(T, H, D)
+        assert torch.allclose(got, ref, atol=tol, rtol=tol), (dtype, float((got - ref).abs().max()))
+        assert float(out[:, H * D:].float().abs().max()) == 0.0
+    assert ops.native().mixed_attention_gave_up() == 0
+
+
+@gpu
+@pytest.mark.parametrize("S,H,G,D,window", [(32, 16, 4, 128, 1024), (3, 8, 2, 64, 500), (40, 4, 4, 32, 0), (150, 8, 1, 48, 200), (1, 32, 8, 128, 0)])
+def test_mixed_heads_decode_steps_without_sink_and_slopes(S, H, G, D, window):
+    """many sequences, one decoded token each at contexts around page borders: the cluster of CTAs per query (how many depends
+    on the batch) gives what the span kernel gives; neither sink nor distance bias"""
+    from bee2bee_b200 import ops
+
+    dev = "cuda"
+    g = torch.Generator().manual_seed(S + D)
+    ctx = [int(v) for v in torch.randint(1, 700, (S,), generator=g)]
+    for i, v in enumerate((64, 65, 63, 1, 128, 129, 448)):
+        ctx[i % S] = v
+    n_pages = sum((c + 63) // 64 for c in ctx) + 1
+    kc = (torch.randn(n_pages, 64, G, D, generator=g)).to(dev, torch.bfloat16)
+    perm = (torch.randperm(n_pages - 1, generator=g) + 1).tolist()
+    mp = 16
+    bt, at = torch.zeros(S, mp, dtype=torch.int32), 0
+    for i, c in enumerate(ctx):
+        m = (c + 63) // 64
+        bt[i, :m] = torch.tensor(perm[at:at + m], dtype=torch.int32)
+        at += m
+    bt = bt.to(dev)
+    q = (torch.randn(S, H * G * D, generator=g) * 2.0 * (G * D) ** -0.5).to(dev, torch.bfloat16)
+    qs = torch.arange(S, dtype=torch.int32, device=dev)
+    ql = torch.ones(S, dtype=torch.int32, device=dev)
+    kvl = torch.tensor(ctx, dtype=torch.int32, device=dev)
+    dec = torch.zeros(S, H * D, device=dev, dtype=torch.bfloat16)
+    span = torch.zeros_like(dec)
+    ops.mixed_attention(q, kc, dec, bt, qs, ql, kvl, S, 1, H, G, D, window)
+    ops.mixed_attention(q, kc, span, bt, qs, ql, kvl, S, 8, H, G, D, window)          # (as part of a longer-span batch)
+    want = torch.zeros(S, H, D, dtype=torch.float64)
+    kf, qf = kc.double().cpu(), q.double().cpu().view(S, H, G * D)
+    for i, c in enumerate(ctx):
+        rows = torch.cat([kf[int(b)] for b in bt[i, :(c + 63) // 64]], 0)[:c]
+        rows = rows[max(0, c - window) if window else 0:]
+        p = torch.softmax(qf[i] @ rows.reshape(-1, G * D).T, -1)
+        for h in range(H):
+            want[i, h] = p[h] @ rows[:, h // (H // G)]
+    for got in (dec, span):
+        d = (got.double().cpu().view(S, H, D) - want).abs().max()
+        assert float(d) < 4e-2, float(d)
+    assert ops.native().mixed_attention_gave_up() == 0
+
+
+@gpu
+@pytest.mark.parametrize("n,off", [(40, 0), (256, 4), (37, 3), (1000, 0), (4096, 8), (5000, 4), (16384, 0), (16400, 0)])
+def test_poly_norm_kernel(n, off):
+    from bee2bee_b200 import ops
+
+    dev, T, eps = "cuda", 5, 1e-3
+    g = torch.Generator().manual_seed(n)
+    x = torch.randn(T, off + n + (4 if n % 4 == 0 else 1), generator=g) * torch.tensor([0.01, 0.3, 1.0, 3.0, 10.0])[:, None]
+    w = torch.tensor([0.7, -0.4, 1.3, 0.25])
+    want = O.poly_norm(x[:, off:off + n].double(), w.double(), eps)
+    for dtype, tol in ((torch.float32, 2e-5), (torch.bfloat16, 2e-2)):
+        out = torch.zeros(T, (n + 63) // 64 * 64, device=dev, dtype=dtype)
+        ops.poly_norm(x.to(dev), off, w.to(dev), out, n, eps, T)
+        assert torch.allclose(out[:, :n].float().cpu().double(), want, atol=tol, rtol=1e-2 if dtype == torch.bfloat16 else 2e-5)
+        assert n % 64 == 0 or float(out[:, n:].float().abs().max()) == 0.0
+
+
+@gpu
+@pytest.mark.parametrize("E,top", [(12, 1), (5, 5), (7, 2), (64, 6), (3, 2), (1, 1)])
+def test_router_kernel_sigmoid_scores(E, top):
+    from bee2bee_b200 import ops
+
+    dev, T = "cuda", 40
+    g = torch.Generator().manual_seed(E)
+    z = torch.randn(T, E + 9, generator=g) * 2.0 - 1.0
+    idx, w = O.choose(z[:, 4:4 + E].double(), top)
+    wt = torch.full((T, E + 2), 9.0, device=dev)
+    idw = torch.full((T,), 9.0, device=dev)
+    sel_i, sel_w = torch.zeros(T, top, dtype=torch.int32, device=dev), torch.zeros(T, top, device=dev)
+    ops.moe_route(z.to(dev), 4, None, E, 1, 1, top, 1.0, wt, idw, T, sel_idx=sel_i, sel_w=sel_w, sigmoid=True)
+    assert sel_i.cpu().tolist() == idx and np.allclose(sel_w.cpu().numpy(), np.asarray(w), atol=1e-6)
+    dense_w = np.zeros((T, E))
+    for t in range(T):
+        dense_w[t, idx[t]] = w[t]
+    assert np.allclose(wt[:, :E].cpu().numpy(), dense_w, atol=1e-6) and float(idw.abs().max()) == 0.0
+
+
+@gpu
+@pytest.mark.parametrize("per,E", [(24, 5), (16, 3), (5, 4), (48, 10)])
+def test_gated_columns_with_scaled_input(per, E):
+    from bee2bee_b200 import ops
+
+    dev, T = "cuda", 11
+    n, off_a = per * E, 8
+    off_b = off_a + n + (4 if n % 4 == 0 else 3)
+    g = torch.Generator().manual_seed(n)
+    x = torch.randn(T, off_b + n + 5, generator=g) * 2.0
+    wt = torch.rand(T, E, generator=g) * (torch.rand(T, E, generator=g) > 0.5)
+    cw = wt.repeat_interleave(per, 1).double()
+    a = cw * x[:, off_a:off_a + n].double()
+    want = a * torch.sigmoid(a) * (cw * x[:, off_b:off_b + n].double())
+    for dtype, tol in ((torch.float32, 1e-5), (torch.bfloat16, 3e-2)):
+        out = torch.zeros(T, (n + 63) // 64 * 64, device=dev, dtype=dtype)
+        ops.gated_cols(x.to(dev), off_a, off_b, out, n, ops.GATE_SILU, T, wt=wt.to(dev), per=per, both=True, scale_input=True)
+        assert torch.allclose(out[:, :n].float().cpu().double(), want, atol=tol, rtol=1e-2)
+
+
+@gpu
+@pytest.mark.parametrize("T", [1, 33, 300])
+def test_linear_with_bias(T):
+    from bee2bee_b200 import ops
+
+    dev, K, N = "cuda", 128, 256
+    g = torch.Generator().manual_seed(T)
+    w, x, b = (torch.randn(*s, generator=g).bfloat16().float() for s in ((N, K), (T, K), (N,)))
+    want = x.double() @ w.double().T + b.double()
+    for dtype in (torch.float32, torch.bfloat16):
+        out = torch.zeros(T, N, device=dev)
+        ops.linear(w.to(dev, dtype), x.to(dev, dtype), out, bias=b.to(dev))
+        assert torch.allclose(out.cpu().double(), want, atol=2e-4, rtol=1e-4)
+
+
+# ---------------------------------------------------------------------------------------- every mechanism alone
+def _plain_talk(t):
+    for k in t:
+        if k.endswith(".talk"):
+            t[k] = torch.eye(t[k].shape[0])
+
+
+def _strong_talk(t):
+    for k in t:
+        if k.endswith(".talk"):
+            t[k] = torch.flip(t[k], (0,))                # every head mostly takes another head's scores
+
+
+def _level_talk(t):
+    """two heads: both rows of the mix orthogonal to the slopes (1/16, 1/256), so that far keys count as much as near ones"""
+    t["l0.mix.talk"] = torch.tensor([[0.0625, -1.0], [-0.0625, 1.0]])
+
+
+SINGLE = {
+    "attention": lambda: make_cfg([att(window=500)]),
+    "attention_windowed": lambda: make_cfg([att(window=20)]),
+    "attention_window_of_one": lambda: make_cfg([att(window=1)]),
+    "heads_with_keys_of_their_own": lambda: make_cfg([att(heads=3, kv=3, dim=24, window=70)]),
+    "one_key_head": lambda: make_cfg([att(heads=5, kv=1, dim=40, window=64)]),
+    "one_head": lambda: make_cfg([att(heads=1, kv=1, dim=64, window=65)]),
+    "heads_swapped_by_the_mix": lambda: make_cfg([att(heads=8, kv=4, dim=16, window=50)]),
+    "no_mix": lambda: make_cfg([att(heads=4, kv=2, window=50)]),
+    "narrow_heads": lambda: make_cfg([att(heads=4, kv=2, dim=6, window=33)]),
+    "poly_norm": lambda: make_cfg([att(window=9, mlp=dense())]),
+    "experts": lambda: make_cfg([att(window=9, mlp=moe())]),
+    "experts_top1": lambda: make_cfg([att(window=9, mlp=moe(experts=9, top=1))]),
+    "experts_all_chosen": lambda: make_cfg([att(window=9, mlp=moe(experts=3, ff=10, top=3))]),
+    "depth_of_five": lambda: make_cfg([att(window=9 + 7 * i, mlp=dense(32) if i % 2 else None) for i in range(5)]),
+    "odd_sizes": lambda: make_cfg([att(heads=6, kv=3, dim=10, window=37, scale=0.21, mlp=moe(experts=7, ff=9, top=3)),
+                                   att(heads=5, kv=5, dim=14, window=101, mlp=dense(45))], width=70, vocab=131, eps=1e-3),
+}
+
+
+@gpu
+@pytest.mark.parametrize("name", sorted(SINGLE))
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_each_mechanism_alone_whole_prompt(tmp_path, name, dtype):
+    cfg = SINGLE[name]()
+    t = make_tensors(cfg, seed=5, tweak={"no_mix": _plain_talk, "heads_swapped_by_the_mix": _strong_talk}.get(name))
+    tokens = toks(150, cfg["vocab"], 3)
+    want, trail = O.forward(cfg, t, tokens)
+    eng = engine(save_model(tmp_path / "m", cfg, t), dtype)
+    piece = eng.runner.piece
+    piece.debug_layers = []
+    got = eng.replay_step([("a", tokens, list(range(150)))], ["a"])
+    layers = [x[:150].float().cpu().double() for x in piece.debug_layers]
+    eng.close()
+    assert_close(got, want.float().numpy(), dtype, cfg, what=name)
+    if dtype == torch.float32:                              # (eager mode: the hook sees every layer exactly once)
+        assert len(layers) == len(trail)
+        for i, (a, b) in enumerate(zip(layers, trail)):
+            assert float((a - b).abs().max()) < 1e-3 * max(1.0, float(b.abs().max())), (name, i)
+
+
+@gpu
+def test_depth_average_reaches_back(tmp_path):
+    """the last average ignores everything but the embedding output and layer 0's result: the layers between do not show"""
+    cfg = make_cfg([att(mlp=dense()), att(window=50, mlp=moe()), att(kv=4)])
+
+    def tweak(t):
+        t["l2.dwa"] = torch.tensor([2.0, -1.5, 0.0, 0.0])
+
+    t = make_tensors(cfg, seed=8, tweak=tweak)
+    tokens = toks(90, cfg["vocab"], 2)
+    want = oracle_logits(tokens, t, cfg)
+    other = dict(t)
+    other["l1.mix.o"] = -t["l1.mix.o"]
+    assert rel_err(oracle_logits(tokens, other, cfg), want).max() < 1e-6
+    for dtype in (torch.float32, torch.bfloat16):
+        eng = engine(save_model(tmp_path / f"m{dtype}", cfg, t), dtype)
+        got = replay(eng, "a", tokens, [40, 2, 40])
+        eng.close()
+        assert rel_err(got, want).max() < TOL[dtype]
+
+
+def mixed_cfg(window=70, experts=True):
+    return make_cfg([att(window=window, mlp=dense(56)), att(heads=6, kv=3, dim=24, window=window + 60, mlp=moe() if experts else None),
+                     att(heads=2, kv=1, dim=32, window=40, mlp=moe(experts=4, top=1) if experts else dense(30))])
+
+
+MODES = [(torch.float32, True), (torch.bfloat16, True), (torch.bfloat16, False)]
+
+
+@gpu
+@pytest.mark.parametrize("dtype,experts", MODES)
+def test_portions_decode_and_page_borders(tmp_path, dtype, experts):
+    """a prompt cut into portions of many sizes (down to two tokens, across page and window borders) and token-by-token
+    decoding give the logits of the whole prompt"""
+    cfg = mixed_cfg(experts=experts)
+    t = make_tensors(cfg, seed=12)
+    tokens = toks(210, cfg["vocab"], 5)
+    want = oracle_logits(tokens, t, cfg)
+    eng = engine(save_model(tmp_path / "m", cfg, t), dtype)
+    runs = {"whole": replay(eng, "a", tokens, [210]),
+            "portions": replay(eng, "b", tokens, [2, 61, 2, 3, 60, 2, 64, 5]),          # cuts at 63 | 65 | 128 | 130, then single tokens
+            "decode": replay(eng, "c", tokens, [1])}
+    eng.close()
+    for k, g in runs.items():
+        assert_close(g, want, dtype, cfg, what=k)
+    if dtype == torch.float32:
+        assert np.abs(runs["portions"] - runs["whole"]).max() < 1e-3 * np.abs(want).max()
+
+
+@gpu
+@pytest.mark.parametrize("window", [1, 2, 17, 63, 64, 65, 127, 128, 129, 200])
+def test_window_edge_stands_out(tmp_path, window):
+    """a sharp softmax (score multiplier x 8, a mix that cancels the slopes) puts nearly all weight on one key, which for many
+    queries is the oldest key of the window: a window that is one token off, in prompts or in decoding, moves those logits by much more than rounding.
+    The oracle must itself change when the window does."""
+    lay = att(heads=2, kv=1, dim=16, window=window)
+    lay["mixer"]["scale"] *= 8.0
+    cfg = make_cfg([lay])
+    t = make_tensors(cfg, seed=21, tweak=_level_talk)
+    n = 200 if window < 100 else 380
+    tokens = toks(n, cfg["vocab"], 7)
+    want = oracle_logits(tokens, t, cfg)
+    for dw in (1, -1):
+        if window + dw < 1:
+            continue
+        other = json.loads(json.dumps(cfg))
+        other["layers"][0]["mixer"]["mask"] = {"size": window + dw}
+        assert rel_err(oracle_logits(tokens, t, other), want).max() > 0.1      # the edge key does matter
+    for dtype in (torch.float32, torch.bfloat16):
+        eng = engine(save_model(tmp_path / f"m{dtype}", cfg, t), dtype)
+        whole = replay(eng, "w", tokens, [n])
+        parts = replay(eng, "p", tokens, [3, 60, 2, 66, 9] + ([n - 200] if n > 200 else []))     # then 60 single tokens
+        eng.close()
+        assert_close(whole, want, dtype, cfg, what=f"window {window}, whole")
+        assert_close(parts, want, dtype, cfg, what=f"window {window}, parts")
+
+
+@gpu
+def test_distance_bias_and_the_one_in_the_denominator(tmp_path):
+    """with all products at zero only the distance bias is left: the weights are exp(-slope d) / (1 + sum), one mixed slope
+    per head, some of them negative (far keys then outweigh near ones); the served model follows the oracle, which changes
+    without the bias"""
+    cfg = make_cfg([att(heads=4, kv=2, window=90)])
+
+    def tweak(t):
+        t["l0.mix.q"], t["l0.mix.q.b"] = torch.zeros_like(t["l0.mix.q"]), torch.zeros_like(t["l0.mix.q.b"])
+        t["l0.mix.talk"] = torch.tensor([[1.0, 0, 0, 0], [0.125, 1.0, 0, 0.5], [-0.25, 0, 0, 0], [0, -2.0, 1.0, 1.0]])
+
+    t = make_tensors(cfg, seed=4, tweak=tweak)
+    tokens = toks(170, cfg["vocab"], 6)
+    want = oracle_logits(tokens, t, cfg)
+    flat = dict(t)
+    flat["l0.mix.talk"] = torch.zeros(4, 4)
+    assert rel_err(oracle_logits(tokens, flat, cfg), want).max() > 0.05
+    for dtype in (torch.float32, torch.bfloat16):
+        eng = engine(save_model(tmp_path / f"m{dtype}", cfg, t), dtype)
+        got = replay(eng, "a", tokens, [63, 2, 3, 80])
+        eng.close()
+        assert_close(got, want, dtype, cfg)
+    # scores far below zero: the one in the denominator empties the attention; the first token is the sharpest case
+    low = dict(t)
+    low["l0.mix.q.b"] = torch.ones_like(t["l0.mix.q.b"]) * 4.0
+    low["l0.mix.k.b"] = torch.ones_like(t["l0.mix.k.b"]) * -4.0
+    low["l0.mix.talk"] = torch.eye(4)
+    wl = oracle_logits(tokens, low, cfg)
+    eng = engine(save_model(tmp_path / "low", cfg, low), torch.float32)
+    got = replay(eng, "a", tokens, [1, 2, 100])
+    eng.close()
+    assert_close(got, wl, torch.float32, cfg)
+
+
+@gpu
+def test_far_key_inside_the_window_stands_out(tmp_path):
+    """a window of 320 keys and a sharp softmax without a slope (the mix cancels it): late queries look at single keys five
+    pages back, the first token among them; prompts that differ in their first token only still differ 200 tokens later, and
+    no longer once the window has moved past it"""
+    lay = att(heads=2, kv=1, dim=16, window=320)
+    lay["mixer"]["scale"] *= 4.0
+    cfg = make_cfg([lay])
+    t = make_tensors(cfg, seed=33, tweak=_level_talk)
+    a = toks(360, cfg["vocab"], 8)
+    b = [(a[0] + 17) % cfg["vocab"]] + a[1:]
+    wa, wb = oracle_logits(a, t, cfg), oracle_logits(b, t, cfg)
+    diff = rel_err(wa, wb)
+    assert diff[200:320].max() > 0.2 and diff[320:].max() < 1e-6
+    for dtype in (torch.float32, torch.bfloat16):
+        eng = engine(save_model(tmp_path / f"m{dtype}", cfg, t), dtype, max_tokens=768)
+        ga = replay(eng, "a", a, [300])                        # 300 in one go (cut by the chunk size), the rest decoded
+        gb = replay(eng, "b", b, [7, 2, 250])
+        eng.close()
+        assert_close(ga, wa, dtype, cfg, what="a")
+        assert_close(gb, wb, dtype, cfg, what="b")
+
+
+@gpu
+@pytest.mark.parametrize("dtype,experts", MODES)
+def test_mixed_batches_and_reused_slots_and_pages(tmp_path, dtype, experts):
+    """unequal requests in one batch (a long portion beside single tokens beside a new request) equal each alone;
+    ended requests give slot and pages back and the next ones get exactly those"""
+    cfg = mixed_cfg(window=44, experts=experts)
+    t = make_tensors(cfg, seed=14)
+    eng = engine(save_model(tmp_path / "m", cfg, t), dtype, max_tokens=320, slots=3)
+    V = cfg["vocab"]
+    seqs = {k: toks(n, V, 20 + i) for i, (k, n) in enumerate([("a", 100), ("b", 37), ("c", 66), ("d", 90), ("e", 30)])}
+    want = {k: oracle_logits(v, t, cfg) for k, v in seqs.items()}
+    got = {k: [] for k in seqs}
+    at = {k: 0 for k in seqs}
+
+    def step(plan, end=()):
+        entries = []
+        for k, n in plan:
+            entries.append((k, seqs[k][at[k]:at[k] + n], list(range(n))))
+        out = eng.replay_step(entries, list(end))
+        o = 0
+        for k, n in plan:
+            got[k].append(out[o:o + n])
+            o += n
+            at[k] += n
+
+    step([("a", 60), ("b", 2)])
+    step([("a", 1), ("b", 30), ("c", 5)])
+    step([("a", 3), ("b", 5), ("c", 61)], end=["b", "c"])            # b and c finish: their slots and pages are free again
+    step([("a", 36), ("d", 64), ("e", 2)], end=["a"])                 # d and e reuse them (pool: 5 pages, 3 slots)
+    step([("d", 1), ("e", 1)])
+    step([("d", 2), ("e", 27)], end=["e"])
+    step([("d", 23)], end=["d"])
+    eng.close()
+    assert not eng._replay
+    for k in seqs:
+        g = np.concatenate(got[k])
+        assert g.shape[0] == len(seqs[k])
+        assert_close(g, want[k], dtype, cfg, what=k)
+
+
+@gpu
+def test_long_decoding_single_tokens(tmp_path):
+    cfg = make_cfg([att(heads=4, kv=2, dim=32, window=100, mlp=moe(experts=4, ff=32, top=2)), att(heads=8, kv=2, dim=48, window=64),
+                    att(heads=2, kv=2, dim=16, window=130, mlp=dense(64))])
+    t = make_tensors(cfg, seed=31)
+    tokens = toks(260, cfg["vocab"], 9)
+    want = oracle_logits(tokens, t, cfg)
+    for dtype in (torch.float32, torch.bfloat16):
+        eng = engine(save_model(tmp_path / f"m{dtype}", cfg, t), dtype)
+        got = replay(eng, "x", tokens, [20])                       # 240 single-token steps across 4 page borders
+        eng.close()
+        assert_close(got, want, dtype, cfg)
+
+
+@gpu
+def test_greedy_generation_through_the_scheduler(tmp_path):
+    """Engine.generate: admission, chunked prefill, CUDA-graph decode bursts, sampler -- greedy tokens equal the
+    oracle's argmax continuation; unequal requests share the batch; the second round of requests shares prompt pages"""
+    from bee2bee_b200.engine.core import Engine, SamplingParams
+
+    cfg = mixed_cfg(window=24)
+    t = make_tensors(cfg, seed=48)
+    path = save_model(tmp_path / "m", cfg, t)
+    prompts = [toks(70, cfg["vocab"], 1), toks(9, cfg["vocab"], 2), toks(3, cfg["vocab"], 3)]
+    n_new = 12
+    want = []
+    for p in prompts:
+        seq = list(p)
+        for _ in range(n_new):
+            lg = oracle_logits(seq, t, cfg)[-1]
+            top2 = np.sort(lg)[-2:]
+            assert top2[1] - top2[0] > 1e-3, "test weights give a near tie: pick another seed"
+            seq.append(int(lg.argmax()))
+        want.append(seq[len(p):])
+    eng = Engine(path, device="cuda:0", max_batch=4, max_seq_len=256, max_prefill_tokens=32, decode_burst=5,
+                 dtype=torch.float32)
+    sp = SamplingParams(max_new_tokens=n_new, temperature=0.0, repetition_penalty=1.0, ignore_eos=True)
+    got = eng.generate(prompts, sp)
+    again = eng.generate(prompts[::-1], sp)                        # slots and pages are used a second time
+    eng.close()
+    assert got == want and again == want[::-1]
+    eng = Engine(path, device="cuda:0", max_batch=4, max_seq_len=256, max_prefill_tokens=64, decode_burst=4)
+    out = eng.generate(prompts, sp)                                # bf16 serving mode: graphs + tcgen05 kernels
+    eng.close()
+    agree = sum(a == b for g, w in zip(out, want) for a, b in zip(g, w))
+    assert all(len(o) == n_new for o in out) and agree >= 0.6 * 3 * n_new
+
+
+@gpu
+def test_preset_generates_with_random_weights():
+    from bee2bee_b200.engine.core import Engine, SamplingParams
+
+    eng = Engine("tiny-kazolorn", device="cuda:0", max_batch=4, max_seq_len=256, decode_burst=4)
+    outs = eng.generate([[1, 5, 9, 33, 2, 7, 8, 100], [4, 4, 19]], SamplingParams(max_new_tokens=8, ignore_eos=True))
+    eng.close()
+    assert all(len(o) == 8 for o in outs)
+
+
+@gpu
+def test_trace_run_command_line(tmp_path):
+    """bin/trace_run: steps on stdin, `done <step>` lines on stdout, logits files in --out; slots and pages of ended
+    sequences serve the next ones (pool of 192 tokens = 3 pages, 2 slots)"""
+    import subprocess
+    import sys
+
+    cfg = make_cfg([att(heads=2, kv=1, dim=16, window=50, mlp=dense(32)), att(heads=4, kv=2, dim=8, window=30)])
+    t = make_tensors(cfg, seed=51)
+    path = save_model(tmp_path / "m", cfg, t)
+    a, b, c = toks(70, cfg["vocab"], 1), toks(40, cfg["vocab"], 2), toks(64, cfg["vocab"], 3)
+    steps = [
+        {"step": 0, "entries": [{"id": "a", "tokens": a[:30], "want": [0, 29]}], "end": []},
+        {"step": 1, "entries": [{"id": "a", "tokens": a[30:], "want": []}, {"id": "b", "tokens": b[:2], "want": [1]}], "end": ["a"]},
+        {"step": 2, "entries": [{"id": "b", "tokens": b[2:], "want": [37]}, {"id": "c", "tokens": c, "want": [0, 63]}],
+         "end": ["b", "c"]},
+    ]
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    out = tmp_path / "out"
+    for dtype, tol in (("float32", 1e-4), ("bfloat16", 5e-2)):
+        res = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", path, "--dtype", dtype,
+                              "--out", str(out), "--max-tokens", "192", "--slots", "2"],
+                             input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
+        assert res.returncode == 0, res.stderr[-2000:]
+        assert [l for l in res.stdout.splitlines() if l.startswith("done")] == ["done 0", "done 1", "done 2"]
+        wa, wb, wc = (oracle_logits(x, t, cfg) for x in (a, b, c))
+        got0 = np.fromfile(out / "0.f32", dtype="<f4").reshape(-1, cfg["vocab"])
+        got1 = np.fromfile(out / "1.f32", dtype="<f4").reshape(-1, cfg["vocab"])
+        got2 = np.fromfile(out / "2.f32", dtype="<f4").reshape(-1, cfg["vocab"])
+        assert rel_err(got0, wa[[0, 29]]).max() < tol and rel_err(got1, wb[[1]]).max() < tol
+        assert rel_err(got2, np.concatenate([wb[[39]], wc[[0, 63]]])).max() < tol
