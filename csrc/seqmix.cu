@@ -90,6 +90,7 @@ struct JoinTerm {
 // of squares, pass 3 writes the operand.  VEC: 16-byte accesses (W and every row stride multiples of 4).
 // replace: the new residual row is the sum of the terms alone (the old row is not read).  gamma == nullptr: the operand is
 // the residual row itself.  gamma2 / h2: a second normed operand of the same row (blocks whose two sublayers have a norm each).
+// WPT = 16: few wide rows (decode steps), sixteen warps per token so that a thread has one or two accesses to wait for.
 // past (depth averages): the joined row is kept as past[k] ([entry of stride `dstride` floats][token][W]) and the residual
 // row becomes sum_j dw[j] past[j] over j <= k; xin: the row that entered the layer (x itself, or past[0] in the first layer).
 // grid (groups of LSJ_WARPS / WPT tokens, sequences) or (groups of rows); dynamic smem LSJ_WARPS / WPT * W floats.
@@ -128,7 +129,7 @@ __device__ __forceinline__ void st_operand(bf16* h, int i, float4 v, bool vec) {
 }
 
 template <typename OT, bool VEC, int WPT>
-__global__ void __launch_bounds__(32 * LSJ_WARPS)
+__global__ void __launch_bounds__(32 * (WPT > LSJ_WARPS ? WPT : LSJ_WARPS))
     ls_join_kernel(float* __restrict__ x, const int* __restrict__ q_start, const int* __restrict__ q_len,
                    const int* __restrict__ rows, int n_rows, JoinTerm a, JoinTerm b, JoinTerm c, float eps,
                    const float* __restrict__ gamma, int gstride, int plus_one, OT* __restrict__ h, int ld_h, int W,
@@ -137,7 +138,7 @@ __global__ void __launch_bounds__(32 * LSJ_WARPS)
   pdl_begin();
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
-  constexpr int TPB = LSJ_WARPS / WPT, NL = 32 * WPT;       // tokens per block, threads per token
+  constexpr int TPB = WPT > LSJ_WARPS ? 1 : LSJ_WARPS / WPT, NL = 32 * WPT;       // tokens per block, threads per token
   const int grp = threadIdx.x / NL, lane = threadIdx.x % NL;
   float* xs = sm + static_cast<size_t>(grp) * ((W + 3) & ~3);
   auto total = [&](float v) { return WPT == 1 ? warp_sum_(v) : block_sum_(v, red); };
@@ -173,6 +174,23 @@ __global__ void __launch_bounds__(32 * LSJ_WARPS)
   float ss = 0.f;
   for (int i = lane; i < nv; i += NL) {
     float4 v = replace ? make_float4(0.f, 0.f, 0.f, 0.f) : Ld4<VEC>::ld(xi, i);
+    // (the older rows first: their loads do not wait for the store of the joined row)
+    float4 old = make_float4(0.f, 0.f, 0.f, 0.f);
+    float* pr = nullptr;
+    if (dep.past != nullptr) {
+      pr = dep.past + static_cast<size_t>(t) * W;
+#pragma unroll 4
+      for (int j = 0; j < dep.k; ++j) {
+        const float4 pv = Ld4<VEC>::ld(pr + j * dep.dstride, i);
+        const float wj = dep.dw[j];
+        old.x += wj * pv.x;
+        if (VEC) {
+          old.y += wj * pv.y;
+          old.z += wj * pv.z;
+          old.w += wj * pv.w;
+        }
+      }
+    }
 #pragma unroll
     for (int k = 0; k < 3; ++k) {
       if (terms[k].y == nullptr) continue;
@@ -187,21 +205,9 @@ __global__ void __launch_bounds__(32 * LSJ_WARPS)
       }
     }
     if (dep.past != nullptr) {
-      float* pr = dep.past + static_cast<size_t>(t) * W;
       if (rows == nullptr) Ld4<VEC>::st(pr + dep.k * dep.dstride, i, v);
       const float wk = dep.dw[dep.k];
-      v.x *= wk; v.y *= wk; v.z *= wk; v.w *= wk;
-#pragma unroll 4
-      for (int j = 0; j < dep.k; ++j) {
-        const float4 pv = Ld4<VEC>::ld(pr + j * dep.dstride, i);
-        const float wj = dep.dw[j];
-        v.x += wj * pv.x;
-        if (VEC) {
-          v.y += wj * pv.y;
-          v.z += wj * pv.z;
-          v.w += wj * pv.w;
-        }
-      }
+      v = make_float4(wk * v.x + old.x, wk * v.y + old.y, wk * v.z + old.z, wk * v.w + old.w);
     }
     ss += v.x * v.x + (VEC ? v.y * v.y + v.z * v.z + v.w * v.w : 0.f);
     Ld4<VEC>::st(xs, i, v);
@@ -327,9 +333,9 @@ __global__ void __launch_bounds__(256)
 // score_h = sum_g talk[h, g] scale (q_g . k_(g's key head)) = qm_h . [k_0 | k_1 | ...] with, per key head c,
 //     qm[h, c, :] = scale * sum over the heads g of key head c of talk[h, g] q_g
 // so a head needs ONE dot product with the whole cached key row (G * D channels) and no exchange with other heads.
-// proj [T, ld] fp32 holds q (H*D) at off_q, k (G*D) at off_k.  One block per token: the query row and the matrix (transposed,
-// rows padded to a multiple of 4) in shared memory; a thread owns E adjacent channels of one key head and writes them for
-// every head.  qm -> q_out [T, H*G*D], key row -> cache.
+// proj [T, ld] fp32 holds q (H*D) at off_q, k (G*D) at off_k.  One block per (token, key head): the queries of its heads and
+// their columns of the matrix (transposed, rows padded to a multiple of 4) in shared memory; a warp owns four mixed rows, a
+// lane E adjacent channels of each (VL: q and k are read with 16-byte loads).  qm -> q_out [T, H*G*D], key row -> cache.
 template <typename CT, int E> __device__ __forceinline__ void st_run(CT* p, const float (&v)[E]) {
   if constexpr (E == 1) stf(p, 0, v[0]);
   else if constexpr (sizeof(CT) == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
@@ -338,35 +344,49 @@ template <typename CT, int E> __device__ __forceinline__ void st_run(CT* p, cons
     return make_uint2(*reinterpret_cast<unsigned*>(&a), *reinterpret_cast<unsigned*>(&b));
   }();
 }
-template <typename QT, typename CT, int E>
+template <typename QT, typename CT, int E, bool VL>
 __global__ void __launch_bounds__(256)
     talk_prep_kernel(const float* __restrict__ proj, int ld, int off_q, int off_k, const float* __restrict__ talk,
                      float scale, const int* __restrict__ slots, QT* __restrict__ q_out, CT* __restrict__ k_cache, int H,
                      int G, int D) {
   pdl_begin();
   extern __shared__ __align__(16) float tp[];
-  const int t = blockIdx.x, slot = slots[t];
+  const int t = blockIdx.x, kv = blockIdx.y, slot = slots[t];
   if (slot < 0) return;                               // padding row of a bucketed chunk (block-uniform)
-  const int Hp = (H + 3) & ~3, nq = H * D, nk = G * D, per = H / G;
-  float* qs = tp;                                     // [H * D]
-  float* tt = tp + ((nq + 3) & ~3);                   // [H (mixed from)][Hp (mixed into)]
-  const float* row = proj + static_cast<size_t>(t) * ld;
-  for (int i = threadIdx.x; i < nq; i += blockDim.x) qs[i] = row[off_q + i] * scale;
-  for (int i = threadIdx.x; i < H * H; i += blockDim.x) tt[i % H * Hp + i / H] = talk[i];
-  if (Hp != H)
-    for (int i = threadIdx.x; i < H * (Hp - H); i += blockDim.x) tt[i / (Hp - H) * Hp + H + i % (Hp - H)] = 0.f;
-  for (int i = threadIdx.x; i < nk; i += blockDim.x) stf(k_cache, static_cast<size_t>(slot) * nk + i, row[off_k + i]);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int Hp = (H + 3) & ~3, nk = G * D, per = H / G, g0 = kv * per;
+  float* qs = tp;                                     // [per][D]
+  float* tt = tp + ((per * D + 3) & ~3);              // [per (mixed from)][Hp (mixed into)]
+  const float* qr = proj + static_cast<size_t>(t) * ld + off_q + g0 * D;
+  const float* kr = proj + static_cast<size_t>(t) * ld + off_k + kv * D;
+  CT* kd = k_cache + static_cast<size_t>(slot) * nk + kv * D;
+  if constexpr (VL) {
+    for (int i = threadIdx.x * 4; i < per * D; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(qr + i);
+      *reinterpret_cast<float4*>(qs + i) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+    }
+    for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(kr + i);
+      const float kv4[4] = {v.x, v.y, v.z, v.w};
+      st_run<CT, 4>(kd + i, kv4);
+    }
+  } else {
+    for (int i = threadIdx.x; i < per * D; i += blockDim.x) qs[i] = qr[i] * scale;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) stf(kd, i, kr[i]);
+  }
+  for (int h = warp; h < Hp; h += nw)
+    for (int g = lane; g < per; g += 32) tt[g * Hp + h] = h < H ? talk[h * H + g0 + g] : 0.f;
   __syncthreads();
-  QT* qo = q_out + static_cast<size_t>(t) * H * nk;
-  for (int c = threadIdx.x * E; c < nk; c += blockDim.x * E) {
-    const int kv = c / D, d = c % D;                  // (E divides D: the run stays inside one key head)
-    for (int h0 = 0; h0 < H; h0 += 4) {
+  QT* qo = q_out + static_cast<size_t>(t) * H * nk + kv * D;
+  for (int h0 = 4 * warp; h0 < H; h0 += 4 * nw) {
+    for (int d = lane * E; d < D; d += 32 * E) {
       float acc[4][E];
 #pragma unroll
       for (int a = 0; a < 4; ++a)
 #pragma unroll
         for (int e = 0; e < E; ++e) acc[a][e] = 0.f;
-      for (int g = kv * per; g < (kv + 1) * per; ++g) {
+#pragma unroll 4
+      for (int g = 0; g < per; ++g) {
         const float4 w = *reinterpret_cast<const float4*>(tt + g * Hp + h0);
         const float wa[4] = {w.x, w.y, w.z, w.w};
         float qv[E];
@@ -383,7 +403,7 @@ __global__ void __launch_bounds__(256)
       }
 #pragma unroll
       for (int a = 0; a < 4; ++a)
-        if (h0 + a < H) st_run<QT, E>(qo + static_cast<size_t>(h0 + a) * nk + c, acc[a]);
+        if (h0 + a < H) st_run<QT, E>(qo + static_cast<size_t>(h0 + a) * nk + d, acc[a]);
     }
   }
 }
@@ -1313,18 +1333,20 @@ int launch_ls_join(float* x, const int* q_start, const int* q_len, const int* ro
                    (y1 == nullptr || (ld1 % 4 == 0 && al16(y1))) && (y2 == nullptr || (ld2 % 4 == 0 && al16(y2))) &&
                    al16(w0) && al16(w1) && al16(w2) && al16(xin) && al16(past) && dstride % 4 == 0 && (h == nullptr || (ld_h % 4 == 0 && al16(h))) &&
                    (gstride == 0 || al16(gamma)) && (h2 == nullptr || (ld_h2 % 4 == 0 && al16(h2) && al16(gamma2)));
+  const bool few = wide && W >= 1024 && static_cast<long long>(grid.x) * grid.y <= 296;
 #define B2B_LSJ1(OT, VEC, WPT)                                                                                          \
   do {                                                                                                                  \
     if (smem > 48 * 1024)                                                                                               \
       cudaFuncSetAttribute(ls_join_kernel<OT, VEC, WPT>, cudaFuncAttributeMaxDynamicSharedMemorySize,                   \
                            static_cast<int>(smem));                                                                     \
-    launch_kernel(ls_join_kernel<OT, VEC, WPT>, grid, dim3(32 * LSJ_WARPS), smem, s, 1u, x, q_start, q_len, rows, n_rows, \
+    launch_kernel(ls_join_kernel<OT, VEC, WPT>, grid, dim3(32 * (WPT > LSJ_WARPS ? WPT : LSJ_WARPS)), smem, s, 1u, x, q_start, q_len, rows, n_rows, \
                   a, b, c, eps, gamma, gstride, plus_one, static_cast<OT*>(h), ld_h, W, gamma2, static_cast<OT*>(h2),    \
                   ld_h2, replace, xin, dep);                                                                            \
   } while (0)
 #define B2B_LSJ(OT, VEC)                                                                                                \
   do {                                                                                                                  \
-    if (wide) B2B_LSJ1(OT, VEC, LSJ_WARPS);                                                                             \
+    if (few) B2B_LSJ1(OT, VEC, 16);                                                                                     \
+    else if (wide) B2B_LSJ1(OT, VEC, LSJ_WARPS);                                                                        \
     else B2B_LSJ1(OT, VEC, 1);                                                                                          \
   } while (0)
   if (f32) {
@@ -1367,16 +1389,26 @@ int launch_talk_prep(const float* proj, int ld, int off_q, int off_k, const floa
                      void* q_out, void* k_cache, int T, int H, int G, int D, int q_f32, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || D <= 0 || (f32 && !q_f32)) return -2;
-  const size_t smem = (static_cast<size_t>((H * D + 3) & ~3) + static_cast<size_t>(H) * ((H + 3) & ~3)) * sizeof(float);
+  const int per = H / G;
+  const size_t smem = (static_cast<size_t>((per * D + 3) & ~3) + static_cast<size_t>(per) * ((H + 3) & ~3)) * sizeof(float);
   if (smem > 200 * 1024) return -2;
   const bool vec = D % 4 == 0 && reinterpret_cast<uintptr_t>(q_out) % 16 == 0;
-  const dim3 block(vec && G * D <= 512 ? 128 : 256);
-#define B2B_TALK(QT, CT, E)                                                                                             \
+  const bool vl = vec && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0 &&
+                  reinterpret_cast<uintptr_t>(k_cache) % 16 == 0;
+  const int groups = (H + 3) / 4;
+  const dim3 block(32 * (groups < 2 ? 2 : (groups > 8 ? 8 : groups)));
+#define B2B_TALK1(QT, CT, E, VL)                                                                                        \
   do {                                                                                                                  \
     if (smem > 48 * 1024)                                                                                               \
-      cudaFuncSetAttribute(talk_prep_kernel<QT, CT, E>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)); \
-    launch_kernel(talk_prep_kernel<QT, CT, E>, dim3(T), block, smem, s, 1u, proj, ld, off_q, off_k, talk, scale, slots,  \
-                  static_cast<QT*>(q_out), static_cast<CT*>(k_cache), H, G, D);                                         \
+      cudaFuncSetAttribute(talk_prep_kernel<QT, CT, E, VL>, cudaFuncAttributeMaxDynamicSharedMemorySize,                \
+                           static_cast<int>(smem));                                                                     \
+    launch_kernel(talk_prep_kernel<QT, CT, E, VL>, dim3(T, G), block, smem, s, 1u, proj, ld, off_q, off_k, talk, scale,  \
+                  slots, static_cast<QT*>(q_out), static_cast<CT*>(k_cache), H, G, D);                                  \
+  } while (0)
+#define B2B_TALK(QT, CT, E)                                                                                             \
+  do {                                                                                                                  \
+    if (E == 4 && vl) B2B_TALK1(QT, CT, E, true);                                                                       \
+    else B2B_TALK1(QT, CT, E, false);                                                                                   \
   } while (0)
   if (f32) {
     if (vec) B2B_TALK(float, float, 4);
@@ -1389,6 +1421,7 @@ int launch_talk_prep(const float* proj, int ld, int off_q, int off_k, const floa
     else B2B_TALK(bf16, bf16, 1);
   }
 #undef B2B_TALK
+#undef B2B_TALK1
   return last_error();
 }
 

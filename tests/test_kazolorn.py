@@ -371,6 +371,30 @@ def test_mixed_heads_attention_kernels(H, G, D, nq, window):
 
 
 @gpu
+@pytest.mark.parametrize("H,G,D,T", [(8, 2, 32, 600), (6, 2, 20, 515), (3, 3, 7, 512), (12, 1, 120, 513)])
+def test_mixed_query_rows_of_many_tokens(H, G, D, T):
+    """a chunk large enough that one block serves several tokens: rows, key copies, padding rows left alone"""
+    from bee2bee_b200 import ops
+
+    dev = "cuda"
+    g = torch.Generator().manual_seed(T)
+    proj, talk = torch.randn(T, (H + G) * D + 3, generator=g), torch.randn(H, H, generator=g)
+    slots = torch.randperm(1024, generator=g)[:T].int()
+    slots[[5, 100, T - 1]] = -1
+    q = proj[:, 2:2 + H * D].double().view(T, G, H // G, D)
+    want = torch.einsum("hcj,tcjd->thcd", talk.double().view(H, G, H // G), q).reshape(T, -1) * 0.3
+    for qdt, cdt, tol in ((torch.float32, torch.float32, 1e-5), (torch.float32, torch.bfloat16, 1e-5), (torch.bfloat16, torch.bfloat16, 3e-2)):
+        out, kc = torch.full((T, H * G * D), 7.0, device=dev, dtype=qdt), torch.full((16, 64, G, D), 7.0, device=dev, dtype=cdt)
+        ops.talk_prep(proj.to(dev), 2, 2 + H * D, talk.to(dev), 0.3, slots.to(dev), out, kc, T, H, G, D)
+        ok = slots >= 0
+        assert torch.allclose(out.cpu().double()[ok], want[ok], atol=tol, rtol=tol) and bool((out.cpu()[~ok] == 7.0).all())
+        rows = kc.view(1024, G * D).float().cpu()
+        assert torch.equal(rows[slots[ok].long()], proj[ok, 2 + H * D:2 + H * D + G * D].to(cdt).float())
+        rest = [i for i in range(1024) if i not in set(slots.tolist())]
+        assert bool((rows[rest] == 7.0).all())
+
+
+@gpu
 @pytest.mark.parametrize("S,H,G,D,window", [(32, 16, 4, 128, 1024), (3, 8, 2, 64, 500), (40, 4, 4, 32, 0), (150, 8, 1, 48, 200), (1, 32, 8, 128, 0)])
 def test_mixed_heads_decode_steps_without_sink_and_slopes(S, H, G, D, window):
     """many sequences, one decoded token each at contexts around page borders: the cluster of CTAs per query (how many depends
