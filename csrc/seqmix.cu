@@ -333,9 +333,10 @@ __global__ void __launch_bounds__(256)
 // score_h = sum_g talk[h, g] scale (q_g . k_(g's key head)) = qm_h . [k_0 | k_1 | ...] with, per key head c,
 //     qm[h, c, :] = scale * sum over the heads g of key head c of talk[h, g] q_g
 // so a head needs ONE dot product with the whole cached key row (G * D channels) and no exchange with other heads.
-// proj [T, ld] fp32 holds q (H*D) at off_q, k (G*D) at off_k.  One block per (token, key head): the queries of its heads and
-// their columns of the matrix (transposed, rows padded to a multiple of 4) in shared memory; a warp owns four mixed rows, a
-// lane E adjacent channels of each (VL: q and k are read with 16-byte loads).  qm -> q_out [T, H*G*D], key row -> cache.
+// proj [T, ld] fp32 holds q (H*D) at off_q, k (G*D) at off_k.  One block per (token, `cnt` key heads): the queries of
+// their heads and their columns of the matrix (transposed, rows padded to a multiple of 4) in shared memory; a warp owns four
+// mixed rows of one key head, a lane E adjacent channels of each (VL: q and k are read with 16-byte loads).
+// qm -> q_out [T, H*G*D], key row -> cache.
 template <typename CT, int E> __device__ __forceinline__ void st_run(CT* p, const float (&v)[E]) {
   if constexpr (E == 1) stf(p, 0, v[0]);
   else if constexpr (sizeof(CT) == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
@@ -348,37 +349,41 @@ template <typename QT, typename CT, int E, bool VL>
 __global__ void __launch_bounds__(256)
     talk_prep_kernel(const float* __restrict__ proj, int ld, int off_q, int off_k, const float* __restrict__ talk,
                      float scale, const int* __restrict__ slots, QT* __restrict__ q_out, CT* __restrict__ k_cache, int H,
-                     int G, int D) {
+                     int G, int D, int cnt) {
   pdl_begin();
   extern __shared__ __align__(16) float tp[];
-  const int t = blockIdx.x, kv = blockIdx.y, slot = slots[t];
+  const int t = blockIdx.x, kv0 = blockIdx.y * cnt, slot = slots[t];
   if (slot < 0) return;                               // padding row of a bucketed chunk (block-uniform)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const int Hp = (H + 3) & ~3, nk = G * D, per = H / G, g0 = kv * per;
-  float* qs = tp;                                     // [per][D]
-  float* tt = tp + ((per * D + 3) & ~3);              // [per (mixed from)][Hp (mixed into)]
+  const int Hp = (H + 3) & ~3, nk = G * D, per = H / G, g0 = kv0 * per, ng = cnt * per;
+  float* qs = tp;                                     // [ng][D]
+  float* tt = tp + ((ng * D + 3) & ~3);               // [ng (mixed from)][Hp (mixed into)]
   const float* qr = proj + static_cast<size_t>(t) * ld + off_q + g0 * D;
-  const float* kr = proj + static_cast<size_t>(t) * ld + off_k + kv * D;
-  CT* kd = k_cache + static_cast<size_t>(slot) * nk + kv * D;
+  const float* kr = proj + static_cast<size_t>(t) * ld + off_k + kv0 * D;
+  CT* kd = k_cache + static_cast<size_t>(slot) * nk + kv0 * D;
   if constexpr (VL) {
-    for (int i = threadIdx.x * 4; i < per * D; i += blockDim.x * 4) {
+    for (int i = threadIdx.x * 4; i < ng * D; i += blockDim.x * 4) {
       const float4 v = *reinterpret_cast<const float4*>(qr + i);
       *reinterpret_cast<float4*>(qs + i) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
     }
-    for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
+    for (int i = threadIdx.x * 4; i < cnt * D; i += blockDim.x * 4) {
       const float4 v = *reinterpret_cast<const float4*>(kr + i);
       const float kv4[4] = {v.x, v.y, v.z, v.w};
       st_run<CT, 4>(kd + i, kv4);
     }
   } else {
-    for (int i = threadIdx.x; i < per * D; i += blockDim.x) qs[i] = qr[i] * scale;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) stf(kd, i, kr[i]);
+    for (int i = threadIdx.x; i < ng * D; i += blockDim.x) qs[i] = qr[i] * scale;
+    for (int i = threadIdx.x; i < cnt * D; i += blockDim.x) stf(kd, i, kr[i]);
   }
   for (int h = warp; h < Hp; h += nw)
-    for (int g = lane; g < per; g += 32) tt[g * Hp + h] = h < H ? talk[h * H + g0 + g] : 0.f;
+    for (int g = lane; g < ng; g += 32) tt[g * Hp + h] = h < H ? talk[h * H + g0 + g] : 0.f;
   __syncthreads();
-  QT* qo = q_out + static_cast<size_t>(t) * H * nk + kv * D;
-  for (int h0 = 4 * warp; h0 < H; h0 += 4 * nw) {
+  const int groups = Hp >> 2;
+  for (int u = warp; u < cnt * groups; u += nw) {
+    const int kv = u / groups, h0 = 4 * (u - kv * groups);
+    const float* tk = tt + kv * per * Hp + h0;
+    const float* qk = qs + kv * per * D;
+    QT* qo = q_out + static_cast<size_t>(t) * H * nk + (kv0 + kv) * D;
     for (int d = lane * E; d < D; d += 32 * E) {
       float acc[4][E];
 #pragma unroll
@@ -387,14 +392,14 @@ __global__ void __launch_bounds__(256)
         for (int e = 0; e < E; ++e) acc[a][e] = 0.f;
 #pragma unroll 4
       for (int g = 0; g < per; ++g) {
-        const float4 w = *reinterpret_cast<const float4*>(tt + g * Hp + h0);
+        const float4 w = *reinterpret_cast<const float4*>(tk + g * Hp);
         const float wa[4] = {w.x, w.y, w.z, w.w};
         float qv[E];
         if constexpr (E == 4) {
-          const float4 v = *reinterpret_cast<const float4*>(qs + g * D + d);
+          const float4 v = *reinterpret_cast<const float4*>(qk + g * D + d);
           qv[0] = v.x; qv[1] = v.y; qv[2] = v.z; qv[3] = v.w;
         } else {
-          qv[0] = qs[g * D + d];
+          qv[0] = qk[g * D + d];
         }
 #pragma unroll
         for (int a = 0; a < 4; ++a)
@@ -1389,21 +1394,22 @@ int launch_talk_prep(const float* proj, int ld, int off_q, int off_k, const floa
                      void* q_out, void* k_cache, int T, int H, int G, int D, int q_f32, int f32, cudaStream_t s) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || D <= 0 || (f32 && !q_f32)) return -2;
-  const int per = H / G;
-  const size_t smem = (static_cast<size_t>((per * D + 3) & ~3) + static_cast<size_t>(per) * ((H + 3) & ~3)) * sizeof(float);
+  // chunks: all key heads of a token in one block; decode steps: one each, so that a few tokens spread over the machine
+  const int cnt = T >= 512 && static_cast<size_t>(H) * (D + H + 3) * sizeof(float) <= 48 * 1024 ? G : 1, ng = cnt * (H / G);
+  const size_t smem = (static_cast<size_t>((ng * D + 3) & ~3) + static_cast<size_t>(ng) * ((H + 3) & ~3)) * sizeof(float);
   if (smem > 200 * 1024) return -2;
   const bool vec = D % 4 == 0 && reinterpret_cast<uintptr_t>(q_out) % 16 == 0;
   const bool vl = vec && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 && reinterpret_cast<uintptr_t>(proj) % 16 == 0 &&
                   reinterpret_cast<uintptr_t>(k_cache) % 16 == 0;
-  const int groups = (H + 3) / 4;
+  const int groups = cnt * ((H + 3) / 4);
   const dim3 block(32 * (groups < 2 ? 2 : (groups > 8 ? 8 : groups)));
 #define B2B_TALK1(QT, CT, E, VL)                                                                                        \
   do {                                                                                                                  \
     if (smem > 48 * 1024)                                                                                               \
       cudaFuncSetAttribute(talk_prep_kernel<QT, CT, E, VL>, cudaFuncAttributeMaxDynamicSharedMemorySize,                \
                            static_cast<int>(smem));                                                                     \
-    launch_kernel(talk_prep_kernel<QT, CT, E, VL>, dim3(T, G), block, smem, s, 1u, proj, ld, off_q, off_k, talk, scale,  \
-                  slots, static_cast<QT*>(q_out), static_cast<CT*>(k_cache), H, G, D);                                  \
+    launch_kernel(talk_prep_kernel<QT, CT, E, VL>, dim3(T, G / cnt), block, smem, s, 1u, proj, ld, off_q, off_k, talk,   \
+                  scale, slots, static_cast<QT*>(q_out), static_cast<CT*>(k_cache), H, G, D, cnt);                                  \
   } while (0)
 #define B2B_TALK(QT, CT, E)                                                                                             \
   do {                                                                                                                  \
