@@ -396,7 +396,7 @@ def test_mixed_query_rows_of_many_tokens(H, G, D, T):
 
 
 @gpu
-@pytest.mark.parametrize("S,H,G,D,window", [(32, 16, 4, 128, 1024), (3, 8, 2, 64, 500), (40, 4, 4, 32, 0), (150, 8, 1, 48, 200), (1, 32, 8, 128, 0)])
+@pytest.mark.parametrize("S,H,G,D,window", [(32, 16, 4, 128, 1024), (3, 8, 2, 64, 500), (40, 4, 4, 32, 0), (150, 8, 1, 56, 200), (1, 32, 8, 128, 0)])
 def test_mixed_heads_decode_steps_without_sink_and_slopes(S, H, G, D, window):
     """many sequences, one decoded token each at contexts around page borders: the cluster of CTAs per query (how many depends
     on the batch) gives what the span kernel gives; neither sink nor distance bias"""
@@ -746,7 +746,7 @@ def test_mixed_batches_and_reused_slots_and_pages(tmp_path, dtype, experts):
 
 @gpu
 def test_long_decoding_single_tokens(tmp_path):
-    cfg = make_cfg([att(heads=4, kv=2, dim=32, window=100, mlp=moe(experts=4, ff=32, top=2)), att(heads=8, kv=2, dim=48, window=64),
+    cfg = make_cfg([att(heads=4, kv=2, dim=32, window=100, mlp=moe(experts=4, ff=32, top=2)), att(heads=8, kv=4, dim=56, window=64),
                     att(heads=2, kv=2, dim=16, window=130, mlp=dense(64))])
     t = make_tensors(cfg, seed=31)
     tokens = toks(260, cfg["vocab"], 9)
