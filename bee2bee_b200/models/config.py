@@ -84,7 +84,16 @@ class LayerSpec:
     ``[heads, heads]`` matrix mixes the heads' scores in front of the softmax); ``sink_one`` (a sink whose score is 0).
     ``ff_act`` = "poly_norm": dense feed-forward without a gate whose activation is a weighted sum of the RMS-normed first
     three powers and a constant.  ``route_kind`` = "sigmoid_topk": the ``top`` largest sigmoid scores, used as they are;
-    ``scale_input``: an expert's weight multiplies its input instead of its output."""
+    ``scale_input``: an expert's weight multiplies its input instead of its output.
+    ``mixer`` = "diff_attention": two softmax maps per head over the same values, ``a_1 - lambda a_2`` with one learned number
+    ``lambda`` per layer (``diff`` is its constant part), divided by its root mean square over the head and multiplied by ``1 -
+    diff``; q, k and v pass short convolutions of ``conv`` taps; queries and keys have ``2 * dim`` channels per head;
+    ``kv_from`` >= 0: keys and values are those of that earlier layer, the layer has none of its own.
+    ``mixer`` = "mamba2": state-space recurrence with one decay per head and token, ``S <- exp(-exp(A) dt) S + dt B x^T``, read with
+    C (``dim`` = state channels, ``kv_heads`` = groups that share B and C), behind a short convolution; the gated output is
+    RMS-normed in ``norm_groups`` parts.  ``mixer`` = "retention": linear attention with a constant ``decay`` per head.
+    ``ff_act`` = "relu_sq" with ``ff_kind`` "moe": experts without a gate; ``router_bias``: the router logits have a bias;
+    ``shared_gate``: the shared expert is multiplied by a sigmoid gate, one number per token."""
     mixer: str = "attention"
     heads: int = 1
     kv_heads: int = 1
@@ -127,6 +136,12 @@ class LayerSpec:
     sink_one: bool = False
     ff_act: str = ""
     scale_input: bool = False
+    diff: float = 0.0                # diff_attention: constant part of the second map's weight
+    kv_from: int = -1                # diff_attention: layer whose keys and values are used, -1 = the layer's own
+    norm_groups: int = 1             # mamba2: parts of the gated output that are normed on their own
+    decay: Tuple[float, ...] = ()    # retention: decay of every head
+    router_bias: bool = False
+    shared_gate: bool = False
 
     @property
     def head_slopes(self) -> Tuple[float, ...]:
@@ -141,7 +156,7 @@ class LayerSpec:
 @dataclass
 class ModelConfig:
     name: str = "tiny-llama"
-    family: str = "llama"            # gpt2 | llama | mistral | gemma2 | kepovik | repudra | lonulix | fisopel | kazolorn
+    family: str = "llama"            # gpt2 | llama | mistral | gemma2 | kepovik | repudra | lonulix | fisopel | kazolorn | nipudra
     vocab_size: int = 512
     hidden_size: int = 256
     n_layers: int = 2
@@ -175,7 +190,8 @@ class ModelConfig:
     pair_mul_prev: int = 0
     pair_mul_cur: int = 0
     block_layout: str = "sequential"  # sequential: norm -> mixer -> join, norm -> ff -> join; parallel: one norm feeds both;
-    #                                   post_norm: x <- norm(skip_scale * x + sublayer(x)), no norm in front of a sublayer
+    #                                   post_norm: x <- norm(skip_scale * x + sublayer(x)), no norm in front of a sublayer;
+    #                                   sandwich: x <- x + norm_b(sublayer(norm_a(x))), mixer then feed-forward
     norm_groups: int = 1             # post_norm: the RMS norm is taken over this many consecutive parts of the width
     skip_scale: float = 1.0          # post_norm: the residual is multiplied by this before the sublayer result is added
     gated_residual: bool = False     # post_norm: sublayer results are multiplied by sigmoid(W x + b) before the sum
@@ -190,6 +206,9 @@ class ModelConfig:
     loop_in: bool = False
     depth_average: bool = False      # parallel blocks: what leaves a layer is a learned weighted sum of its result, all earlier
     #                                  layers' results and the embedding output
+    token_side: int = 0              # sandwich: every layer adds norm(W_p (gelu(W_g x) * e)) with e = this many channels that the token
+    #                                  has for the layer in a table of its own
+    logit_scale: float = 1.0         # the logits are multiplied by this (before a soft cap)
 
     # ------------------------------------------------------------------ derived
     @property
@@ -199,7 +218,7 @@ class ModelConfig:
     @property
     def recurrent(self) -> bool:
         """True when some layer keeps per-sequence state besides the paged KV cache (no prefix sharing, no piece split)."""
-        return any(leaf.mixer not in ("attention", "softmax_attention", "latent_attention")
+        return any(leaf.mixer not in ("attention", "softmax_attention", "latent_attention")      # (diff_attention: its convolutions)
                    for sp in self.layer_specs for leaf in sp.leaves) \
             or self.pair_buckets > 0
 
@@ -603,7 +622,123 @@ class ModelConfig:
                 "width": self.hidden_size}
 
     @staticmethod
+    def from_nipudra_dict(d: Dict, name: str = "") -> "ModelConfig":
+        """``config.json`` of a Nipudra checkpoint: ``layers`` lists {type, mixer sizes, mlp | null}; types ``attention``
+        (differential, windowed, short convolutions, optionally the keys and values of an earlier layer), ``mamba2`` and
+        ``retention``; ``mlp.kind`` ``moe`` (squared-relu experts, optionally beside a gated shared one)."""
+        who = name or "nipudra"
+        specs: List[LayerSpec] = []
+
+        def rotary(m: Dict, dim: int) -> Optional[RotarySpec]:
+            r = m.get("rot")
+            if not r or not int(r.get("dims", 0)):
+                return None
+            sc = r.get("scaling") or {}
+            rot = RotarySpec(dims=int(r["dims"]), base=float(r["base"]), factor=float(sc.get("factor", 0.0)),
+                             original=int(sc.get("original", 0)), fast=float(sc.get("fast", 32.0)),
+                             slow=float(sc.get("slow", 1.0)), half=True)
+            if rot.dims % 2 or rot.dims > dim:
+                raise ValueError(f"{who}: rotary dims {rot.dims} do not fit a head of {dim} channels")
+            return rot
+
+        for l, lay in enumerate(d["layers"]):
+            m, mlp, kind = lay.get("mixer") or {}, lay.get("mlp"), lay["type"]
+            heads = int(m["heads"])
+            if kind == "attention":
+                dim = int(m["dim"])
+                sp = LayerSpec(mixer="diff_attention", heads=heads, kv_heads=int(m.get("kv_heads", heads)), dim=dim,
+                               vdim=int(m.get("vdim", dim)), scale=float(m.get("scale", dim ** -0.5)),
+                               window=int((m.get("mask") or {}).get("size", 0) or 0), rot=rotary(m, dim), qk_norm="none",
+                               v_norm=False, proj_bias=True, conv=int(m.get("conv", 1)), diff=float(m["diff"]),
+                               kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else -1)
+                if sp.heads % sp.kv_heads:
+                    raise ValueError(f"{who}: {sp.heads} heads cannot share {sp.kv_heads} key heads")
+                if sp.kv_from >= 0:
+                    src = specs[sp.kv_from] if sp.kv_from < l else None
+                    if src is None or src.mixer != "diff_attention" or src.kv_from >= 0 or \
+                            (src.kv_heads, src.dim, src.vdim, src.rot) != (sp.kv_heads, sp.dim, sp.vdim, sp.rot):
+                        raise ValueError(f"{who}: layer {l} cannot use the keys and values of layer {sp.kv_from}")
+            elif kind == "mamba2":
+                groups = int(m.get("groups", 1))
+                sp = LayerSpec(mixer=kind, heads=heads, kv_heads=groups, dim=int(m["state"]), vdim=int(m["vdim"]),
+                               conv=int(m.get("conv", 1)), norm_groups=int(m.get("norm_groups", 1)))
+                if heads % groups or (heads * sp.vdim) % sp.norm_groups:
+                    raise ValueError(f"{who}: {heads} heads of {sp.vdim} channels do not form {groups} groups and "
+                                     f"{sp.norm_groups} norm groups")
+            elif kind == "retention":
+                dim = int(m["dim"])
+                sp = LayerSpec(mixer=kind, heads=heads, kv_heads=heads, dim=dim, vdim=int(m.get("vdim", dim)),
+                               rot=rotary(m, dim), decay=tuple(float(v) for v in m["decay"]))
+                if len(sp.decay) != heads:
+                    raise ValueError(f"{who}: {len(sp.decay)} decays for {heads} heads")
+            else:
+                raise ValueError(f"{who}: unknown layer type {kind!r}")
+            if mlp:
+                if mlp.get("kind", "moe") != "moe":
+                    raise ValueError(f"{who}: feed-forward kind {mlp.get('kind')!r} is not implemented")
+                r = mlp["router"]
+                sp.ff_kind, sp.expert_ff, sp.experts, sp.top = "moe", int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"])
+                sp.route_kind, sp.ff_act, sp.router_bias = "logit_topk", "relu_sq", True
+                sp.shared_ff = int((mlp.get("shared") or {}).get("ff", 0))
+                sp.shared_gate = sp.shared_ff > 0
+                sp.ff = sp.experts * sp.expert_ff + sp.shared_ff
+                if not 0 < sp.top <= sp.experts:
+                    raise ValueError(f"{who}: {sp.top} of {sp.experts} experts cannot be chosen")
+            specs.append(sp)
+        att = [sp for sp in specs if sp.mixer == "diff_attention"] or specs
+        return ModelConfig(
+            name=name or "nipudra", family="nipudra", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+            n_layers=len(specs), n_heads=max(sp.heads for sp in att), n_kv_heads=max(sp.kv_heads for sp in att),
+            head_dim=max(2 * sp.dim if sp.mixer == "diff_attention" else sp.dim for sp in att),
+            ffn_size=max([sp.ff for sp in specs] + [0]), max_position=1 << 30, norm="ln",
+            norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)), act="relu_sq", glu=False, rope_theta=0.0,
+            tie_embeddings=True, embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+            final_softcap=float(d.get("logit_softcap") or 0.0), logit_scale=float(d.get("logit_scale", 1.0)),
+            layer_specs=tuple(specs), streams=0, block_layout="sandwich",
+            token_side=int((d.get("token_side") or {}).get("dim", 0)))
+
+    def to_nipudra_dict(self) -> Dict:
+        def rotary(rot: RotarySpec) -> Dict:
+            r = {"base": rot.base, "dims": rot.dims}
+            if rot.factor > 0:
+                r["scaling"] = {"factor": rot.factor, "fast": rot.fast, "original": rot.original, "slow": rot.slow}
+            return r
+
+        layers = []
+        for sp in self.layer_specs:
+            if sp.mixer == "diff_attention":
+                m = {"conv": sp.conv, "diff": sp.diff, "dim": sp.dim, "heads": sp.heads, "kv_heads": sp.kv_heads,
+                     "scale": sp.scale, "vdim": sp.vdim}
+                if sp.window:
+                    m["mask"] = {"size": sp.window}
+                if sp.kv_from >= 0:
+                    m["kv_from"] = sp.kv_from
+            elif sp.mixer == "mamba2":
+                m = {"conv": sp.conv, "groups": sp.kv_heads, "heads": sp.heads, "norm_groups": sp.norm_groups, "state": sp.dim,
+                     "vdim": sp.vdim}
+            else:
+                m = {"decay": list(sp.decay), "dim": sp.dim, "heads": sp.heads, "vdim": sp.vdim}
+            if sp.rot is not None:
+                m["rot"] = rotary(sp.rot)
+            mlp = None
+            if sp.ff:
+                mlp = {"expert": {"ff": sp.expert_ff}, "kind": "moe", "router": {"experts": sp.experts, "top": sp.top}}
+                if sp.shared_ff:
+                    mlp["shared"] = {"ff": sp.shared_ff}
+            layers.append({"type": "attention" if sp.mixer == "diff_attention" else sp.mixer, "mixer": m, "mlp": mlp})
+        d = {"architecture": "Nipudra", "embedding": {"scale": self.embed_scale}, "layers": layers,
+             "logit_scale": self.logit_scale, "norm": {"eps": self.norm_eps}, "vocab": self.vocab_size,
+             "width": self.hidden_size}
+        if self.final_softcap > 0:
+            d["logit_softcap"] = self.final_softcap
+        if self.token_side:
+            d["token_side"] = {"dim": self.token_side}
+        return d
+
+    @staticmethod
     def from_hf_dict(d: Dict, name: str = "") -> "ModelConfig":
+        if str(d.get("architecture", "")).lower() == "nipudra":
+            return ModelConfig.from_nipudra_dict(d, name)
         if str(d.get("architecture", "")).lower() == "kazolorn":
             return ModelConfig.from_kazolorn_dict(d, name)
         if str(d.get("architecture", "")).lower() == "fisopel":
@@ -665,6 +800,8 @@ class ModelConfig:
             return self.to_fisopel_dict()
         if self.family == "kazolorn":
             return self.to_kazolorn_dict()
+        if self.family == "nipudra":
+            return self.to_nipudra_dict()
         if self.family == "gpt2":
             return {"model_type": "gpt2", "architectures": ["GPT2LMHeadModel"], "vocab_size": self.vocab_size,
                     "n_embd": self.hidden_size, "n_layer": self.n_layers, "n_head": self.n_heads,
@@ -891,6 +1028,46 @@ def _kazolorn(name, width, vocab, layers):
 # heads with keys of their own and no feed-forward, experts again
 PRESETS["tiny-kazolorn"] = _kazolorn("tiny-kazolorn", 128, 512, [
     (4, 2, 32, 40, 192), (4, 1, 16, 72, (5, 32, 2)), (2, 2, 32, 100, 0), (6, 3, 16, 40, (4, 48, 1))])
+
+
+def _nipudra(name, width, vocab, layers, side=16, softcap=20.0, logit_scale=0.5):
+    """layers: ("attention", H, G, dim, vdim, window, conv, kv_from, mlp) | ("mamba2", H, vdim, state, groups, conv, mlp) |
+    ("retention", H, dim, vdim, mlp); mlp: 0 (none) | (experts, expert_ff, top, shared_ff)"""
+    specs = []
+    for lay in layers:
+        mlp = lay[-1]
+        if lay[0] == "attention":
+            _, h, g, d, v, win, conv, src, _ = lay
+            rot = RotarySpec(dims=d // 2 // 2 * 2, base=20000.0, factor=4.0, original=256, half=True)
+            sp = LayerSpec(mixer="diff_attention", heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, window=win, rot=rot,
+                           qk_norm="none", v_norm=False, proj_bias=True, conv=conv, diff=0.4, kv_from=src)
+        elif lay[0] == "mamba2":
+            _, h, v, n, g, conv, _ = lay
+            sp = LayerSpec(mixer="mamba2", heads=h, kv_heads=g, dim=n, vdim=v, conv=conv, norm_groups=g)
+        else:
+            _, h, d, v, _ = lay
+            sp = LayerSpec(mixer="retention", heads=h, kv_heads=h, dim=d, vdim=v, rot=RotarySpec(dims=d, base=10000.0, half=True),
+                           decay=tuple(1.0 - 2.0 ** (-5.0 - 3.0 * i / max(1, h - 1)) for i in range(h)))
+        if mlp:
+            e, eff, top, sh = mlp
+            sp.ff_kind, sp.experts, sp.expert_ff, sp.top, sp.shared_ff = "moe", e, eff, top, sh
+            sp.route_kind, sp.ff_act, sp.router_bias, sp.shared_gate, sp.ff = "logit_topk", "relu_sq", True, sh > 0, e * eff + sh
+        specs.append(sp)
+    att = [sp for sp in specs if sp.mixer == "diff_attention"] or specs
+    return ModelConfig(name=name, family="nipudra", vocab_size=vocab, hidden_size=width, n_layers=len(specs),
+                       n_heads=max(sp.heads for sp in att), n_kv_heads=max(sp.kv_heads for sp in att),
+                       head_dim=max(2 * sp.dim if sp.mixer == "diff_attention" else sp.dim for sp in att),
+                       ffn_size=max(sp.ff for sp in specs), max_position=1 << 30, norm="ln", norm_eps=1e-5, act="relu_sq", glu=False,
+                       rope_theta=0.0, tie_embeddings=True, embed_scale=width ** 0.5, final_softcap=softcap,
+                       logit_scale=logit_scale, layer_specs=tuple(specs), block_layout="sandwich", token_side=side,
+                       eos_token_id=-1, bos_token_id=-1)
+
+
+# sandwich-norm hybrid test preset: differential attention, mamba2, retention without a feed-forward, differential attention over
+# the first layer's keys and values with a window of its own
+PRESETS["tiny-nipudra"] = _nipudra("tiny-nipudra", 128, 512, [
+    ("attention", 4, 2, 16, 24, 40, 3, -1, (6, 32, 2, 48)), ("mamba2", 4, 24, 32, 2, 4, (4, 48, 1, 0)), ("retention", 2, 32, 48, 0),
+    ("attention", 2, 2, 16, 24, 72, 2, 0, (5, 32, 2, 32))])
 PRESETS["tiny-gpt2"].vocab_size = 384
 PRESETS["tiny-gpt2"].eos_token_id = 1
 PRESETS["tiny-gpt2"].bos_token_id = 0

@@ -32,6 +32,14 @@ in front of the softmax, and a one in the denominator.  The score mix is served 
 is ONE dot product of a mixed query row over all key heads with the cached key row, so every head attends on its own.
 Feed-forward: PolyNorm, or gated silu experts chosen by sigmoid scores that multiply the expert's input.
 
+Family ``nipudra``: sandwich layers -- a layer norm in front of and behind each sublayer (``x <- x + n1b(mixer(n1 x))``, ``x <- x +
+n2b(ff(n2 x))``), then a contribution of the token itself (``x <- x + rms(W_p (gelu(W_g x) * e)) w`` with a row ``e`` of a
+per-layer token table), logits from the embedding table.  Mixers: differential attention (two softmax maps per head over the same
+values, combined with a learned weight; short convolutions on q, k and v, half-split rotary pairs with YaRN frequencies, a
+window; a layer may use an earlier layer's keys and values), a state-space recurrence with one decay per head and token
+(mamba2), retention (a constant decay per head, rotated q and k).  Feed-forward: squared-relu experts without a gate beside a
+shared expert with a sigmoid gate.
+
 Same interface as ``native.NativePiece`` (the runner drives both through ``forward(BatchMeta)``): a flat batch of spans
 (prompt portions of any length beside single decoded tokens), physical KV slots and block tables from the page allocator,
 logits for the rows named by ``last_idx``.  What is new here and lives next to the shared machinery:
@@ -81,6 +89,7 @@ class _Mix:
     join_norm: bool = False                  # its output is divided by its root mean square over the width first
     amp: float = 1.0                         # rotary amplitude
     w_uv: Optional[torch.Tensor] = None      # latent attention with an output gate: [heads, vdim, kv_rank] value up-projections
+    lam: float = 0.0                         # differential attention: weight of the second map
 
 
 @dataclass
@@ -98,6 +107,9 @@ class _Layer:
     b_cat: Optional[torch.Tensor] = None   # bias of the fused projection (padded to its rows)
     mix: tuple = ()                     # parallel blocks: the mixers that read the layer's input side by side
     act_params: tuple = (0.0, 0.0)      # xIELU: softplus(p), 1/2 + softplus(q)
+    b_up: Optional[torch.Tensor] = None    # bias of the stacked up-projection (router rows)
+    w_side: Optional[torch.Tensor] = None  # token contribution: gate and output matrices
+    w_side_out: Optional[torch.Tensor] = None
 
 
 # projections of each mixer kind that read the layer input, in the order they are stacked into the fused GEMM
@@ -148,7 +160,9 @@ class HybridPiece:
                            and os.environ.get("B2B_HYBRID_OVERLAP", "1") == "1")
         self._side = torch.cuda.Stream(device=dev) if self.overlap_ff else None
         self._side2 = torch.cuda.Stream(device=dev) if self.overlap_ff else None     # second mixer of a parallel pair
-        self.caps_logits = self.parallel_blocks and cfg.final_softcap > 0     # the piece applies the logit soft cap itself
+        self.sandwich = cfg.block_layout == "sandwich"
+        self.caps_logits = (self.parallel_blocks or self.sandwich) and cfg.final_softcap > 0   # the piece applies the soft cap itself
+        self.rot_tabs: Dict[tuple, tuple] = {}      # sandwich: rotary tables of a step, one per distinct set of frequencies
         self.L: Dict[int, _Layer] = {}
         for l in self.layers:
             sp, p = cfg.layer_specs[l], f"l{l}."
@@ -158,6 +172,9 @@ class HybridPiece:
                 continue
             if self.post_norm:
                 self.L[l] = self._build_post_norm_layer(L, l, tensors, mat, vec)
+                continue
+            if self.sandwich:
+                self.L[l] = self._build_sandwich_layer(L, l, tensors, mat, vec)
                 continue
             if sp.mixer == "attention":
                 L.w_cat = mat(p + "mix.q", p + "mix.k", p + "mix.v", p + "mix.g")
@@ -182,6 +199,10 @@ class HybridPiece:
         self.embed = tensors["embed"].to(device=dev, dtype=dtype).contiguous()
         self.pair = tensors["bigram"].to(device=dev, dtype=dtype).contiguous() if cfg.pair_buckets else None
         self.final_norm = vec("final.norm").reshape(-1)
+        if self.sandwich:            # the logit scale rides on the model norm (fp32) in front of the head matrix
+            self.final_norm = (self.final_norm * cfg.logit_scale).contiguous()
+            self.final_bias = (vec("final.norm.b") * cfg.logit_scale).contiguous()
+        self.side_embed = tensors["side.embed"].to(device=dev, dtype=dtype).contiguous() if cfg.token_side else None
         self.w_head = mat("embed" if cfg.tie_embeddings else "head")
         self.w_loop = mat("loop.in") if cfg.loop_in else None       # [x ; embedding output] -> the residual entering a pass
         self.runs = [r for r in cfg.layer_runs() if r[0] in self.L]  # (layer, pass, first of a pass) in execution order
@@ -198,7 +219,7 @@ class HybridPiece:
         self.conv_tail: Dict[str, torch.Tensor] = {}   # short convolutions: the last taps - 1 inputs [slots, taps - 1, channels]
         for l in self.layers:
             sp = cfg.layer_specs[l]
-            if self.parallel_blocks or self.post_norm:
+            if self.parallel_blocks or self.post_norm or self.sandwich:
                 for self._pass in sorted({p for ll, p, _ in self.runs if ll == l}):     # a cache / state per pass of a looped layer
                     for mx in self.L[l].mix:
                         self._alloc_mixer_state(mx, num_pages)
@@ -237,7 +258,7 @@ class HybridPiece:
         if self.w_loop is not None:
             yield self.w_loop
         for L in self.L.values():
-            for t in (L.w_cat, L.w_o, L.w2, L.w_up, L.w_down, L.w_glu):
+            for t in (L.w_cat, L.w_o, L.w2, L.w_up, L.w_down, L.w_glu, L.w_side, L.w_side_out):
                 if t is not None:
                     yield t
             for mx in L.mix:
@@ -248,6 +269,7 @@ class HybridPiece:
     def weight_bytes(self) -> int:
         n = sum(t.numel() * t.element_size() for t in self._matrices())
         n += self.w_head.numel() * self.w_head.element_size() + self.embed.numel() * self.embed.element_size()
+        n += self.side_embed.numel() * self.side_embed.element_size() if self.side_embed is not None else 0
         return n + (self.pair.numel() * self.pair.element_size() if self.pair is not None else 0)
 
     def streamed_weight_bytes(self) -> int:
@@ -259,6 +281,12 @@ class HybridPiece:
         return sum(s[0].numel() * 4 for d in (self.state, self.nstate, self.mstate, self.conv_tail) for s in d.values())
 
     def n_launches(self) -> int:
+        if self.sandwich:
+            per = {"diff_attention": 2, "mamba2": 4, "retention": 2}         # between the fused and the output projection (decode)
+            n = 3 + len(self.rot_tabs) + (1 if self.caps_logits else 0)      # embedding, first norm, (table, soft cap), commit
+            for L in self.L.values():
+                n += 3 + per[L.spec.mixer] + (5 if L.spec.ff else 0) + (4 if self.cfg.token_side else 0)
+            return n
         if self.post_norm:
             n = 3                                        # embedding, its operand copy, final norm (head GEMM: the runner)
             for L in self.L.values():
@@ -295,6 +323,8 @@ class HybridPiece:
             return self._forward_parallel_blocks(m)
         if self.post_norm:
             return self._forward_post_norm(m)
+        if self.sandwich:
+            return self._forward_sandwich(m)
         ops.hyb_embed(m.ids, m.positions, m.q_start, m.q_len, seq_slot, self.prev_tok, self.embed, self.pair,
                       c.pair_buckets, c.pair_mul_prev, c.pair_mul_cur, st, S, mq)
         h = self.h[:T]
@@ -457,7 +487,7 @@ class HybridPiece:
         return rows
 
     def _build_routed_ff(self, L: _Layer, p: str, tensors: Tensors) -> None:
-        """Gated experts chosen by their router logits, beside a shared expert: ONE up matrix ``[router | gate rows of
+        """Experts chosen by their router logits, beside a shared expert: ONE up matrix ``[router | gate rows of
         the shared expert and of every expert | their up rows]`` and ONE down matrix with the down-projections side by
         side, so a token's weighted expert sum is a column scaling between two GEMMs (no sorting, no host)."""
         sp, dev, f64 = L.spec, self.device, torch.float64
@@ -468,6 +498,20 @@ class HybridPiece:
             return tensors[n].to(device=dev, dtype=f64)
 
         router = t64(p + "mlp.router")
+        if not sp.expert_gated:          # [router | gate of the shared expert | up rows], no gate rows
+            if sp.shared_gate:
+                router = torch.cat([router, t64(p + "mlp.shared.sg")], 0)
+            pad = router.new_zeros(((-router.shape[0]) % 4, W))
+            ups = torch.cat([t64(f"{p}mlp.{n}.up") for n in names], 0)
+            n_r = router.shape[0] + pad.shape[0]
+            L.ff_off = {"router": 0, "sg": sp.experts if sp.shared_gate else -1, "up": n_r, "hidden": ups.shape[0]}
+            L.w_up = ops.pad_weight(torch.cat([router, pad, ups], 0).to(torch.float32), 128, 64).to(self.dtype).contiguous()
+            if sp.router_bias:
+                L.b_up = torch.zeros(L.w_up.shape[0], device=dev)
+                L.b_up[:sp.experts] = tensors[p + "mlp.router.b"].to(device=dev, dtype=torch.float32)
+            down = torch.cat([t64(f"{p}mlp.{n}.down") for n in names], 1)
+            L.w_down = ops.pad_weight(down.to(torch.float32), 128, 64).to(self.dtype).contiguous()
+            return
         pad = router.new_zeros(((-router.shape[0]) % 4, W))          # the blocks behind it start at multiples of four
         gates = torch.cat([t64(f"{p}mlp.{n}.gate") for n in names], 0)
         ups = torch.cat([t64(f"{p}mlp.{n}.up") for n in names], 0)
@@ -480,6 +524,18 @@ class HybridPiece:
     def _alloc_mixer_state(self, mx: _Mix, num_pages: int) -> None:
         sp, dev, f32 = mx.spec, self.device, torch.float32
         key = self._key(mx)
+        if sp.mixer == "diff_attention":
+            if sp.kv_from < 0:
+                self.k_cache[key] = torch.zeros((num_pages, ops.PAGE, 2 * sp.kv_heads, sp.dim), device=dev, dtype=self.dtype)
+                self.v_cache[key] = torch.zeros((num_pages, ops.PAGE, sp.kv_heads, sp.vdim), device=dev, dtype=self.dtype)
+            else:                             # an earlier layer's cache, as it is
+                src = f"{sp.kv_from}.0"
+                self.k_cache[key], self.v_cache[key] = self.k_cache[src], self.v_cache[src]
+        if "conv" in mx.f:                    # the taps are the tensor's, whatever the config says
+            ch, taps = mx.f["conv"].shape
+            self.conv_tail[key] = torch.zeros((self.state_slots, max(1, taps - 1), ch), device=dev, dtype=f32)
+        if sp.mixer == "diff_attention":
+            return
         if sp.mixer == "latent_attention":      # one row per token: [rotated key part | latent]; the values are its latent slice
             self.k_cache[key] = torch.zeros((num_pages, ops.PAGE, 1, sp.rot_dim + sp.kv_rank), device=dev, dtype=self.dtype)
             self.v_cache[key] = self.k_cache[key][..., sp.rot_dim:]
@@ -493,9 +549,6 @@ class HybridPiece:
         if sp.mixer == "mlstm":
             self.nstate[key] = torch.zeros((self.state_slots, sp.heads, sp.dim), device=dev, dtype=f32)
             self.mstate[key] = torch.zeros((self.state_slots, sp.heads), device=dev, dtype=f32)
-        elif sp.mixer == "channel_delta":
-            ch, taps = mx.f["conv"].shape                 # the taps are the tensor's, whatever the config says
-            self.conv_tail[key] = torch.zeros((self.state_slots, max(1, taps - 1), ch), device=dev, dtype=f32)
 
     def _forward_parallel_blocks(self, m) -> torch.Tensor:
         """x = scale * embed;  per layer: h = norm(x), x += sum of the layer-scaled mixer / feed-forward outputs (all
@@ -753,11 +806,16 @@ class HybridPiece:
         their sigmoids (then on the expert's input): one GEMM (router logits, all gate rows, all up rows), the router, ``silu(gate) * up * weight`` per hidden column,
         one GEMM over the down-projections side by side"""
         sp, o, f32 = L.spec, L.ff_off, torch.float32
-        p2 = ops.linear(L.w_up, h, self._buf("proj2", f32, L.w_up.shape[0])[:T])
+        p2 = ops.linear(L.w_up, h, self._buf("proj2", f32, L.w_up.shape[0])[:T], bias=L.b_up)
         wt = self._buf("route", f32, max(1, sp.experts))[:T]
         idw = self._buf("keep", f32, 1)[:T]
-        ops.moe_route(p2, o["router"], None, sp.experts, 1, 1, sp.top, 1.0, wt, idw, T, sigmoid=sp.route_kind == "sigmoid_topk")
+        ops.moe_route(p2, o["router"], None, sp.experts, 1, 1, sp.top, 1.0, wt, idw, T, sigmoid=sp.route_kind == "sigmoid_topk",
+                      off_gate=o.get("sg", -1))
         hid = self._buf("ff", self.dtype, L.w_down.shape[1])[:T]
+        if not sp.expert_gated:          # squared relu times the expert's weight, the shared expert's gate in front
+            ops.gated_cols(p2, o["up"], 0, hid, o["hidden"], ops.GATE_RELU_SQ, T, wt=wt, per=sp.expert_ff, lead=sp.shared_ff,
+                           lead_w=idw if sp.shared_gate else None)
+            return ops.linear(L.w_down, hid, self._buf("yff", f32, L.w_down.shape[0])[:T])
         ops.gated_cols(p2, o["gate"], o["up"], hid, o["hidden"], ops.GATE_SILU, T, wt=wt, per=sp.expert_ff, both=True,
                        lead=sp.shared_ff, scale_input=sp.scale_input)
         return ops.linear(L.w_down, hid, self._buf("yff", f32, L.w_down.shape[0])[:T])
@@ -903,3 +961,174 @@ class HybridPiece:
         do = self._buf(f"mix{d}", self.dtype, L.w_o.shape[1])[:T]
         ops.delta_post(o, proj, 3 * d, L.f["norm"], do, T, H, D, c.norm_eps)
         return ops.linear(L.w_o, do, self._buf("y", torch.float32, L.w_o.shape[0])[:T])
+
+    # ================================================================== sandwich layers (a norm in front of and behind each sublayer)
+    def _rot_tab(self, rot) -> Optional[tuple]:
+        """key of the rotary table of these frequencies (computed once per step for all layers that turn by them)"""
+        if rot is None or rot.dims <= 0:
+            return None
+        key = (rot.dims, rot.base, rot.factor, rot.original, rot.fast, rot.slow)
+        if key not in self.rot_tabs:
+            hi, lo = ops.split_frequencies(rot.frequencies(), self.device)
+            tab = torch.zeros((self.max_tokens, rot.dims), device=self.device, dtype=torch.float32)
+            self.rot_tabs[key] = (hi, lo, rot.amplitude, tab)
+        return key
+
+    def _build_sandwich_layer(self, L: _Layer, l: int, tensors: Tensors, mat, vec) -> _Layer:
+        """Layer ``l`` of a sandwich-norm model; the input projections of its mixer are ONE matrix.  Differential attention: the
+        query rows of a key/value head are reordered to (map, head), so that the heads which read the same key map are
+        neighbours and the attention kernels see twice the heads over twice the key heads.  Retention: rotary pairs stored
+        half-split (i with i + dims / 2) become neighbours on the query and key rows alike."""
+        sp, p, dev = L.spec, f"l{l}.", self.device
+        q, W = p + "mix.", self.cfg.hidden_size
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if sp.ff else ()):
+            L.f[n], L.f[n + ".b"] = vec(p + n), vec(p + n + ".b")
+        mx = _Mix(spec=sp, key=f"{l}.0", idx=0)
+        H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
+
+        def rows(n):
+            return tensors[n].to(device=dev, dtype=torch.float64)
+
+        def stack(ws):
+            return ops.pad_weight(torch.cat(ws, 0).to(torch.float32), 128, 64).to(self.dtype).contiguous()
+
+        mx.w_o = mat(q + "o")
+        if sp.mixer == "diff_attention":
+            order = torch.arange(2 * H * D, device=dev).view(G, H // G, 2, D).transpose(1, 2).reshape(-1)
+            parts = {"q": order}
+            if sp.kv_from < 0:
+                parts.update({"k": slice(None), "v": slice(None)})
+            L.w_cat = stack([rows(q + n)[i] for n, i in parts.items()])
+            bias = torch.cat([vec(q + n + ".b")[i] for n, i in parts.items()])
+            L.b_cat = torch.zeros(L.w_cat.shape[0], device=dev)
+            L.b_cat[:bias.numel()] = bias
+            mx.f["conv"] = torch.cat([vec(q + n + ".conv")[i] for n, i in parts.items()], 0).contiguous()
+            mx.b_o = torch.zeros(mx.w_o.shape[0], device=dev)
+            mx.b_o[:W] = vec(q + "o.b")
+            t = {n: rows(q + n) for n in ("lq1", "lk1", "lq2", "lk2")}
+            mx.lam = float(torch.exp((t["lq1"] * t["lk1"]).sum()) - torch.exp((t["lq2"] * t["lk2"]).sum())) + sp.diff
+            mx.rank = 2 * D * (H + (G if sp.kv_from < 0 else 0)) + (G * V if sp.kv_from < 0 else 0)
+        elif sp.mixer == "mamba2":
+            inner, gn = H * V, G * D
+            L.w_cat = stack([rows(q + "in")])
+            mx.off.update({"z": 0, "xbc": inner, "dt": 2 * inner + 2 * gn})
+            mx.f["conv"] = vec(q + "conv")
+            for n in ("conv.b", "dt_bias", "A_log", "D", "norm"):
+                mx.f[n] = vec(q + n)
+        elif sp.mixer == "retention":
+            perm = torch.arange(D, device=dev)
+            if sp.rot is not None and sp.rot.half:
+                rd = sp.rot.dims
+                perm[:rd] = torch.arange(rd, device=dev).view(2, rd // 2).t().reshape(-1)       # new 2i <- i, new 2i+1 <- i + rd/2
+            turned = [rows(q + n).view(H, D, W)[:, perm].reshape(H * D, W) for n in ("q", "k")]
+            L.w_cat = stack(turned + [rows(q + "v"), rows(q + "g")])
+            mx.off.update({"q": 0, "k": H * D, "v": 2 * H * D, "g": 2 * H * D + H * V})
+            mx.f["decay"] = torch.tensor(sp.decay, dtype=torch.float64).to(device=dev, dtype=torch.float32)
+            mx.f["norm"] = torch.ones(V, device=dev)                     # the heads' outputs are normed without a weight
+        else:
+            raise ValueError(f"{self.cfg.name}: layer {l} has mixer {sp.mixer!r}, which sandwich layers do not have")
+        self._rot_tab(sp.rot)
+        L.mix = (mx,)
+        if sp.ff:
+            self._build_routed_ff(L, p, tensors)
+        if self.cfg.token_side:
+            L.w_side, L.w_side_out = mat(p + "side.gate"), mat(p + "side.proj")
+            L.f["side"] = vec(p + "side.norm")
+        return L
+
+    def _forward_sandwich(self, m) -> torch.Tensor:
+        """x = scale * embed;  per layer x += n1b(mixer(n1 x)), x += n2b(ff(n2 x)), x += rms(W_p (gelu(W_g x) * e)) w;  logits =
+        cap(scale * head(norm(x))).  The norm behind a sublayer, the join and the norm in front of the next one are one kernel."""
+        c = self.cfg
+        T, S, mq, eps = m.n_tokens, m.n_seqs, m.max_q, c.norm_eps
+        W, f32 = c.hidden_size, torch.float32
+        x = self.streams[:T].view(T, W)
+        ops.hyb_embed(m.ids, m.positions, m.q_start, m.q_len, m.seq_slot, self.prev_tok, self.embed, None, 0, 0, 0,
+                      self.streams[:T], S, mq, scale=c.embed_scale)
+        for hi, lo, amp, tab in self.rot_tabs.values():
+            ops.rot_table(m.positions, hi, lo, amp, tab, T)
+        h = self.h[:T]
+        pend: dict = {}                  # (y, norm_y, kind_y) of the sublayer whose result has not joined the residual yet
+
+        def join(norm_h=None, **kw):
+            ops.sandwich_join(x, eps=eps, h=h, norm_h=norm_h, kind_h=ops.NORM_LAYER if norm_h is not None else ops.NORM_NONE, **pend, **kw)
+
+        for l in self.layers:
+            L = self.L[l]
+            mx, f = L.mix[0], L.f
+            join((f["norm1"], f["norm1.b"]))
+            proj = ops.linear(L.w_cat, h, self._buf("proj", f32, L.w_cat.shape[0])[:T], bias=L.b_cat)
+            y = getattr(self, "_mix_" + mx.spec.mixer)(mx, proj, m, self._buf("y0", f32, mx.w_o.shape[0])[:T])
+            pend = dict(y=y, norm_y=(f["norm1b"], f["norm1b.b"]))
+            if L.spec.ff:
+                join((f["norm2"], f["norm2.b"]))
+                pend = dict(y=self._ff_routed(L, h, T), norm_y=(f["norm2b"], f["norm2b.b"]))
+            if c.token_side:
+                join()                   # h: the residual itself as the operand
+                z = ops.linear(L.w_side, h, self._buf("side", f32, L.w_side.shape[0])[:T])
+                g = self._buf(f"sideg{c.token_side}", self.dtype, L.w_side_out.shape[1])[:T]
+                ops.side_gate(z, m.ids, self.side_embed, l * c.token_side, g, c.token_side, T)
+                y = ops.linear(L.w_side_out, g, self._buf("yside", f32, L.w_side_out.shape[0])[:T])
+                pend = dict(y=y, norm_y=(f["side"], None), kind_y=ops.NORM_RMS)
+            if self.debug_layers is not None:
+                self.debug_layers.append(self._debug_sandwich(x, pend, T))
+        R = m.n_out or S
+        rows = m.last_idx if m.last_idx is not None else m.q_start
+        xl = self.last_x[:R]
+        ops.sandwich_join(x, eps=eps, h=xl, norm_h=(self.final_norm, self.final_bias), rows=rows, n_rows=R, **pend)
+        logits = ops.linear(self.w_head, xl, self.logits[:R])
+        if self.caps_logits:
+            ops.act_cols(logits, 0, logits, logits.shape[1], ops.COLS_SOFTCAP, R, p0=c.final_softcap)
+        return logits
+
+    def _debug_sandwich(self, x: torch.Tensor, pend: dict, T: int) -> torch.Tensor:
+        """the residual after the pending result has joined it (plain torch, tests only)"""
+        W, eps = self.cfg.hidden_size, self.cfg.norm_eps
+        y, (w, b) = pend["y"][:T, :W], pend["norm_y"]
+        if pend.get("kind_y", ops.NORM_LAYER) == ops.NORM_LAYER:
+            y = y - y.mean(-1, keepdim=True)
+        y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * w
+        return x[:T] + (y + b if b is not None else y)
+
+    def _mix_diff_attention(self, mx: _Mix, proj: torch.Tensor, m, y: torch.Tensor) -> torch.Tensor:
+        sp, T = mx.spec, m.n_tokens
+        H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
+        key = self._key(mx)
+        kc, vc = self.k_cache[key], self.v_cache[key]
+        own = sp.kv_from < 0
+        tk = self._rot_tab(sp.rot)
+        q = self._buf(f"q{mx.idx}", torch.float32, 2 * H * D)[:T]
+        ops.conv_rot_prep(proj, 0, mx.f["conv"], self.conv_tail[key], self.rot_tabs[tk][3] if tk else None, sp.scale, m.slots, q,
+                          kc if own else None, vc if own else None, m.q_start, m.q_len, m.kv_len, m.seq_slot, m.n_seqs, m.max_q,
+                          2 * H, 2 * G if own else 0, G if own else 0, D, V)
+        ao = self._buf(f"mix{mx.idx}.{H * V}", self.dtype, mx.w_o.shape[1])[:T]
+        maps = self._buf(f"maps{mx.idx}", torch.float32, 2 * H * V)[:T]
+        ops.softmax_attention(q, kc, vc, maps, m.block_table, m.q_start, m.q_len, m.kv_len, m.n_seqs, m.max_q, 2 * H, 2 * G, D, V,
+                              sp.window, 1.0, v_heads=G)
+        ops.diff_combine(maps, mx.lam, 1.0 - sp.diff, ao, T, H, G, V, self.cfg.norm_eps)
+        return ops.linear(mx.w_o, ao, y, bias=mx.b_o)
+
+    def _mix_mamba2(self, mx: _Mix, proj: torch.Tensor, m, y: torch.Tensor) -> torch.Tensor:
+        sp, T = mx.spec, m.n_tokens
+        H, G, N, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
+        key, inner = self._key(mx), H * V
+        cw = mx.f["conv"]
+        xbc = self._buf(f"conv{mx.idx}", torch.float32, ops.pad_to(cw.shape[0], 4))[:T]
+        ops.short_conv(proj, mx.off["xbc"], cw, self.conv_tail[key], xbc, m.q_start, m.q_len, m.kv_len, m.seq_slot, m.n_seqs, m.max_q,
+                       bias=mx.f["conv.b"])
+        o = self._buf(f"o{mx.idx}", torch.float32, inner)[:T]
+        ops.lin_scan(ops.SCAN_SSD, xbc, inner + G * N, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len, m.seq_slot,
+                     m.n_seqs, m.max_q, H, G, N, V, zbias=mx.f["dt_bias"], hparam=mx.f["A_log"], beta=proj, off_b=mx.off["dt"])
+        go = self._buf(f"mix{mx.idx}.{inner}", self.dtype, mx.w_o.shape[1])[:T]
+        ops.ssd_post(o, xbc, 0, proj, mx.off["z"], mx.f["D"], mx.f["norm"], go, T, H, V, sp.norm_groups, self.cfg.norm_eps)
+        return ops.linear(mx.w_o, go, y)
+
+    def _mix_retention(self, mx: _Mix, proj: torch.Tensor, m, y: torch.Tensor) -> torch.Tensor:
+        sp, T = mx.spec, m.n_tokens
+        H, D, V = sp.heads, sp.dim, sp.vdim
+        tk = self._rot_tab(sp.rot)
+        o = self._buf(f"o{mx.idx}", torch.float32, H * V)[:T]
+        ops.lin_scan(ops.SCAN_RETENTION, proj, mx.off["q"], mx.off["k"], proj, mx.off["v"], self.state[self._key(mx)], o, m.q_start,
+                     m.q_len, m.kv_len, m.seq_slot, m.n_seqs, m.max_q, H, H, D, V, z=self.rot_tabs[tk][3] if tk else None,
+                     hparam=mx.f["decay"], qscale=D ** -0.5, rdims=sp.rot.dims if tk else 0)
+        return self._scan_out(mx, o, proj, mx.off["g"], ops.POST_SILU, None, m, y)

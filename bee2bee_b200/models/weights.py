@@ -249,10 +249,60 @@ def kazolorn_tensor_specs(cfg: ModelConfig, layers: Iterable[int], first: bool, 
     return specs
 
 
+def nipudra_tensor_specs(cfg: ModelConfig, layers: Iterable[int], first: bool, last: bool):
+    """(checkpoint name, shape, kind) of a Nipudra model; matrices are kept as [out, in].  Layer norms have a weight and a bias
+    (``.b``); the logits come from the embedding table; every layer has its share of the per-token table ``side.embed``."""
+    W = cfg.hidden_size
+    specs = [("embed", (cfg.vocab_size, W), "w")] if (first or last) else []
+    if first and cfg.token_side:
+        specs.append(("side.embed", (cfg.vocab_size, cfg.n_layers * cfg.token_side), "w"))
+
+    def norm(n):
+        return [(n, (W,), "one"), (n + ".b", (W,), "bias")]
+
+    for l in layers:
+        sp, p = cfg.layer_specs[l], f"l{l}."
+        m = p + "mix."
+        specs += norm(p + "norm1") + norm(p + "norm1b")
+        H, G, D, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
+        if sp.mixer == "diff_attention":
+            rows = {"q": 2 * H * D}
+            if sp.kv_from < 0:
+                rows.update({"k": 2 * G * D, "v": G * V})
+            for n, r in rows.items():
+                specs += [(m + n, (r, W), "w"), (m + n + ".b", (r,), "bias"), (m + n + ".conv", (r, sp.conv), "conv")]
+            specs += [(m + n, (D,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")]
+            specs += [(m + "o", (W, H * V), "w"), (m + "o.b", (W,), "bias")]
+        elif sp.mixer == "mamba2":
+            inner, ch = H * V, H * V + 2 * G * D
+            specs += [(m + "in", (inner + ch + H, W), "w"), (m + "conv", (ch, sp.conv), "conv"), (m + "conv.b", (ch,), "bias"),
+                      (m + "dt_bias", (H,), "bias"), (m + "A_log", (H,), "neg"), (m + "D", (H,), "one"),
+                      (m + "norm", (inner,), "one"), (m + "o", (W, inner), "w")]
+        elif sp.mixer == "retention":
+            specs += [(m + "q", (H * D, W), "w"), (m + "k", (H * D, W), "w"), (m + "v", (H * V, W), "w"), (m + "g", (H * V, W), "w"),
+                      (m + "o", (W, H * V), "w")]
+        else:
+            raise ValueError(f"{cfg.name}: layer {l} has mixer {sp.mixer!r}, which is not part of this family")
+        if sp.ff:
+            specs += norm(p + "norm2") + norm(p + "norm2b")
+            for n in [f"e{e}" for e in range(sp.experts)] + (["shared"] if sp.shared_ff else []):
+                f = sp.shared_ff if n == "shared" else sp.expert_ff
+                specs += [(f"{p}mlp.{n}.up", (f, W), "w"), (f"{p}mlp.{n}.down", (W, f), "w")]
+            specs += [(p + "mlp.router", (sp.experts, W), "w"), (p + "mlp.router.b", (sp.experts,), "bias")]
+            if sp.shared_ff:
+                specs.append((p + "mlp.shared.sg", (1, W), "w"))
+        if cfg.token_side:
+            specs += [(p + "side.gate", (cfg.token_side, W), "w"), (p + "side.proj", (W, cfg.token_side), "w"),
+                      (p + "side.norm", (W,), "small")]
+    if last:
+        specs += norm("final.norm")
+    return specs
+
+
 def hybrid_tensor_specs(cfg: ModelConfig, layers: Iterable[int], first: bool, last: bool):
     """tensor list of a hybrid family (configs with per-layer mixer specs)"""
     fn = {"repudra": repudra_tensor_specs, "lonulix": lonulix_tensor_specs,
-          "fisopel": fisopel_tensor_specs, "kazolorn": kazolorn_tensor_specs}.get(cfg.family, kepovik_tensor_specs)
+          "fisopel": fisopel_tensor_specs, "kazolorn": kazolorn_tensor_specs, "nipudra": nipudra_tensor_specs}.get(cfg.family, kepovik_tensor_specs)
     return fn(cfg, layers, first, last)
 
 
@@ -260,8 +310,8 @@ def _init_random_hybrid(cfg: ModelConfig, layers, first, last, device, dtype, se
     t: Tensors = {}
     for name, shape, kind in hybrid_tensor_specs(cfg, layers, first, last):
         if kind == "w":
-            std = 1.0 if name in ("embed", "bigram") else shape[-1] ** -0.5
-            if cfg.family in ("repudra", "lonulix", "fisopel") and name == "embed":
+            std = 1.0 if name in ("embed", "bigram", "side.embed") else shape[-1] ** -0.5
+            if cfg.family in ("repudra", "lonulix", "fisopel", "nipudra") and name == "embed":
                 std = 1.0 / max(cfg.embed_scale, 1e-6)        # the scaled embedding has unit variance
             t[name] = _randn(name, shape, std, seed, device, dtype)
             continue

@@ -17,9 +17,10 @@ import torch
 EPI_PLAIN, EPI_RESIDUAL, EPI_GLU, EPI_QKV_ROPE, EPI_GELU = 0, 1, 2, 3, 4
 ACT_SILU, ACT_GELU, ACT_RELU_SQ, ACT_XIELU = 0, 1, 2, 3   # ``act_gelu`` of ``gemm``: GLU gate activation / EPI_GELU activation
 COLS_COPY, COLS_TANH, COLS_RELU_SQ, COLS_XIELU, COLS_SOFTCAP = 0, 1, 2, 3, 4     # ``act`` of ``act_cols``
-SCAN_GLA, SCAN_DELTA, SCAN_MLSTM, SCAN_HGRN2 = 0, 1, 2, 3     # ``mode`` of ``lin_scan``
+SCAN_GLA, SCAN_DELTA, SCAN_MLSTM, SCAN_HGRN2, SCAN_SSD, SCAN_RETENTION = 0, 1, 2, 3, 4, 5     # ``mode`` of ``lin_scan``
 POST_SIGMOID, POST_SILU, POST_NONE = 0, 1, 2     # ``act`` of ``scan_post``: the output gate
-GATE_SILU, GATE_GELU, GATE_GELU_TANH = 0, 1, 2   # ``act`` of ``gated_cols`` (GELU = the exact erf form)
+GATE_SILU, GATE_GELU, GATE_GELU_TANH, GATE_RELU_SQ = 0, 1, 2, 3   # ``act`` of ``gated_cols`` (GELU = the exact erf form)
+NORM_RMS, NORM_LAYER, NORM_NONE = 0, 1, 2        # norm kinds of ``sandwich_join``
 PAGE = 64           # tokens per KV page (csrc/attention.cu)
 NUM_SMS = 148
 
@@ -35,7 +36,8 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "set_decode_state", "hyb_embed", "hyb_commit_prev", "hc_step", "act_cols", "attn_prep",
                         "sig_attention", "delta_scan", "delta_post", "ls_join", "rot_attn_prep", "softmax_attention",
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
-                        "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention")
+                        "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention", "sandwich_join", "rot_table",
+                        "conv_rot_prep", "diff_combine", "ssd_post", "side_gate")
 
 
 class _CountedModule:
@@ -564,15 +566,16 @@ def softmax_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_
     """causal softmax attention over the paged cache; ``window`` > 0: the last ``window`` keys and the first ``keep_first``
     ones; ``softcap`` > 0: ``score <- softcap * tanh(score / softcap)``; ``sink`` [H]: ``exp(sink_h)`` joins the denominator;
     ``slopes`` [H]: ``score -= slopes[h] * (query position - key position)``; ``v_heads``: value heads per cache row when they
-    differ from the ``G`` key heads (head ``h`` reads value head ``h // (H / v_heads)``)"""
+    differ from the ``G`` key heads (head ``h`` reads value head ``h // (H / v_heads)``); ``out`` has the dtype of the cache or
+    float32"""
     native().softmax_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, V,
                                window, float(scale), float(softcap), int(keep_first), sink, int(v_heads), slopes)
 
 
-def short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q):
-    """y[t, c] = silu(causal convolution of columns off .. off + C of x with w [C, taps]); ``tail`` [slots, taps-1, C]
+def short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, bias=None, silu=True):
+    """y[t, c] = silu(causal convolution of columns off .. off + C of x with w [C, taps] + bias[c]); ``tail`` [slots, taps-1, C]
     holds the inputs before the span and receives the last ones (a second kernel, after the first has read them)"""
-    native().short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q)
+    native().short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, bias, int(bool(silu)))
     if w.shape[1] > 1:
         LAUNCHES[0] += 1
 
@@ -584,11 +587,11 @@ def mlstm_gates(proj, off_q, off_k, off_i, off_f, bi, bf, cap, qscale, nstate, m
 
 
 def lin_scan(mode, qk, off_q, off_k, v, off_v, state, out, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, H, G, dk, dv, *,
-             z=None, off_z=0, zbias=None, hparam=None, beta=None, off_b=0, aux=None, qscale=1.0, inv_tau=1.0):
-    """Gated linear recurrence over the spans (``mode`` = SCAN_GLA / SCAN_DELTA / SCAN_MLSTM); ``max_q`` = longest span
-    of the batch (1: the decode variant)."""
+             z=None, off_z=0, zbias=None, hparam=None, beta=None, off_b=0, aux=None, qscale=1.0, inv_tau=1.0, rdims=0):
+    """Gated linear recurrence over the spans (``mode`` = SCAN_*); ``max_q`` = longest span of the batch (1: the decode
+    variant).  SCAN_RETENTION: ``z`` is the rotary table of the step, the first ``rdims`` channels of q and k turn."""
     native().lin_scan(mode, qk, off_q, off_k, v, off_v, z, off_z, zbias, hparam, beta, off_b, aux, float(qscale),
-                      float(inv_tau), state, out, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, H, G, dk, dv)
+                      float(inv_tau), state, out, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, H, G, dk, dv, int(rdims))
 
 
 def scan_post(o, gate, off_g, weight, act, aux, out, T, H, dv, eps):
@@ -653,21 +656,66 @@ def poly_norm(x, off, w, out, n, eps, T):
     native().poly_norm(x, off, w, out, n, float(eps), T)
 
 
-def moe_route(proj, off, corr, n_real, count, keep, top, scale, wt, idw, T, sel_idx=None, sel_w=None, sigmoid=False):
+def moe_route(proj, off, corr, n_real, count, keep, top, scale, wt, idw, T, sel_idx=None, sel_w=None, sigmoid=False, off_gate=-1):
     """softmax router over ``corr.numel()`` outputs (the last ones beyond ``n_real`` are identity experts): dense weight
     rows ``wt`` [T, n_real] and the summed identity weight ``idw`` [T]; optionally the choices in order.  ``corr`` None:
-    ``n_real`` outputs, the largest logits are chosen and the weights are the softmax over the chosen logits alone; ``sigmoid``: their sigmoids times ``scale``"""
+    ``n_real`` outputs, the largest logits are chosen and the weights are the softmax over the chosen logits alone; ``sigmoid``: their sigmoids times ``scale``; ``off_gate`` >= 0: ``idw`` is the sigmoid of that column (gate of a shared expert)"""
     native().moe_route(proj, off, corr, corr.numel() if corr is not None else n_real, n_real, count, keep, top,
-                       float(scale), wt, idw, sel_idx, sel_w, T, int(bool(sigmoid)))
+                       float(scale), wt, idw, sel_idx, sel_w, T, int(bool(sigmoid)), int(off_gate))
 
 
-def gated_cols(x, off_a, off_b, out, n, act, T, wt=None, per=0, both=False, lead=0, scale_input=False):
+def gated_cols(x, off_a, off_b, out, n, act, T, wt=None, per=0, both=False, lead=0, scale_input=False, lead_w=None):
     """``out[t, c] = act(x[t, off_a + c]) * x[t, off_b + c]``, or ``* wt[t, c // per]`` with per-expert weights, or
     (``both``) times the two of them, the first ``lead`` columns having weight 1 (a shared expert in front of the routed ones);
-    ``scale_input`` (with ``both``): ``act(w a) * (w b)``, the expert's input carries the weight"""
-    native().gated_cols(x, off_a, off_b, wt, per, out, n, act, T, 2 if scale_input else int(bool(both)), int(lead))
+    ``scale_input`` (with ``both``): ``act(w a) * (w b)``, the expert's input carries the weight; ``lead_w`` [T]: weight of the
+    leading columns instead of 1"""
+    native().gated_cols(x, off_a, off_b, wt, per, out, n, act, T, 2 if scale_input else int(bool(both)), int(lead), lead_w)
 
 
 def head_up_gate(a, U, out, T, H, V, C, gate=None, off_g=0):
     """``out[t, h V + v] = sigmoid(gate[t, off_g + h V + v]) * sum_c U[h, v, c] a[t, h C + c]`` (no gate: the plain product)"""
     native().head_up_gate(a, U, gate, off_g, out, T, H, V, C)
+
+
+# ------------------------------------------------------- sandwich-norm hybrids (differential attention, state-space, retention)
+def sandwich_join(x, *, y=None, norm_y=None, kind_y=NORM_LAYER, h=None, norm_h=None, kind_h=NORM_LAYER, eps=1e-6, rows=None,
+                  n_rows=0):
+    """``x <- x + N_y(y)``, then ``h = N_h(x)`` as the operand of the next matrix product; ``norm_*`` = (weight, bias or None),
+    ``kind_*`` = NORM_RMS / NORM_LAYER / (h) NORM_NONE.  ``rows`` (with ``n_rows``): ``h[r]`` is the operand of token
+    ``rows[r]`` and the residual is left as it is."""
+    wy, by = norm_y if norm_y is not None else (None, None)
+    wh, bh = norm_h if norm_h is not None else (None, None)
+    native().sandwich_join(x, rows, n_rows if rows is not None else x.shape[0], y, kind_y, wy, by, kind_h, wh, bh, float(eps), h)
+
+
+def rot_table(positions, freq, freq_lo, amp, tab, T):
+    """``tab`` [T, 2 * pairs] = (cos, sin) of position * (freq + freq_lo) for every pair, times ``amp``"""
+    native().rot_table(positions, freq, freq_lo, float(amp), tab, T)
+
+
+def conv_rot_prep(proj, off, w, tail, tab, qscale, slots, q_out, k_cache, v_cache, q_start, q_len, kv_len, seq_slot, n_seqs, max_q,
+                  Hq, Gk, Gv, D, V):
+    """Attention with short convolutions: columns ``off`` .. of ``proj`` = [q | k | v] pass a causal convolution per channel (``w``
+    [channels, taps], inputs in front of the span in ``tail`` [slots, taps - 1, channels]), queries and keys turn in pairs
+    (i, i + half) by the step's rotary table ``tab`` [T, 2 * half] (None: no rotation); queries times ``qscale`` -> ``q_out``,
+    keys and values -> paged cache (``Gk`` = ``Gv`` = 0: another layer's are used)."""
+    native().conv_rot_prep(proj, off, w, tail, tab, float(qscale), slots, q_out, k_cache, v_cache, q_start, q_len, kv_len, seq_slot,
+                           n_seqs, max_q, Hq, Gk, Gv, D, V)
+    if max_q > 1 and w.shape[1] > 1:
+        LAUNCHES[0] += 1
+
+
+def diff_combine(a, lam, gain, out, T, H, G, V, eps):
+    """``out[t, h] = d / rms(d) * gain``, ``d = a_1 - lam * a_2`` for map outputs ``a`` [T, 2 H V] in the order (key/value head, map,
+    head of its group)"""
+    native().diff_combine(a, float(lam), float(gain), out, T, H, G, V, float(eps))
+
+
+def ssd_post(o, x, off_x, z, off_z, skip, w, out, T, H, V, parts, eps):
+    """``out = groupnorm((o + skip_h x) * silu(z)) * w`` with the RMS norm over ``parts`` equal parts of the ``H * V`` channels"""
+    native().ssd_post(o, x, off_x, z, off_z, skip, w, out, T, H, V, parts, float(eps))
+
+
+def side_gate(z, ids, table, off, out, n, T):
+    """``out[t, c] = gelu_tanh(z[t, c]) * table[ids[t], off + c]`` for c < n"""
+    native().side_gate(z, ids, table, off, out, n, T)

@@ -594,17 +594,17 @@ void softmax_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   c10::cuda::CUDAGuard guard(q.device());
   TORCH_CHECK(!(sink.has_value() && sink->defined()) || sink->numel() >= H, "softmax_attention: one sink per head");
   TORCH_CHECK(!(slopes.has_value() && slopes->defined()) || slopes->numel() >= H, "softmax_attention: one slope per head");
-  TORCH_CHECK(k_cache.scalar_type() == out.scalar_type() && v_cache.scalar_type() == out.scalar_type(),
-              "softmax_attention: cache and output dtypes must match");
+  TORCH_CHECK(k_cache.scalar_type() == v_cache.scalar_type() && (k_cache.scalar_type() == out.scalar_type() || is_f32(out)),
+              "softmax_attention: the output has the dtype of the cache or is float");
   check(b2b::launch_softmax_attention(fp(q), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
                                       static_cast<int>(out.stride(0)), ip(block_table),
                                       static_cast<int>(block_table.stride(0)), ip(q_start), ip(q_len), ip(kv_len),
                                       static_cast<int>(n_seqs), static_cast<int>(max_q), static_cast<int>(H),
                                       static_cast<int>(G), static_cast<int>(D), static_cast<int>(V),
                                       static_cast<int>(window), static_cast<float>(scale),
-                                      static_cast<int>(v_cache.stride(1)), is_f32(out), static_cast<float>(softcap),
+                                      static_cast<int>(v_cache.stride(1)), is_f32(k_cache), static_cast<float>(softcap),
                                       static_cast<int>(keep_first), fp_or_null(sink), static_cast<int>(v_heads),
-                                      fp_or_null(slopes), cur_stream()),
+                                      fp_or_null(slopes), is_f32(out), cur_stream()),
         "softmax_attention");
 }
 
@@ -643,13 +643,15 @@ void talk_prep(const Tensor& proj, int64_t off_q, int64_t off_k, const Tensor& t
 }
 
 void short_conv(const Tensor& x, int64_t off, const Tensor& w, const Tensor& tail, const Tensor& y, const Tensor& q_start,
-                const Tensor& q_len, const Tensor& kv_len, const Tensor& seq_slot, int64_t n_seqs, int64_t max_q) {
+                const Tensor& q_len, const Tensor& kv_len, const Tensor& seq_slot, int64_t n_seqs, int64_t max_q,
+                const OptT& bias, int64_t act) {
   c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(!(bias.has_value() && bias->defined()) || bias->numel() == w.size(0), "short_conv: one bias per channel");
   check(b2b::launch_short_conv(fp(x), static_cast<int>(x.stride(0)), static_cast<int>(off), fp(w),
                                const_cast<float*>(fp(tail)), const_cast<float*>(fp(y)), static_cast<int>(y.stride(0)),
                                ip(q_start), ip(q_len), ip(kv_len), ip(seq_slot), static_cast<int>(n_seqs),
                                static_cast<int>(max_q), static_cast<int>(w.size(0)), static_cast<int>(w.size(1)),
-                               cur_stream()),
+                               fp_or_null(bias), static_cast<int>(act), cur_stream()),
         "short_conv");
 }
 
@@ -671,10 +673,13 @@ void lin_scan(int64_t mode, const Tensor& qk, int64_t off_q, int64_t off_k, cons
               int64_t off_z, const OptT& zbias, const OptT& hparam, const OptT& beta, int64_t off_b, const OptT& aux,
               double qscale, double inv_tau, const Tensor& state, const Tensor& out, const Tensor& q_start,
               const Tensor& q_len, const Tensor& kv_len, const Tensor& seq_slot, int64_t n_seqs, int64_t max_q, int64_t H,
-              int64_t G, int64_t dk, int64_t dv) {
+              int64_t G, int64_t dk, int64_t dv, int64_t rdims) {
   c10::cuda::CUDAGuard guard(qk.device());
   auto ld = [](const OptT& t) { return (t.has_value() && t->defined()) ? static_cast<int>(t->stride(0)) : 0; };
-  TORCH_CHECK(mode == 2 ? fp_or_null(aux) != nullptr : (fp_or_null(z) != nullptr && fp_or_null(zbias) != nullptr),
+  TORCH_CHECK(mode == 2   ? fp_or_null(aux) != nullptr
+              : mode == 4 ? fp_or_null(zbias) != nullptr && fp_or_null(hparam) != nullptr && fp_or_null(beta) != nullptr
+              : mode == 5 ? fp_or_null(hparam) != nullptr && (rdims == 0 || fp_or_null(z) != nullptr)
+                          : fp_or_null(z) != nullptr && fp_or_null(zbias) != nullptr,
               "lin_scan: missing gate inputs for this mode");
   TORCH_CHECK(mode != 1 || (fp_or_null(hparam) != nullptr && fp_or_null(beta) != nullptr), "lin_scan: delta rule inputs");
   check(b2b::launch_lin_scan(static_cast<int>(mode), fp(qk), static_cast<int>(qk.stride(0)), static_cast<int>(off_q),
@@ -685,7 +690,7 @@ void lin_scan(int64_t mode, const Tensor& qk, int64_t off_q, int64_t off_k, cons
                              const_cast<float*>(fp(out)), static_cast<int>(out.stride(0)), ip(q_start), ip(q_len),
                              ip(kv_len), ip(seq_slot), static_cast<int>(n_seqs), static_cast<int>(max_q),
                              static_cast<int>(H), static_cast<int>(G), static_cast<int>(dk), static_cast<int>(dv),
-                             cur_stream()),
+                             static_cast<int>(rdims), cur_stream()),
         "lin_scan");
 }
 
@@ -749,7 +754,7 @@ void rot_heads(const Tensor& src, int64_t off, const Tensor& dst, int64_t H, int
 
 void moe_route(const Tensor& proj, int64_t off, const OptT& corr, int64_t E, int64_t n_real, int64_t count, int64_t keep,
                int64_t top, double scale, const Tensor& wt, const Tensor& idw, const OptT& sel_idx, const OptT& sel_w,
-               int64_t T, int64_t sigmoid) {
+               int64_t T, int64_t sigmoid, int64_t off_gate) {
   c10::cuda::CUDAGuard guard(proj.device());
   const bool has_sel = sel_idx.has_value() && sel_idx->defined();
   TORCH_CHECK(!(corr.has_value() && corr->defined()) || corr->numel() == E, "moe_route: one correction per router output");
@@ -759,7 +764,7 @@ void moe_route(const Tensor& proj, int64_t off, const OptT& corr, int64_t E, int
                               const_cast<float*>(fp(wt)), static_cast<int>(wt.stride(0)), const_cast<float*>(fp(idw)),
                               has_sel ? const_cast<int*>(ip(*sel_idx)) : nullptr,
                               const_cast<float*>(fp_or_null(sel_w)), static_cast<int>(T), static_cast<int>(sigmoid),
-                              cur_stream()),
+                              static_cast<int>(off_gate), cur_stream()),
         "moe_route");
 }
 
@@ -773,14 +778,14 @@ void poly_norm(const Tensor& in, int64_t off, const Tensor& w, const Tensor& out
 }
 
 void gated_cols(const Tensor& in, int64_t off_a, int64_t off_b, const OptT& wt, int64_t per, const Tensor& out, int64_t n,
-                int64_t act, int64_t T, int64_t both, int64_t lead) {
+                int64_t act, int64_t T, int64_t both, int64_t lead, const OptT& lead_w) {
   c10::cuda::CUDAGuard guard(in.device());
   const bool has_wt = wt.has_value() && wt->defined();
   check(b2b::launch_gated_cols(fp(in), static_cast<int>(in.stride(0)), static_cast<int>(off_a), static_cast<int>(off_b),
                                fp_or_null(wt), has_wt ? static_cast<int>(wt->stride(0)) : 0,
                                static_cast<int>(per > 0 ? per : 1), out.data_ptr(), static_cast<int>(out.stride(0)),
                                static_cast<int>(n), static_cast<int>(act), static_cast<int>(T), is_f32(out),
-                               static_cast<int>(both), static_cast<int>(lead), cur_stream()),
+                               static_cast<int>(both), static_cast<int>(lead), fp_or_null(lead_w), cur_stream()),
         "gated_cols");
 }
 
@@ -797,6 +802,85 @@ void head_up_gate(const Tensor& a, const Tensor& U, const OptT& gate, int64_t of
                                  static_cast<int>(out.stride(0)), static_cast<int>(T), static_cast<int>(H),
                                  static_cast<int>(V), static_cast<int>(C), is_f32(out), cur_stream()),
         "head_up_gate");
+}
+
+// ---- a norm behind and in front of every sublayer, differential attention prep, state-space output (csrc/sandwich.cu)
+void sandwich_join(const Tensor& x, const OptT& rows, int64_t n_rows, const OptT& y, int64_t kind_y, const OptT& wy, const OptT& by,
+                   int64_t kind_h, const OptT& wh, const OptT& bh, double eps, const OptT& h) {
+  c10::cuda::CUDAGuard guard(x.device());
+  const bool has_h = h.has_value() && h->defined(), has_y = y.has_value() && y->defined();
+  const int W = static_cast<int>(x.size(-1));
+  auto vec = [&](const OptT& t) { return !(t.has_value() && t->defined()) || t->numel() == W; };
+  TORCH_CHECK(vec(wy) && vec(by) && vec(wh) && vec(bh), "sandwich_join: norm weights and biases have the width of x");
+  check(b2b::launch_sandwich_join(const_cast<float*>(fp(x)), (rows.has_value() && rows->defined()) ? ip(*rows) : nullptr,
+                                  static_cast<int>(n_rows), fp_or_null(y), has_y ? static_cast<int>(y->stride(0)) : 0,
+                                  static_cast<int>(kind_y), fp_or_null(wy), fp_or_null(by), static_cast<int>(kind_h), fp_or_null(wh),
+                                  fp_or_null(bh), static_cast<float>(eps), has_h ? h->data_ptr() : nullptr,
+                                  has_h ? static_cast<int>(h->stride(0)) : 0, W, has_h ? is_f32(*h) : 1, cur_stream()),
+        "sandwich_join");
+}
+
+void rot_table(const Tensor& positions, const Tensor& freq, const Tensor& freq_lo, double amp, const Tensor& tab, int64_t T) {
+  c10::cuda::CUDAGuard guard(tab.device());
+  TORCH_CHECK(freq.numel() == freq_lo.numel() && tab.is_contiguous() && tab.size(-1) == 2 * freq.numel() && tab.size(0) >= T,
+              "rot_table: sizes");
+  check(b2b::launch_rot_table(ip(positions), fp(freq), fp(freq_lo), static_cast<int>(freq.numel()), static_cast<float>(amp),
+                              const_cast<float*>(fp(tab)), static_cast<int>(T), cur_stream()),
+        "rot_table");
+}
+
+// proj columns off .. : q (Hq heads of D) | k (Gk heads of D) | v (Gv heads of V); w [channels, taps]; tab [T, 2 half]
+void conv_rot_prep(const Tensor& proj, int64_t off, const Tensor& w, const Tensor& tail, const OptT& tab, double qscale,
+                   const Tensor& slots, const Tensor& q_out, const OptT& k_cache, const OptT& v_cache, const Tensor& q_start,
+                   const Tensor& q_len, const Tensor& kv_len, const Tensor& seq_slot, int64_t n_seqs, int64_t max_q, int64_t Hq,
+                   int64_t Gk, int64_t Gv, int64_t D, int64_t V) {
+  c10::cuda::CUDAGuard guard(proj.device());
+  const bool has_tab = tab.has_value() && tab->defined(), has_k = k_cache.has_value() && k_cache->defined();
+  TORCH_CHECK(w.size(0) == (Hq + Gk) * D + Gv * V && w.is_contiguous(), "conv_rot_prep: one row of taps per channel");
+  TORCH_CHECK(w.size(1) == 1 || (tail.size(1) == w.size(1) - 1 && tail.size(2) == w.size(0) && tail.is_contiguous()),
+              "conv_rot_prep: the tail is [slots, taps - 1, channels]");
+  TORCH_CHECK(q_out.is_contiguous() && q_out.size(-1) == Hq * D, "conv_rot_prep: dense query rows");
+  TORCH_CHECK((Gk == 0 && Gv == 0) || (has_k && v_cache.has_value() && v_cache->defined()), "conv_rot_prep: keys need a cache");
+  check(b2b::launch_conv_rot_prep(fp(proj), static_cast<int>(proj.stride(0)), static_cast<int>(off), fp(w),
+                                  const_cast<float*>(fp(tail)), fp_or_null(tab), has_tab ? static_cast<int>(tab->size(-1) / 2) : 0,
+                                  static_cast<float>(qscale), ip(slots), q_out.data_ptr(), is_f32(q_out),
+                                  has_k ? k_cache->data_ptr() : nullptr, has_k ? v_cache->data_ptr() : nullptr,
+                                  has_k ? is_f32(*k_cache) : 0, ip(q_start), ip(q_len), ip(kv_len), ip(seq_slot),
+                                  static_cast<int>(n_seqs), static_cast<int>(max_q), static_cast<int>(Hq), static_cast<int>(Gk),
+                                  static_cast<int>(Gv), static_cast<int>(D), static_cast<int>(V), static_cast<int>(w.size(1)),
+                                  cur_stream()),
+        "conv_rot_prep");
+}
+
+void diff_combine(const Tensor& in, double lambda, double gain, const Tensor& out, int64_t T, int64_t H, int64_t G, int64_t V,
+                  double eps) {
+  c10::cuda::CUDAGuard guard(in.device());
+  TORCH_CHECK(in.size(-1) >= 2 * H * V && out.size(-1) >= H * V, "diff_combine: rows too short");
+  check(b2b::launch_diff_combine(fp(in), static_cast<int>(in.stride(0)), static_cast<float>(lambda), static_cast<float>(gain),
+                                 out.data_ptr(), static_cast<int>(out.stride(0)), static_cast<int>(T), static_cast<int>(H),
+                                 static_cast<int>(G), static_cast<int>(V), static_cast<float>(eps), is_f32(out), cur_stream()),
+        "diff_combine");
+}
+
+void ssd_post(const Tensor& o, const Tensor& x, int64_t off_x, const Tensor& z, int64_t off_z, const Tensor& skip, const Tensor& w,
+              const Tensor& out, int64_t T, int64_t H, int64_t V, int64_t parts, double eps) {
+  c10::cuda::CUDAGuard guard(o.device());
+  TORCH_CHECK(skip.numel() == H && w.numel() == H * V && out.size(-1) >= H * V, "ssd_post: sizes");
+  check(b2b::launch_ssd_post(fp(o), static_cast<int>(o.stride(0)), fp(x) + off_x, static_cast<int>(x.stride(0)), fp(z) + off_z,
+                             static_cast<int>(z.stride(0)), fp(skip), fp(w), out.data_ptr(), static_cast<int>(out.stride(0)),
+                             static_cast<int>(T), static_cast<int>(H), static_cast<int>(V), static_cast<int>(parts),
+                             static_cast<float>(eps), is_f32(out), cur_stream()),
+        "ssd_post");
+}
+
+void side_gate(const Tensor& z, const Tensor& ids, const Tensor& table, int64_t off, const Tensor& out, int64_t n, int64_t T) {
+  c10::cuda::CUDAGuard guard(z.device());
+  TORCH_CHECK(table.scalar_type() == out.scalar_type() && off >= 0 && off + n <= table.size(1) && out.size(-1) >= n,
+              "side_gate: table and output");
+  check(b2b::launch_side_gate(fp(z), static_cast<int>(z.stride(0)), ip(ids), table.data_ptr(), static_cast<int>(table.stride(0)),
+                              static_cast<int>(off), static_cast<int>(table.size(0)), out.data_ptr(), static_cast<int>(out.stride(0)),
+                              static_cast<int>(n), static_cast<int>(T), is_f32(out), cur_stream()),
+        "side_gate");
 }
 }  // namespace
 
@@ -863,4 +947,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("poly_norm", &poly_norm);
   m.def("gated_cols", &gated_cols);
   m.def("head_up_gate", &head_up_gate);
+  m.def("sandwich_join", &sandwich_join);
+  m.def("rot_table", &rot_table);
+  m.def("conv_rot_prep", &conv_rot_prep);
+  m.def("diff_combine", &diff_combine);
+  m.def("ssd_post", &ssd_post);
+  m.def("side_gate", &side_gate);
 }

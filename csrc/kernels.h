@@ -116,21 +116,25 @@ int launch_softmax_attention(const float* q, const void* k_cache, const void* v_
                              const int* block_table, int max_pages, const int* q_start, const int* q_len,
                              const int* kv_len, int n_seqs, int max_q, int H, int G, int D, int V, int window,
                              float scale, int ldv, int f32, float softcap, int keep_first, const float* sink, int Gv,
-                             const float* slope, cudaStream_t s);
+                             const float* slope, int out_f32, cudaStream_t s);
 int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* tail, float* y, int ld_y,
                       const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs,
-                      int max_q, int C, int taps, cudaStream_t s);
+                      int max_q, int C, int taps, const float* bias, int act, cudaStream_t s);
+int launch_short_conv_commit(const float* x, int ld_x, int off, float* tail, const int* q_start, const int* q_len,
+                             const int* kv_len, const int* seq_slot, int n_seqs, int C, int taps, cudaStream_t s);
 int launch_mlstm_gates(const float* proj, int ld, int off_q, int off_k, int off_i, int off_f, const float* bi,
                        const float* bf_, float cap, float qscale, float* nstate, float* mstate, float* aux,
                        const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs, int H,
                        int dk, cudaStream_t s);
 // mode: 0 diag-gated linear attention, 1 delta rule with channel decay, 2 mLSTM matrix memory, 3 HGRN2 (forget gate with a
-// lower bound, its complement is the write strength; hparam = the bound [H * dk], z = the gate projection, no keys)
+// lower bound, its complement is the write strength; hparam = the bound [H * dk], z = the gate projection, no keys), 4
+// state-space recurrence (hparam = A_log [H], zbias = bias of the step size [H], beta = its projection), 5 retention (hparam =
+// decay [H], z = rotary table [T, rdims] of (cos, sin) pairs)
 int launch_lin_scan(int mode, const float* qk, int ld_qk, int off_q, int off_k, const float* v, int ld_v, int off_v,
                     const float* z, int ld_z, int off_z, const float* zbias, const float* hparam, const float* beta,
                     int ld_b, int off_b, const float* aux, float qscale, float inv_tau, float* state, float* out,
                     int ld_out, const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs,
-                    int max_q, int H, int G, int dk, int dv, cudaStream_t s);
+                    int max_q, int H, int G, int dk, int dv, int rdims, cudaStream_t s);
 int launch_scan_post(const float* o, int ld_o, const float* gate, int ld_g, int off_g, const float* weight, int wshared,
                      int act, const float* aux, void* out, int ld_out, int T, int H, int dv, float eps, int f32,
                      cudaStream_t s);
@@ -153,14 +157,33 @@ int launch_rot_heads(const float* src, int ld, int off, float* dst, int H, int D
                      cudaStream_t s);
 int launch_moe_route(const float* proj, int ld, int off, const float* corr, int E, int n_real, int count, int keep,
                      int top, float scale, float* wt, int ld_wt, float* idw, int* sel_idx, float* sel_w, int T,
-                     int sigmoid, cudaStream_t s);
+                     int sigmoid, int off_gate, cudaStream_t s);
 int launch_poly_norm(const float* in, int ld_in, int off, const float* w, void* out, int ld_out, int n, float eps, int T,
                      int f32, cudaStream_t s);
 int launch_gated_cols(const float* in, int ld_in, int off_a, int off_b, const float* wt, int ld_wt, int per, void* out,
-                      int ld_out, int n, int act, int T, int f32, int both, int lead, cudaStream_t s);
+                      int ld_out, int n, int act, int T, int f32, int both, int lead, const float* lead_w, cudaStream_t s);
 // out[t, h, :] = gate * U[h] a[t, h, :]: one [V, C] matrix per head (operands bf16, or float when f32), sigmoid gate from fp32 rows
 int launch_head_up_gate(const void* a, int ld_a, const void* U, const float* gate, int ld_g, int off_g, void* out,
                         int ld_out, int T, int H, int V, int C, int f32, cudaStream_t s);
+
+// sandwich.cu: a norm behind and in front of every sublayer (kind 0 RMS norm, 1 layer norm, 2 none), rotary table of a step,
+// convolution + rotation + cache rows of (differential) attention, a_1 - lambda a_2 of its two maps, output of the state-space
+// recurrence (skip, gate, grouped norm), gelu gate times a token's own channels
+int launch_sandwich_join(float* x, const int* rows, int n_rows, const float* y, int ld_y, int kind_y, const float* wy,
+                         const float* by, int kind_h, const float* wh, const float* bh, float eps, void* h, int ld_h, int W, int f32,
+                         cudaStream_t s);
+int launch_rot_table(const int* positions, const float* freq, const float* freq_lo, int pairs, float amp, float* tab, int T,
+                     cudaStream_t s);
+int launch_conv_rot_prep(const float* proj, int ld, int off, const float* w, float* tail, const float* tab, int half, float qscale,
+                         const int* slots, void* q_out, int q_f32, void* k_cache, void* v_cache, int c_f32, const int* q_start,
+                         const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs, int max_q, int Hq, int Gk, int Gv,
+                         int D, int V, int taps, cudaStream_t s);
+int launch_diff_combine(const float* in, int ld_in, float lambda, float gain, void* out, int ld_out, int T, int H, int G, int V,
+                        float eps, int f32, cudaStream_t s);
+int launch_ssd_post(const float* o, int ld_o, const float* x, int ld_x, const float* z, int ld_z, const float* skip, const float* w,
+                    void* out, int ld_out, int T, int H, int V, int parts, float eps, int f32, cudaStream_t s);
+int launch_side_gate(const float* z, int ld_z, const int* ids, const void* table, int ld_t, int off, int vocab, void* out, int ld_out,
+                     int n, int T, int f32, cudaStream_t s);
 
 // bounded handoff waits: device abort word + time limit for the waits of each translation unit (0 / null = trap policy)
 int set_wait_policy_gemm(uint32_t* abort_word, unsigned long long limit_ns);

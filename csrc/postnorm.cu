@@ -339,10 +339,12 @@ __global__ void __launch_bounds__(PN_THREADS)
 // idw[t]; wt [T, ld_wt] receives the dense weight row of the real experts (0 = not chosen).  sel_idx / sel_w [T, top]
 // (optional) list the choices in order.  sigmoid != 0 (with corr == nullptr): the weights are sigmoid(z) * scale of the chosen
 // logits, not renormalised (the largest logits have the largest sigmoids).
+// off_gate >= 0: idw[t] = sigmoid(column off_gate of the row), the gate of a shared expert (there are no identity experts then).
 __global__ void __launch_bounds__(128)
     moe_route_kernel(const float* __restrict__ proj, int ld, int off, const float* __restrict__ corr, int E, int n_real,
                      int count, int keep, int top, float scale, float* __restrict__ wt, int ld_wt,
-                     float* __restrict__ idw, int* __restrict__ sel_idx, float* __restrict__ sel_w, int T, int sigmoid) {
+                     float* __restrict__ idw, int* __restrict__ sel_idx, float* __restrict__ sel_w, int T, int sigmoid,
+                     int off_gate) {
   pdl_begin();
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -437,7 +439,7 @@ __global__ void __launch_bounds__(128)
     if (sel_w != nullptr) sel_w[static_cast<size_t>(t) * top + k] = wgt;
   }
   keep_w = warp_sum_(keep_w);
-  if (lane == 0) idw[t] = keep_w;
+  if (lane == 0) idw[t] = off_gate >= 0 ? sigmoid_(proj[static_cast<size_t>(t) * ld + off_gate]) : keep_w;
 }
 
 // ------------------------------------------------------------------------------------------- gated columns
@@ -445,22 +447,28 @@ __global__ void __launch_bounds__(128)
 // act(a) * in[t, off_b + c] * weight, where the first `lead` columns have weight 1 and column c >= lead has
 // wt[t, (c - lead) / per] (gated experts side by side behind a shared one).  both == 2: act(w a) * (w b), the weight scales what
 // goes into the expert.
-// act: 0 silu, 1 exact (erf) gelu, 2 tanh gelu.  Four columns per thread when every offset allows 16-byte accesses.
+// lead_w (optional): the leading columns have the token's weight lead_w[t] instead of 1 (a gated shared expert).
+// act: 0 silu, 1 exact (erf) gelu, 2 tanh gelu, 3 squared relu.  Four columns per thread when every offset allows 16-byte accesses.
 __device__ __forceinline__ float act_(float z, int act) {
   if (act == 0) return z / (1.f + expf(-z));
   if (act == 1) return 0.5f * z * (1.f + erff(z * 0.70710678118654752440f));
+  if (act == 3) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  }
   return 0.5f * z * (1.f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
 }
 template <typename OT>
 __global__ void __launch_bounds__(256)
     gated_cols_kernel(const float* __restrict__ in, int ld_in, int off_a, int off_b, const float* __restrict__ wt,
-                      int ld_wt, int per, OT* __restrict__ out, int ld_out, int n, int act, int T, int both, int lead) {
+                      int ld_wt, int per, OT* __restrict__ out, int ld_out, int n, int act, int T, int both, int lead,
+                      const float* __restrict__ lead_w) {
   pdl_begin();
   const long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (e >= static_cast<long long>(T) * n) return;
   const int c = static_cast<int>(e % n);
   const size_t t = static_cast<size_t>(e / n);
-  float b = wt != nullptr ? (c < lead ? 1.f : wt[t * ld_wt + (c - lead) / per]) : in[t * ld_in + off_b + c];
+  float b = wt != nullptr ? (c < lead ? (lead_w != nullptr ? lead_w[t] : 1.f) : wt[t * ld_wt + (c - lead) / per]) : in[t * ld_in + off_b + c];
   const float a = act_(in[t * ld_in + off_a + c] * (both == 2 ? b : 1.f), act);
   if (both && wt != nullptr) b *= in[t * ld_in + off_b + c];
   stf(out, t * ld_out + c, a * b);
@@ -470,7 +478,8 @@ __global__ void __launch_bounds__(256)
 template <typename OT>
 __global__ void __launch_bounds__(256)
     gated_cols_vec_kernel(const float* __restrict__ in, int ld_in, int off_a, int off_b, const float* __restrict__ wt,
-                          int ld_wt, int per, OT* __restrict__ out, int ld_out, int n, int act, int both, int lead) {
+                          int ld_wt, int per, OT* __restrict__ out, int ld_out, int n, int act, int both, int lead,
+                          const float* __restrict__ lead_w) {
   pdl_begin();
   const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
   if (c >= n) return;
@@ -478,7 +487,7 @@ __global__ void __launch_bounds__(256)
   float4 a = *reinterpret_cast<const float4*>(in + t * ld_in + off_a + c);
   float4 b;
   if (wt != nullptr) {
-    const float wv = c < lead ? 1.f : wt[t * ld_wt + (c - lead) / per];      // per and lead are multiples of four: one expert for the four columns
+    const float wv = c < lead ? (lead_w != nullptr ? lead_w[t] : 1.f) : wt[t * ld_wt + (c - lead) / per];      // per and lead are multiples of four: one expert for the four columns
     b = make_float4(wv, wv, wv, wv);
     if (both == 2) a = make_float4(wv * a.x, wv * a.y, wv * a.z, wv * a.w);
     if (both) {
@@ -742,9 +751,10 @@ int launch_rot_heads(const float* src, int ld, int off, float* dst, int H, int D
 
 int launch_moe_route(const float* proj, int ld, int off, const float* corr, int E, int n_real, int count, int keep,
                      int top, float scale, float* wt, int ld_wt, float* idw, int* sel_idx, float* sel_w, int T,
-                     int sigmoid, cudaStream_t s) {
+                     int sigmoid, int off_gate, cudaStream_t s) {
   if (T <= 0) return 0;
   if (sigmoid && corr != nullptr) return -2;
+  if (off_gate >= 0 && n_real != E) return -2;
   if (E <= 0 || n_real < 0 || n_real > E || count <= 0 || E % count != 0 || top <= 0 || top > E) return -2;
   if (corr == nullptr && count > 1 && keep < count) return -2;      // group-limited choice is defined on corrected scores
   int warps = 4;
@@ -752,7 +762,7 @@ int launch_moe_route(const float* proj, int ld, int off, const float* corr, int 
   const size_t smem = static_cast<size_t>(warps) * 4 * E * sizeof(float);
   if (smem > 48 * 1024) return -2;
   launch_kernel(moe_route_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, s, 1u, proj, ld, off, corr, E,
-                n_real, count, keep, top, scale, wt, ld_wt, idw, sel_idx, sel_w, T, sigmoid);
+                n_real, count, keep, top, scale, wt, ld_wt, idw, sel_idx, sel_w, T, sigmoid, off_gate);
   return last_error();
 }
 
@@ -782,7 +792,7 @@ int launch_poly_norm(const float* in, int ld_in, int off, const float* w, void* 
 }
 
 int launch_gated_cols(const float* in, int ld_in, int off_a, int off_b, const float* wt, int ld_wt, int per, void* out,
-                      int ld_out, int n, int act, int T, int f32, int both, int lead, cudaStream_t s) {
+                      int ld_out, int n, int act, int T, int f32, int both, int lead, const float* lead_w, cudaStream_t s) {
   const long long tot = static_cast<long long>(T) * n;
   if (tot <= 0) return 0;
   if (n % 4 == 0 && ld_in % 4 == 0 && off_a % 4 == 0 && (wt != nullptr ? per % 4 == 0 && lead % 4 == 0 : off_b % 4 == 0) &&
@@ -791,19 +801,19 @@ int launch_gated_cols(const float* in, int ld_in, int off_a, int off_b, const fl
     const dim3 vgrid((n / 4 + 255) / 256, T);
     if (f32)
       launch_kernel(gated_cols_vec_kernel<float>, vgrid, dim3(256), 0, s, 1u, in, ld_in, off_a, off_b, wt, ld_wt, per,
-                    static_cast<float*>(out), ld_out, n, act, both, lead);
+                    static_cast<float*>(out), ld_out, n, act, both, lead, lead_w);
     else
       launch_kernel(gated_cols_vec_kernel<bf16>, vgrid, dim3(256), 0, s, 1u, in, ld_in, off_a, off_b, wt, ld_wt, per,
-                    static_cast<bf16*>(out), ld_out, n, act, both, lead);
+                    static_cast<bf16*>(out), ld_out, n, act, both, lead, lead_w);
     return last_error();
   }
   const dim3 grid(static_cast<unsigned>((tot + 255) / 256));
   if (f32)
     launch_kernel(gated_cols_kernel<float>, grid, dim3(256), 0, s, 1u, in, ld_in, off_a, off_b, wt, ld_wt, per,
-                  static_cast<float*>(out), ld_out, n, act, T, both, lead);
+                  static_cast<float*>(out), ld_out, n, act, T, both, lead, lead_w);
   else
     launch_kernel(gated_cols_kernel<bf16>, grid, dim3(256), 0, s, 1u, in, ld_in, off_a, off_b, wt, ld_wt, per,
-                  static_cast<bf16*>(out), ld_out, n, act, T, both, lead);
+                  static_cast<bf16*>(out), ld_out, n, act, T, both, lead, lead_w);
   return last_error();
 }
 

@@ -14,10 +14,11 @@
 //                        linear distance bias, value heads counted apart from key heads; an
 //                        exact CUDA-core kernel (one warp per query and head, online softmax) and a tensor-core kernel
 //                        for spans in the bf16 mode
-//   * short_conv         causal per-channel convolution over time + silu, with the last taps-1 inputs per sequence slot
+//   * short_conv         causal per-channel convolution over time (optional bias) + silu, with the last taps-1 inputs per sequence slot
 //   * mlstm_gates        the scalar part of the matrix memory (mLSTM): capped gates, running maximum, normaliser
 //   * lin_scan           gated linear recurrences with an fp32 [dk, dv] state per head and sequence slot:
-//                        diag-gated (GLA), delta rule with a decay per key channel, mLSTM matrix memory
+//                        diag-gated (GLA), delta rule with a decay per key channel, mLSTM matrix memory, HGRN2, state-space
+//                        recurrence with a decay per head and token, retention with a constant decay per head
 //   * scan_post          per-head output norm, weight, output gate -> GEMM operand
 //
 // Everything the designs want in 32-bit stays in fp32: the residual, every norm, angles, attention scores and weights,
@@ -783,16 +784,17 @@ __global__ void __launch_bounds__(32 * SMX_MMA_WARPS, 3)
 }
 
 // ---------------------------------------------------------------------------------------- short convolution
-// y[t, c] = silu(sum_j w[c, j] * x[t - (taps-1) + j, c]) per sequence; inputs before the span come from
+// y[t, c] = silu(bias[c] + sum_j w[c, j] * x[t - (taps-1) + j, c]) per sequence (bias optional, act 0: no silu); inputs before the span come from
 // tail [slots, taps-1, C] (oldest first; zeros when the span starts the sequence).  x = proj columns off .. off + C.
 // grid (channel blocks, token groups, sequences); a thread walks `tpt` tokens of one channel with the window in registers.
-constexpr int CONV_MAX_TAPS = 8;
+constexpr int CONV_MAX_TAPS = 32;      // (MT: taps the registers of an instance hold)
 
+template <int MT>
 __global__ void __launch_bounds__(128)
     short_conv_kernel(const float* __restrict__ x, int ld_x, int off, const float* __restrict__ w,
                       const float* __restrict__ tail, float* __restrict__ y, int ld_y, const int* __restrict__ q_start,
                       const int* __restrict__ q_len, const int* __restrict__ kv_len, const int* __restrict__ seq_slot,
-                      int C, int taps, int tpt) {
+                      int C, int taps, int tpt, const float* __restrict__ bias, int act) {
   pdl_begin();
   const int s = blockIdx.z, n = q_len[s];
   const int i0 = blockIdx.y * tpt;
@@ -800,9 +802,9 @@ __global__ void __launch_bounds__(128)
   if (i0 >= n || c >= C) return;
   const int t0 = q_start[s], pos0 = kv_len[s] - n;
   const float* tl = tail + static_cast<size_t>(seq_slot[s]) * (taps - 1) * C;
-  float wr[CONV_MAX_TAPS], win[CONV_MAX_TAPS];        // win[j]: input at distance taps-1-j behind the current token
+  float wr[MT], win[MT];        // win[j]: input at distance taps-1-j behind the current token
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_TAPS; ++j) {
+  for (int j = 0; j < MT; ++j) {
     wr[j] = j < taps ? w[static_cast<size_t>(c) * taps + j] : 0.f;
     win[j] = 0.f;
     if (j < taps - 1) {
@@ -812,23 +814,25 @@ __global__ void __launch_bounds__(128)
     }
   }
   const int i1 = min(n, i0 + tpt);
+  const float b = bias != nullptr ? bias[c] : 0.f;
   for (int i = i0; i < i1; ++i) {
     const float cur = x[static_cast<size_t>(t0 + i) * ld_x + off + c];
-    float acc = 0.f;
+    float acc = b;
 #pragma unroll
-    for (int j = 0; j < CONV_MAX_TAPS; ++j) {
+    for (int j = 0; j < MT; ++j) {
       if (j < taps - 1) {
         acc += wr[j] * win[j];
-        win[j] = (j + 1 < taps - 1) ? win[j + 1] : cur;
+        win[j] = (j + 1 < MT && j + 1 < taps - 1) ? win[j + 1 < MT ? j + 1 : j] : cur;
       } else if (j == taps - 1) {
         acc += wr[j] * cur;
       }
     }
-    y[static_cast<size_t>(t0 + i) * ld_y + c] = silu_(acc);
+    y[static_cast<size_t>(t0 + i) * ld_y + c] = act ? silu_(acc) : acc;
   }
 }
 
 // the last taps-1 inputs of every sequence -> tail (runs after the convolution of the step has read the old tail)
+template <int MT>
 __global__ void short_conv_commit_kernel(const float* __restrict__ x, int ld_x, int off, float* __restrict__ tail,
                                          const int* __restrict__ q_start, const int* __restrict__ q_len,
                                          const int* __restrict__ kv_len, const int* __restrict__ seq_slot, int C,
@@ -839,9 +843,9 @@ __global__ void short_conv_commit_kernel(const float* __restrict__ x, int ld_x, 
   if (n <= 0 || c >= C) return;
   const int t0 = q_start[s], pos0 = kv_len[s] - n;
   float* tl = tail + static_cast<size_t>(seq_slot[s]) * (taps - 1) * C;
-  float nv[CONV_MAX_TAPS];
+  float nv[MT];
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_TAPS; ++j) {
+  for (int j = 0; j < MT; ++j) {
     nv[j] = 0.f;
     if (j < taps - 1) {
       const int i = n - (taps - 1) + j;
@@ -850,7 +854,7 @@ __global__ void short_conv_commit_kernel(const float* __restrict__ x, int ld_x, 
     }
   }
 #pragma unroll
-  for (int j = 0; j < CONV_MAX_TAPS; ++j)
+  for (int j = 0; j < MT; ++j)
     if (j < taps - 1) tl[static_cast<size_t>(j) * C + c] = nv[j];
 }
 
@@ -1018,11 +1022,15 @@ __global__ void __launch_bounds__(32)
 //     LS_MLSTM  q = x_q * qscale, k = take * x_k, d = keep   (keep, take from mlstm_gates)
 //     LS_HGRN2  q = silu(x_q), d = lo + (1 - lo) sigmoid(z + bias), k = 1 - d   (keyless: the write strength is the
 //               complement of the forget gate; lo [H * dk] = hparam bounds the gate from below, z is a plain projection)
+//     LS_SSD    q = x_q, k = dt x_k (head h reads q/k head h / (H/G)), d = exp(-exp(A_h) dt) with dt = softplus(x_b + bias_h):
+//               one decay per head and token, the step size also scales the write (state-space recurrence)
+//     LS_RET    q = turn(x_q) * qscale, k = turn(x_k), d = hparam[h]: a constant decay per head; the first rdims channels turn in
+//               adjacent pairs by z [T, rdims] = (cos, sin) per pair, the token's rotary table
 // Columns of S are independent: a block owns CB columns of one (sequence, head); LN lanes share a column group, each with
 // R key channels in registers (channel of (lane l, register m) = l + LN m; dk padded to R * LN with zeros).  Spans: while
 // the scan warps walk tile i (the only token-sequential work) the staging warps prepare tile i + 1 in the other half of a
 // double buffer; decode steps (DEC): every span is one token, all threads stage, then scan.
-enum { LS_GLA = 0, LS_DELTA = 1, LS_MLSTM = 2, LS_HGRN2 = 3 };
+enum { LS_GLA = 0, LS_DELTA = 1, LS_MLSTM = 2, LS_HGRN2 = 3, LS_SSD = 4, LS_RET = 5 };
 // staging threads of a span block (8 warps with one token each per tile measured no better than 4 with two)
 __host__ __device__ constexpr int ls_stage_threads(int) { return 128; }
 // state columns per thread: 2 for spans; 4 with 16-byte state accesses for decode steps (a stream over the states)
@@ -1040,6 +1048,7 @@ struct ScanArgs {
   float* state; float* out; int ld_out;
   const int* q_start; const int* q_len; const int* kv_len; const int* seq_slot;
   int H, G, dk, dv;
+  int rdims;                                      // RET: rotated channels
 };
 
 template <int MODE, int R, int LN, bool DEC, int CB>
@@ -1071,7 +1080,8 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
   const int sw = DEC ? warp : warp - NSCAN / 32;
   const int cgp = (tid % NSCAN) / LN, l = tid % LN;
   const int c0 = blockIdx.x * CB + cgp * C;
-  const int hqk = MODE == LS_DELTA ? hd / (H / a.G) : hd;
+  constexpr bool ZC = MODE == LS_GLA || MODE == LS_DELTA || MODE == LS_HGRN2;      // a gate input per key channel
+  const int hqk = (MODE == LS_DELTA || MODE == LS_SSD) ? hd / (H / a.G) : hd;
   float* S_g = a.state + (static_cast<size_t>(a.seq_slot[s]) * H + hd) * static_cast<size_t>(dk) * dv;
   const bool vec = C == 4 && (dv % 4 == 0) && (c0 + C <= dv);        // 16-byte state accesses
   float S[C][R];
@@ -1096,10 +1106,11 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
 #pragma unroll
   for (int e = 0; e < EPL; ++e) {
     const int i = lane + 32 * e;
-    zb[e] = (MODE != LS_MLSTM && stager && i < dk) ? a.zbias[hd * dk + i] : 0.f;
+    zb[e] = (ZC && stager && i < dk) ? a.zbias[hd * dk + i] : 0.f;
     lob[e] = (MODE == LS_HGRN2 && stager && i < dk) ? a.hparam[hd * dk + i] : 0.f;
   }
-  const float rate = MODE == LS_DELTA ? expf(a.hparam[hd]) : 0.f;
+  const float rate = (MODE == LS_DELTA || MODE == LS_SSD) ? expf(a.hparam[hd]) : 0.f;
+  const float hconst = MODE == LS_RET ? a.hparam[hd] : (MODE == LS_SSD ? a.zbias[hd] : 0.f);      // decay; bias of the step size
   float pq[TPW][EPL], pk[TPW][EPL], pz[TPW][EPL], pv[TPW], pb[TPW], pd[TPW];
   const int vc = blockIdx.x * CB + lane;
   auto load_tile = [&](int tb) {
@@ -1115,7 +1126,8 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
         const bool ok = tok && i < dk;
         pq[tw][e] = ok ? qrow[a.off_q + i] : 0.f;
         pk[tw][e] = (MODE != LS_HGRN2 && ok) ? qrow[a.off_k + i] : 0.f;
-        if (MODE != LS_MLSTM) pz[tw][e] = ok ? a.z[t * a.ld_z + a.off_z + hd * dk + i] : 0.f;
+        if (ZC) pz[tw][e] = ok ? a.z[t * a.ld_z + a.off_z + hd * dk + i] : 0.f;
+        if (MODE == LS_RET) pz[tw][e] = (tok && i < a.rdims) ? a.z[t * a.ld_z + i] : ((i & 1) ? 0.f : 1.f);
       }
       pv[tw] = 0.f;
       if (CB <= 32) {
@@ -1123,7 +1135,7 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
       }
       pb[tw] = 1.f;
       pd[tw] = 1.f;
-      if (MODE == LS_DELTA) pb[tw] = tok ? a.beta[t * a.ld_b + a.off_b + hd] : 0.f;
+      if (MODE == LS_DELTA || MODE == LS_SSD) pb[tw] = tok ? a.beta[t * a.ld_b + a.off_b + hd] : 0.f;
       if (MODE == LS_MLSTM) {
         const float4 g = tok ? *reinterpret_cast<const float4*>(a.aux + (t * H + hd) * 4) : make_float4(1.f, 0.f, 0.f, 0.f);
         pd[tw] = g.x;
@@ -1147,6 +1159,22 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
         rk = 1.f / sqrtf(warp_sum_(sk) + 1e-6f);
       }
       if (MODE == LS_MLSTM) rk = pb[tw];
+      float ssd_decay = 1.f;
+      if (MODE == LS_SSD) {
+        rk = softplus_(pb[tw] + hconst);
+        ssd_decay = expf(-rate * rk);
+      }
+      if (MODE == LS_RET) {                             // pairs (2i, 2i + 1) sit in adjacent lanes; past rdims the turn is (1, 0)
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) {
+          const float zo = __shfl_xor_sync(0xffffffffu, pz[tw][e], 1);
+          const float qo = __shfl_xor_sync(0xffffffffu, pq[tw][e], 1), ko = __shfl_xor_sync(0xffffffffu, pk[tw][e], 1);
+          const bool odd = lane & 1;
+          const float cs = odd ? zo : pz[tw][e], sn = odd ? pz[tw][e] : -zo;
+          pq[tw][e] = pq[tw][e] * cs + qo * sn;
+          pk[tw][e] = pk[tw][e] * cs + ko * sn;
+        }
+      }
 #pragma unroll
       for (int e = 0; e < EPL; ++e) {
         const int i = lane + 32 * e;
@@ -1156,6 +1184,8 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
           if (MODE == LS_GLA) d = expf(logsigmoid_(pz[tw][e] + zb[e]) * a.inv_tau);
           if (MODE == LS_DELTA) d = expf(-rate * softplus_(pz[tw][e] + zb[e]));
           if (MODE == LS_MLSTM) d = pd[tw];
+          if (MODE == LS_SSD) d = ssd_decay;
+          if (MODE == LS_RET) d = hconst;
           if (MODE == LS_HGRN2) {
             d = lob[e] + (1.f - lob[e]) * sigmoid_(pz[tw][e] + zb[e]);
             qs[tt * DKP + i] = silu_(pq[tw][e]);
@@ -1435,11 +1465,11 @@ int launch_softmax_attention(const float* q, const void* k_cache, const void* v_
                              const int* block_table, int max_pages, const int* q_start, const int* q_len,
                              const int* kv_len, int n_seqs, int max_q, int H, int G, int D, int V, int window,
                              float scale, int ldv, int f32, float softcap, int keep_first, const float* sink, int Gv,
-                             const float* slope, cudaStream_t s) {
+                             const float* slope, int out_f32, cudaStream_t s) {
   if (n_seqs <= 0 || max_q <= 0) return 0;
   if (Gv <= 0) Gv = G;
   if (Gv > H || H % Gv != 0) return -2;
-  const bool plain = Gv == G && slope == nullptr;      // (the tensor-core variant has neither option)
+  const bool plain = Gv == G && slope == nullptr && !out_f32;      // (the tensor-core variant has neither option)
   if (window <= 0) keep_first = 0;          // every earlier key is visible anyway
   if (V > 64 * SMX_VR || G <= 0 || H % G != 0) return -2;
   const bool wide_v = V > 32 * SMX_VR;      // values of 257 .. 512 channels: 16 channels per lane
@@ -1466,17 +1496,20 @@ int launch_softmax_attention(const float* q, const void* k_cache, const void* v_
 #undef B2B_SMXMMA
     return last_error();
   }
-#define B2B_SMX(CT, WPQ, VR_, GRID, BLOCK, SMEM)                                                                         \
-  launch_kernel(softmax_attention_kernel<CT, CT, WPQ, VR_>, dim3(GRID), dim3(BLOCK), SMEM, s, 1u, q,                     \
-                static_cast<const CT*>(k_cache), static_cast<const CT*>(v_cache), static_cast<CT*>(out), ld_out,        \
+#define B2B_SMX(CT, OT, WPQ, VR_, GRID, BLOCK, SMEM)                                                                         \
+  launch_kernel(softmax_attention_kernel<CT, OT, WPQ, VR_>, dim3(GRID), dim3(BLOCK), SMEM, s, 1u, q,                     \
+                static_cast<const CT*>(k_cache), static_cast<const CT*>(v_cache), static_cast<OT*>(out), ld_out,        \
                 block_table, max_pages, q_start, q_len, kv_len, H, G, D, V, window, scale, ldv, softcap, keep_first, sink, Gv, slope)
 #define B2B_SMX_T(WPQ, GRID, BLOCK, SMEM)                                                                               \
   if (f32) {                                                                                                            \
-    if (wide_v) B2B_SMX(float, WPQ, 2 * SMX_VR, GRID, BLOCK, SMEM);                                                     \
-    else B2B_SMX(float, WPQ, SMX_VR, GRID, BLOCK, SMEM);                                                                \
+    if (wide_v) B2B_SMX(float, float, WPQ, 2 * SMX_VR, GRID, BLOCK, SMEM);                                              \
+    else B2B_SMX(float, float, WPQ, SMX_VR, GRID, BLOCK, SMEM);                                                         \
+  } else if (out_f32) {                                                                                                 \
+    if (wide_v) B2B_SMX(bf16, float, WPQ, 2 * SMX_VR, GRID, BLOCK, SMEM);                                               \
+    else B2B_SMX(bf16, float, WPQ, SMX_VR, GRID, BLOCK, SMEM);                                                          \
   } else {                                                                                                              \
-    if (wide_v) B2B_SMX(bf16, WPQ, 2 * SMX_VR, GRID, BLOCK, SMEM);                                                      \
-    else B2B_SMX(bf16, WPQ, SMX_VR, GRID, BLOCK, SMEM);                                                                 \
+    if (wide_v) B2B_SMX(bf16, bf16, WPQ, 2 * SMX_VR, GRID, BLOCK, SMEM);                                                \
+    else B2B_SMX(bf16, bf16, WPQ, SMX_VR, GRID, BLOCK, SMEM);                                                           \
   }
   if (max_q <= SMX_DEC_MAX_Q) {
     dim3 grid(max_q, H, n_seqs);
@@ -1492,19 +1525,33 @@ int launch_softmax_attention(const float* q, const void* k_cache, const void* v_
   return last_error();
 }
 
+int launch_short_conv_commit(const float* x, int ld_x, int off, float* tail, const int* q_start, const int* q_len,
+                             const int* kv_len, const int* seq_slot, int n_seqs, int C, int taps, cudaStream_t s) {
+  if (n_seqs <= 0 || C <= 0 || taps <= 1) return 0;
+  const dim3 grid((C + 127) / 128, n_seqs);
+  if (taps <= 8)
+    launch_kernel(short_conv_commit_kernel<8>, grid, dim3(128), 0, s, 1u, x, ld_x, off, tail, q_start, q_len, kv_len, seq_slot, C, taps);
+  else
+    launch_kernel(short_conv_commit_kernel<CONV_MAX_TAPS>, grid, dim3(128), 0, s, 1u, x, ld_x, off, tail, q_start, q_len, kv_len,
+                  seq_slot, C, taps);
+  return last_error();
+}
+
 int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* tail, float* y, int ld_y,
                       const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs,
-                      int max_q, int C, int taps, cudaStream_t s) {
+                      int max_q, int C, int taps, const float* bias, int act, cudaStream_t s) {
   if (n_seqs <= 0 || max_q <= 0 || C <= 0) return 0;
   if (taps < 1 || taps > CONV_MAX_TAPS) return -2;
   const int tpt = 16;
   dim3 grid((C + 127) / 128, (max_q + tpt - 1) / tpt, n_seqs);
-  launch_kernel(short_conv_kernel, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail), y, ld_y,
-                q_start, q_len, kv_len, seq_slot, C, taps, tpt);
-  if (taps > 1)
-    launch_kernel(short_conv_commit_kernel, dim3((C + 127) / 128, n_seqs), dim3(128), 0, s, 1u, x, ld_x, off, tail,
-                  q_start, q_len, kv_len, seq_slot, C, taps);
-  return last_error();
+  if (taps <= 8)
+    launch_kernel(short_conv_kernel<8>, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail), y, ld_y,
+                  q_start, q_len, kv_len, seq_slot, C, taps, tpt, bias, act);
+  else
+    launch_kernel(short_conv_kernel<CONV_MAX_TAPS>, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail), y,
+                  ld_y, q_start, q_len, kv_len, seq_slot, C, taps, tpt, bias, act);
+  const int e = last_error();
+  return e ? e : launch_short_conv_commit(x, ld_x, off, tail, q_start, q_len, kv_len, seq_slot, n_seqs, C, taps, s);
 }
 
 int launch_mlstm_gates(const float* proj, int ld, int off_q, int off_k, int off_i, int off_f, const float* bi,
@@ -1562,14 +1609,16 @@ int launch_lin_scan(int mode, const float* qk, int ld_qk, int off_q, int off_k, 
                     const float* z, int ld_z, int off_z, const float* zbias, const float* hparam, const float* beta,
                     int ld_b, int off_b, const float* aux, float qscale, float inv_tau, float* state, float* out,
                     int ld_out, const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs,
-                    int max_q, int H, int G, int dk, int dv, cudaStream_t s) {
+                    int max_q, int H, int G, int dk, int dv, int rdims, cudaStream_t s) {
   if (n_seqs <= 0) return 0;
   if (G <= 0 || H % G != 0) return -2;
   ScanArgs a{qk, ld_qk, off_q, off_k, v, ld_v, off_v, z, ld_z, off_z, zbias, hparam, beta, ld_b, off_b, aux, qscale,
-             inv_tau, state, out, ld_out, q_start, q_len, kv_len, seq_slot, H, G, dk, dv};
+             inv_tau, state, out, ld_out, q_start, q_len, kv_len, seq_slot, H, G, dk, dv, rdims};
   if (mode == LS_GLA) return launch_scan_mode<LS_GLA>(a, n_seqs, max_q, s);
   if (mode == LS_DELTA) return launch_scan_mode<LS_DELTA>(a, n_seqs, max_q, s);
   if (mode == LS_MLSTM) return launch_scan_mode<LS_MLSTM>(a, n_seqs, max_q, s);
+  if (mode == LS_SSD) return launch_scan_mode<LS_SSD>(a, n_seqs, max_q, s);
+  if (mode == LS_RET) return rdims >= 0 && rdims <= dk && rdims % 2 == 0 ? launch_scan_mode<LS_RET>(a, n_seqs, max_q, s) : -2;
   if (mode == LS_HGRN2) return launch_scan_mode<LS_HGRN2>(a, n_seqs, max_q, s);
   return -2;
 }
