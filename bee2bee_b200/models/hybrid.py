@@ -1097,11 +1097,18 @@ class HybridPiece:
         kc, vc = self.k_cache[key], self.v_cache[key]
         own = sp.kv_from < 0
         tk = self._rot_tab(sp.rot)
-        q = self._buf(f"q{mx.idx}", torch.float32, 2 * H * D)[:T]
-        ops.conv_rot_prep(proj, 0, mx.f["conv"], self.conv_tail[key], self.rot_tabs[tk][3] if tk else None, sp.scale, m.slots, q,
+        fast = self.dtype == torch.bfloat16 and ops.diff_attention_supported(H, G, D, V)
+        qb = self._buf(f"q{mx.idx}", torch.bfloat16 if fast else torch.float32, 2 * H * D)
+        q = qb[:T]
+        ops.conv_rot_prep(proj, 0, mx.f["conv"], self.conv_tail[key], self.rot_tabs[tk][3] if tk else None,
+                          sp.scale * (ops.LOG2E if fast else 1.0), m.slots, q,
                           kc if own else None, vc if own else None, m.q_start, m.q_len, m.kv_len, m.seq_slot, m.n_seqs, m.max_q,
                           2 * H, 2 * G if own else 0, G if own else 0, D, V)
         ao = self._buf(f"mix{mx.idx}.{H * V}", self.dtype, mx.w_o.shape[1])[:T]
+        if fast:
+            ops.diff_attention(qb, kc, vc, ao, m.block_table, m.q_start, m.q_len, m.kv_len, m.n_seqs, m.max_q, H, G, D, V, sp.window,
+                               mx.lam, 1.0 - sp.diff, self.cfg.norm_eps)
+            return ops.linear(mx.w_o, ao, y, bias=mx.b_o)
         maps = self._buf(f"maps{mx.idx}", torch.float32, 2 * H * V)[:T]
         ops.softmax_attention(q, kc, vc, maps, m.block_table, m.q_start, m.q_len, m.kv_len, m.n_seqs, m.max_q, 2 * H, 2 * G, D, V,
                               sp.window, 1.0, v_heads=G)

@@ -37,7 +37,7 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "sig_attention", "delta_scan", "delta_post", "ls_join", "rot_attn_prep", "softmax_attention",
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
                         "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention", "sandwich_join", "rot_table",
-                        "conv_rot_prep", "diff_combine", "ssd_post", "side_gate")
+                        "conv_rot_prep", "diff_combine", "diff_attention", "ssd_post", "side_gate")
 
 
 class _CountedModule:
@@ -709,6 +709,22 @@ def diff_combine(a, lam, gain, out, T, H, G, V, eps):
     """``out[t, h] = d / rms(d) * gain``, ``d = a_1 - lam * a_2`` for map outputs ``a`` [T, 2 H V] in the order (key/value head, map,
     head of its group)"""
     native().diff_combine(a, float(lam), float(gain), out, T, H, G, V, float(eps))
+
+
+LOG2E = 1.4426950408889634
+
+
+def diff_attention_supported(H, G, D, V):
+    """whether ``diff_attention`` has a kernel for these sizes (else: ``softmax_attention`` over both maps and ``diff_combine``)"""
+    return bool(native().diff_attention_supported(int(H), int(G), int(D), int(V)))
+
+
+def diff_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, V, window, lam, gain, eps):
+    """Differential softmax attention behind ``conv_rot_prep`` on tcgen05: ``out[t, h] = d / rms(d) * gain`` with ``d`` = output of map
+    1 minus ``lam`` times that of map 2; bf16 query rows [rows, 2 H D] in the order (key/value head, map, head of its group),
+    multiplied by scale * ``LOG2E``; key rows hold 2 G heads of D channels, value rows G of V"""
+    native().diff_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_len, n_seqs, max_q, H, G, D, V, window, float(lam),
+                            float(gain), float(eps))
 
 
 def ssd_post(o, x, off_x, z, off_z, skip, w, out, T, H, V, parts, eps):

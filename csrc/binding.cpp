@@ -143,6 +143,7 @@ void set_wait_policy(int64_t abort_word, double limit_ms) {
   check(b2b::set_wait_policy_gemm(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(gemm)");
   check(b2b::set_wait_policy_elementwise(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(elementwise)");
   check(b2b::set_wait_policy_mixed(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(mixed)");
+  check(b2b::set_wait_policy_diff(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(diff)");
 }
 
 void set_pdl(bool on) { b2b::g_pdl_mode = on ? 1 : 0; }
@@ -862,6 +863,27 @@ void diff_combine(const Tensor& in, double lambda, double gain, const Tensor& ou
         "diff_combine");
 }
 
+// q [rows, 2 H D] bf16, k_cache [pages, 64, 2 G, D], v_cache [pages, 64, G, V] bf16, out [T, >= H V] bf16
+void diff_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& out, const Tensor& block_table,
+                    const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int64_t n_seqs, int64_t max_q, int64_t H,
+                    int64_t G, int64_t D, int64_t V, int64_t window, double lambda, double gain, double eps) {
+  c10::cuda::CUDAGuard guard(q.device());
+  check_bf16(q, "q");
+  check_bf16(k_cache, "k_cache");
+  check_bf16(v_cache, "v_cache");
+  check_bf16(out, "out");
+  TORCH_CHECK(q.is_contiguous() && q.size(1) == 2 * H * D && k_cache.is_contiguous() && v_cache.is_contiguous() &&
+                  k_cache.size(1) == 64 && k_cache.size(2) * k_cache.size(3) == 2 * G * D && v_cache.size(2) * v_cache.size(3) == G * V &&
+                  v_cache.size(0) == k_cache.size(0) && out.size(1) >= H * V, "diff_attention: sizes");
+  check(b2b::launch_diff_attention(q.data_ptr(), static_cast<int>(q.size(0)), k_cache.data_ptr(), v_cache.data_ptr(),
+                                   static_cast<int>(k_cache.size(0)), out.data_ptr(), static_cast<int>(out.stride(0)), ip(block_table),
+                                   static_cast<int>(block_table.stride(0)), ip(q_start), ip(q_len), ip(kv_len),
+                                   static_cast<int>(n_seqs), static_cast<int>(max_q), static_cast<int>(H), static_cast<int>(G),
+                                   static_cast<int>(D), static_cast<int>(V), static_cast<int>(window), static_cast<float>(lambda),
+                                   static_cast<float>(gain), static_cast<float>(eps), cur_stream()),
+        "diff_attention");
+}
+
 void ssd_post(const Tensor& o, const Tensor& x, int64_t off_x, const Tensor& z, int64_t off_z, const Tensor& skip, const Tensor& w,
               const Tensor& out, int64_t T, int64_t H, int64_t V, int64_t parts, double eps) {
   c10::cuda::CUDAGuard guard(o.device());
@@ -951,6 +973,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rot_table", &rot_table);
   m.def("conv_rot_prep", &conv_rot_prep);
   m.def("diff_combine", &diff_combine);
+  m.def("diff_attention", &diff_attention);
+  m.def("diff_attention_supported", &b2b::diff_attention_supported);
+  m.def("diff_attention_gave_up", &b2b::diff_attention_gave_up);
   m.def("ssd_post", &ssd_post);
   m.def("side_gate", &side_gate);
 }

@@ -185,9 +185,19 @@ int launch_ssd_post(const float* o, int ld_o, const float* x, int ld_x, const fl
 int launch_side_gate(const float* z, int ld_z, const int* ids, const void* table, int ld_t, int off, int vocab, void* out, int ld_out,
                      int n, int T, int f32, cudaStream_t s);
 
+// diff_attention.cu: two maps per head over the same values, combined and normed per head (bf16 query rows [rows, 2 H D] in the order
+// (key/value head, map, head of its group), times scale log2(e); key rows [2 G, D], value rows [G, V]); _gave_up: CTAs whose bounded
+// waits ran out so far, 0 unless there is a bug
+bool diff_attention_supported(int H, int G, int D, int V);
+unsigned diff_attention_gave_up();
+int launch_diff_attention(const void* q, int q_rows, const void* k_cache, const void* v_cache, int n_pages, void* out, int ld_out,
+                          const int* block_table, int max_pages, const int* q_start, const int* q_len, const int* kv_len, int n_seqs,
+                          int max_q, int H, int G, int D, int V, int window, float lambda, float gain, float eps, cudaStream_t s);
+
 // bounded handoff waits: device abort word + time limit for the waits of each translation unit (0 / null = trap policy)
 int set_wait_policy_gemm(uint32_t* abort_word, unsigned long long limit_ns);
 int set_wait_policy_mixed(uint32_t* abort_word, unsigned long long limit_ns);
+int set_wait_policy_diff(uint32_t* abort_word, unsigned long long limit_ns);
 int set_wait_policy_elementwise(uint32_t* abort_word, unsigned long long limit_ns);
 
 // gemm_tc.cu

@@ -333,6 +333,14 @@ def test_rotary_table_kernel_far_positions():
     assert torch.allclose(got[..., 0], torch.cos(a) * amp, atol=1e-6) and torch.allclose(got[..., 1], torch.sin(a) * amp, atol=1e-6)
 
 
+def _paged(rows, page_ids, dtype):
+    """rows [n, G, D] of one sequence -> cache [pages, 64, G, D] with the sequence's pages at ``page_ids``"""
+    cache = torch.full((max(page_ids) + 2, 64) + tuple(rows.shape[1:]), 3.0)      # other pages hold junk, not zeros
+    for j in range(rows.shape[0]):
+        cache[page_ids[j // 64], j % 64] = rows[j]
+    return cache.to("cuda", dtype)
+
+
 def _spans(lens, pos0, slots, dev="cuda"):
     """(q_start, q_len, kv_len, seq_slot) of a batch of spans"""
     i = dict(dtype=torch.int32, device=dev)
@@ -404,6 +412,101 @@ def test_convolution_rotation_and_cache_rows(Hq, Gk, Gv, D, V, half, taps):
             for s in (0, 2):
                 assert torch.equal(td[slot_of[s]].cpu(), hist[s][at[s] - taps + 1:at[s]])
             assert bool((td[[0, 2, 4]] == 7.0).all())
+
+
+def diff_reference(q, k, v, window, lam, gain, eps):
+    """q [T, H, 2, D] (times the scale), k [T, G, 2, D], v [T, G, V], float64 -> [T, H, V]"""
+    T, H = q.shape[:2]
+    G = k.shape[1]
+    ok, out = O.in_window(T, window), []
+    for h in range(H):
+        g = h // (H // G)
+        a = [torch.softmax((q[:, h, m] @ k[:, g, m].T).masked_fill(~ok, -float("inf")), -1) @ v[:, g] for m in range(2)]
+        out.append(O.rms(a[0] - lam * a[1], eps) * gain)
+    return torch.stack(out, 1)
+
+
+DIFF_SHAPES = [(4, 2, 16, 24), (8, 2, 64, 128), (3, 3, 32, 64), (6, 2, 40, 72), (5, 1, 128, 128), (16, 1, 64, 64), (1, 1, 8, 8), (12, 4, 72, 16),
+               (4, 2, 20, 24), (2, 1, 136, 40), (2, 2, 64, 136)]          # (the last three: exact kernel in both modes)
+
+
+@gpu
+@pytest.mark.parametrize("H,G,D,V", DIFF_SHAPES)
+@pytest.mark.parametrize("nq,window", [(300, 0), (300, 70), (300, 129), (2, 1), (1, 0), (1, 65), (7, 33), (129, 128), (2, 190), (1, 290)])
+def test_differential_attention_kernels(H, G, D, V, nq, window):
+    """both maps, their combination and the norm per head for the last ``nq`` of 300 positions on scattered pages, beside an idle
+    sequence and a sequence of its own length: bf16 on the tensor-core kernel (where the sizes allow), float32 on the exact one"""
+    from bee2bee_b200 import ops
+
+    n, n2, dev, lam, gain, eps = 300, 45, "cuda", 0.6, 0.7, 1e-5
+    g = torch.Generator().manual_seed(H * 100 + D + nq)
+    pages = {0: [4, 1, 6, 9, 2], 1: [7]}
+    data, want = {}, {}
+    for s, m in ((0, n), (1, n2)):
+        q, k, v = (torch.randn(m, *sh, generator=g) for sh in ((H, 2, D), (G, 2, D), (G, V)))
+        data[s] = ((q * 2.0 * D ** -0.5).bfloat16().float(), k.bfloat16().float(), v.bfloat16().float())
+        want[s] = diff_reference(*(x.double() for x in data[s]), window, lam, gain, eps)
+    lens = [nq, 0, min(nq, n2)]
+    T = sum(lens)
+    sp = _spans(lens, (n - lens[0], 0, n2 - lens[2]), (0, 0, 1))[:3]
+    bt = torch.tensor([pages[0] + [0] * 3, [0] * 8, pages[1] + [0] * 7], dtype=torch.int32, device=dev)
+    ref = torch.cat([want[0][n - lens[0]:], want[1][n2 - lens[2]:]], 0)
+    qq = torch.cat([data[0][0][n - lens[0]:], data[1][0][n2 - lens[2]:]], 0)
+    rows = qq.view(T, G, H // G, 2, D).transpose(2, 3).reshape(T, -1)           # (key/value head, map, head of the group)
+    fast = D % 8 == 0 and V % 8 == 0 and D <= 128 and V <= 128
+    assert ops.diff_attention_supported(H, G, D, V) == fast
+    for dtype, tol in ((torch.float32, 3e-5), (torch.bfloat16, 4e-2)):
+        kc = _paged(data[0][1].reshape(n, 2 * G, D), pages[0], dtype)
+        vc = _paged(data[0][2], pages[0], dtype)
+        kc[7, :n2], vc[7, :n2] = data[1][1].reshape(n2, 2 * G, D).to(dev, dtype), data[1][2].to(dev, dtype)
+        out = torch.zeros(T, (H * V + 7) // 8 * 8 + 8, device=dev, dtype=dtype)
+        if dtype == torch.bfloat16 and fast:
+            q = torch.zeros(T + 3, 2 * H * D, device=dev, dtype=dtype)
+            q[:T] = (rows * ops.LOG2E).to(dev)
+            ops.diff_attention(q, kc, vc, out, bt, *sp, 3, nq, H, G, D, V, window, lam, gain, eps)
+        else:
+            maps = torch.zeros(T, 2 * H * V, device=dev)
+            ops.softmax_attention(rows.to(dev), kc, vc, maps, bt, *sp, 3, nq, 2 * H, 2 * G, D, V, window, 1.0, v_heads=G)
+            ops.diff_combine(maps, lam, gain, out, T, H, G, V, eps)
+        got = out[:, :H * V].float().cpu().double().view(T, H, V)
+        assert torch.allclose(got, ref, atol=tol, rtol=tol), (dtype, float((got - ref).abs().max()))
+        assert float(out[:, H * V:].float().abs().max()) == 0.0
+    assert ops.native().diff_attention_gave_up() == 0
+
+
+@gpu
+@pytest.mark.parametrize("S,H,G,D,V,window", [(32, 16, 4, 64, 128, 1024), (3, 8, 2, 64, 64, 500), (1, 32, 8, 32, 64, 0), (150, 4, 1, 128, 128, 200)])
+def test_differential_attention_decode_steps(S, H, G, D, V, window):
+    """many sequences, one decoded token each at contexts around page borders: one CTA per key/value head or a cluster of them"""
+    from bee2bee_b200 import ops
+
+    dev = "cuda"
+    g = torch.Generator().manual_seed(S + D)
+    ctx = [int(v) for v in torch.randint(1, 900, (S,), generator=g)]
+    for i, v in enumerate((64, 65, 63, 1, 128, 129, 448)):
+        ctx[i % S] = v if S > 1 else 871
+    kc = torch.randn(sum((c + 63) // 64 for c in ctx) + 1, 64, 2 * G, D, generator=g).to(dev, torch.bfloat16)
+    vc = torch.randn(kc.shape[0], 64, G, V, generator=g).to(dev, torch.bfloat16)
+    perm = (torch.randperm(kc.shape[0] - 1, generator=g) + 1).tolist()
+    bt, at = torch.zeros(S, 16, dtype=torch.int32), 0
+    for i, c in enumerate(ctx):
+        m = (c + 63) // 64
+        bt[i, :m] = torch.tensor(perm[at:at + m], dtype=torch.int32)
+        at += m
+    q = (torch.randn(S, 2 * H * D, generator=g) * 2.0 * D ** -0.5).to(dev, torch.bfloat16)
+    out = torch.zeros(S, H * V, device=dev, dtype=torch.bfloat16)
+    ops.diff_attention(q, kc, vc, out, bt.to(dev), *_spans([1] * S, [c - 1 for c in ctx], list(range(S)))[:3], S, 1, H, G, D, V, window, 0.4, 0.5, 1e-6)
+    kf, vf, qf = kc.double().cpu(), vc.double().cpu(), q.double().cpu().view(S, G, 2, H // G, D) / ops.LOG2E
+    for i, c in enumerate(ctx):
+        ids = [int(b) for b in bt[i, :(c + 63) // 64]]
+        lo = max(0, c - window) if window else 0
+        k, v = (torch.cat([f[b] for b in ids], 0)[lo:c] for f in (kf, vf))
+        for g_ in range(G):
+            a = [torch.softmax(qf[i, g_, m] @ k[:, 2 * g_ + m].T, -1) @ v[:, g_] for m in range(2)]
+            want = O.rms(a[0] - 0.4 * a[1], 1e-6) * 0.5
+            got = out[i].double().cpu().view(G, H // G, V)[g_]
+            assert float((got - want).abs().max()) < 4e-2, (i, c)
+    assert ops.native().diff_attention_gave_up() == 0
 
 
 @gpu
