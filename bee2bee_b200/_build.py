@@ -23,9 +23,10 @@ CUDA_HOME = os.environ.get("CUDA_HOME", "/usr/local/cuda")
 NVCC = os.path.join(CUDA_HOME, "bin", "nvcc")
 
 CU_SOURCES = ["gemm_tc.cu", "elementwise.cu", "attention.cu", "attention_tc.cu", "sampler.cu", "hybrid.cu", "seqmix.cu", "postnorm.cu",
-              "mixed_attention.cu", "sandwich.cu", "diff_attention.cu"]
+              "mixed_attention.cu", "sandwich.cu", "diff_attention.cu",
+              "lin_chunk.cu"]
 # translation units whose arithmetic must be exact fp32 (no approximate division / exp / sqrt, no flush to zero)
-EXACT_MATH = {"hybrid.cu", "seqmix.cu", "postnorm.cu", "mixed_attention.cu", "sandwich.cu", "diff_attention.cu"}
+EXACT_MATH = {"hybrid.cu", "seqmix.cu", "postnorm.cu", "mixed_attention.cu", "sandwich.cu", "diff_attention.cu", "lin_chunk.cu"}
 CPP_SOURCES = ["peer.cpp", "binding.cpp"]
 
 NVCC_FLAGS = [

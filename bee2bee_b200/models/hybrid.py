@@ -1120,22 +1120,39 @@ class HybridPiece:
         H, G, N, V = sp.heads, sp.kv_heads, sp.dim, sp.vdim
         key, inner = self._key(mx), H * V
         cw = mx.f["conv"]
-        xbc = self._buf(f"conv{mx.idx}", torch.float32, ops.pad_to(cw.shape[0], 4))[:T]
+        chunked = self._chunked(m, N, V)              # (then everything behind the convolution is bf16, as projections are)
+        xbc = self._buf(f"conv{mx.idx}", torch.bfloat16 if chunked else torch.float32, ops.pad_to(cw.shape[0], 8))[:T]
         ops.short_conv(proj, mx.off["xbc"], cw, self.conv_tail[key], xbc, m.q_start, m.q_len, m.kv_len, m.seq_slot, m.n_seqs, m.max_q,
                        bias=mx.f["conv.b"])
         o = self._buf(f"o{mx.idx}", torch.float32, inner)[:T]
-        ops.lin_scan(ops.SCAN_SSD, xbc, inner + G * N, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len, m.seq_slot,
-                     m.n_seqs, m.max_q, H, G, N, V, zbias=mx.f["dt_bias"], hparam=mx.f["A_log"], beta=proj, off_b=mx.off["dt"])
+        if chunked:
+            ops.lin_chunk(ops.SCAN_SSD, xbc, inner + G * N, xbc, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len,
+                          m.seq_slot, m.n_seqs, H, G, N, V, step=proj, off_step=mx.off["dt"], bias=mx.f["dt_bias"], hparam=mx.f["A_log"])
+        else:
+            ops.lin_scan(ops.SCAN_SSD, xbc, inner + G * N, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len,
+                         m.seq_slot, m.n_seqs, m.max_q, H, G, N, V, zbias=mx.f["dt_bias"], hparam=mx.f["A_log"], beta=proj,
+                         off_b=mx.off["dt"])
         go = self._buf(f"mix{mx.idx}.{inner}", self.dtype, mx.w_o.shape[1])[:T]
         ops.ssd_post(o, xbc, 0, proj, mx.off["z"], mx.f["D"], mx.f["norm"], go, T, H, V, sp.norm_groups, self.cfg.norm_eps)
         return ops.linear(mx.w_o, go, y)
+
+    def _chunked(self, m, dk: int, dv: int) -> bool:
+        """whether the recurrence runs over whole chunks on tensor cores (bf16 mode, long spans)"""
+        return self.dtype == torch.bfloat16 and m.max_q >= ops.CHUNK_MIN_Q and ops.lin_chunk_supported(dk, dv)
 
     def _mix_retention(self, mx: _Mix, proj: torch.Tensor, m, y: torch.Tensor) -> torch.Tensor:
         sp, T = mx.spec, m.n_tokens
         H, D, V = sp.heads, sp.dim, sp.vdim
         tk = self._rot_tab(sp.rot)
         o = self._buf(f"o{mx.idx}", torch.float32, H * V)[:T]
-        ops.lin_scan(ops.SCAN_RETENTION, proj, mx.off["q"], mx.off["k"], proj, mx.off["v"], self.state[self._key(mx)], o, m.q_start,
-                     m.q_len, m.kv_len, m.seq_slot, m.n_seqs, m.max_q, H, H, D, V, z=self.rot_tabs[tk][3] if tk else None,
-                     hparam=mx.f["decay"], qscale=D ** -0.5, rdims=sp.rot.dims if tk else 0)
+        tab, rd, st = self.rot_tabs[tk][3] if tk else None, sp.rot.dims if tk else 0, self.state[self._key(mx)]
+        if self._chunked(m, D, V):
+            qk = self._buf(f"qk{mx.idx}", torch.bfloat16, 2 * H * D)[:T]
+            v = self._buf(f"v{mx.idx}", torch.bfloat16, H * V)[:T]
+            ops.rot_cast(proj, mx.off["q"], mx.off["v"], tab, rd, m.slots, qk, v, T, 2 * H, D)
+            ops.lin_chunk(ops.SCAN_RETENTION, qk, 0, qk, H * D, v, 0, st, o, m.q_start, m.q_len, m.kv_len, m.seq_slot, m.n_seqs, H, H, D,
+                          V, hparam=mx.f["decay"], qscale=D ** -0.5)
+        else:
+            ops.lin_scan(ops.SCAN_RETENTION, proj, mx.off["q"], mx.off["k"], proj, mx.off["v"], st, o, m.q_start, m.q_len, m.kv_len,
+                         m.seq_slot, m.n_seqs, m.max_q, H, H, D, V, z=tab, hparam=mx.f["decay"], qscale=D ** -0.5, rdims=rd)
         return self._scan_out(mx, o, proj, mx.off["g"], ops.POST_SILU, None, m, y)

@@ -37,7 +37,8 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "sig_attention", "delta_scan", "delta_post", "ls_join", "rot_attn_prep", "softmax_attention",
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
                         "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention", "sandwich_join", "rot_table",
-                        "conv_rot_prep", "diff_combine", "diff_attention", "ssd_post", "side_gate")
+                        "conv_rot_prep", "diff_combine", "diff_attention", "ssd_post", "side_gate", "rot_cast",
+                        "lin_chunk")
 
 
 class _CountedModule:
@@ -574,7 +575,8 @@ def softmax_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_
 
 def short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, bias=None, silu=True):
     """y[t, c] = silu(causal convolution of columns off .. off + C of x with w [C, taps] + bias[c]); ``tail`` [slots, taps-1, C]
-    holds the inputs before the span and receives the last ones (a second kernel, after the first has read them)"""
+    holds the inputs before the span and receives the last ones (a second kernel, after the first has read them); ``y`` float32
+    or bf16"""
     native().short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, bias, int(bool(silu)))
     if w.shape[1] > 1:
         LAUNCHES[0] += 1
@@ -592,6 +594,28 @@ def lin_scan(mode, qk, off_q, off_k, v, off_v, state, out, q_start, q_len, kv_le
     variant).  SCAN_RETENTION: ``z`` is the rotary table of the step, the first ``rdims`` channels of q and k turn."""
     native().lin_scan(mode, qk, off_q, off_k, v, off_v, z, off_z, zbias, hparam, beta, off_b, aux, float(qscale),
                       float(inv_tau), state, out, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, H, G, dk, dv, int(rdims))
+
+
+#: spans from this length on run on ``lin_chunk`` where it has a kernel (its tile is 64 tokens)
+CHUNK_MIN_Q = 32
+
+
+def lin_chunk_supported(dk, dv):
+    """whether ``lin_chunk`` has a kernel for these state sizes (else: ``lin_scan``)"""
+    return bool(native().lin_chunk_supported(int(dk), int(dv)))
+
+
+def lin_chunk(mode, q, off_q, k, off_k, v, off_v, state, out, q_start, q_len, kv_len, seq_slot, n_seqs, H, G, dk, dv, *, step=None,
+              off_step=0, bias=None, hparam=None, qscale=1.0):
+    """SCAN_SSD / SCAN_RETENTION over chunks of 64 tokens on tensor cores (bf16 rows, the fp32 states of ``lin_scan``)"""
+    native().lin_chunk(mode, q, off_q, k, off_k, v, off_v, step, off_step, bias, hparam, float(qscale), state, out, q_start, q_len, kv_len,
+                       seq_slot, n_seqs, H, G, dk, dv)
+
+
+def rot_cast(proj, off, off_v, tab, rdims, slots, qk, v, T, H2, D):
+    """bf16 rows of a recurrence: ``H2`` heads (queries, then keys) of D channels at column ``off`` with rotary positions on the first
+    ``rdims`` (pairs 2i, 2i + 1; ``tab`` [T, rdims]) -> ``qk``; the columns from ``off_v`` on -> ``v``"""
+    native().rot_cast(proj, off, off_v, tab, int(rdims), slots, qk, v, T, H2, D)
 
 
 def scan_post(o, gate, off_g, weight, act, aux, out, T, H, dv, eps):

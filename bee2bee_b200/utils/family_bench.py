@@ -3,7 +3,9 @@ next to the closest uniform decoder (Llama), or (``--family repudra``) the paral
 closest hybrid (Kepovik), or (``--family lonulix``) the post-norm Lonulix graph next to Repudra (the other family whose
 attention and recurrences run on the kernels of ``csrc/seqmix.cu``), or (``--family fisopel``) the looped Fisopel graph next
 to Lonulix (the other family with latent attention and routed experts), or (``--family kazolorn``) the depth-averaged Kazolorn
-graph next to Fisopel (the other family of parallel blocks with two norms, windowed attention and gated experts); random weights, layer shapes of real models.
+graph next to Fisopel (the other family of parallel blocks with two norms, windowed attention and gated experts), or (``--family
+nipudra``) the sandwich-norm Nipudra graph next to Lonulix (the other sequential hybrid: windowed attention, a linear recurrence,
+routed experts without a gate); random weights, layer shapes of real models.
 
 Per width it reports (1) prefill and decode tokens/s through the same ``GpuRunner`` calls that serving uses (chunked
 graph prefill, CUDA-graph decode steps), timed with CUDA events, and (2) a per-kernel breakdown of one eager prefill
@@ -161,6 +163,38 @@ def kazolorn_sized(width: int, vocab: int = 32000) -> ModelConfig:
                        depth_average=True)
 
 
+def nipudra_sized(width: int, vocab: int = 32000) -> ModelConfig:
+    """six sandwich-norm layers: differential attention (width / 128 heads of two 64-channel maps over 128 value channels, grouped 4:1,
+    window 1024, 4 taps), mamba2 (width / 32 heads of 64 channels, 128 state channels, one group), retention (width / 128 heads of
+    128), the same three again with the first layer's keys and values in the second attention; every layer has 8 experts of 15
+    width / 64 hidden channels (2 per token) beside a gated shared one and a token input of 128 channels.  The layer matrices
+    hold about 53 width^2 parameters, as ``lonulix_sized(width)`` does."""
+    H, eff = width // 128, 15 * width // 64
+
+    def routed(sp):
+        sp.ff_kind, sp.experts, sp.expert_ff, sp.top, sp.shared_ff = "moe", 8, eff, 2, eff
+        sp.route_kind, sp.ff_act, sp.router_bias, sp.shared_gate, sp.ff = "logit_topk", "relu_sq", True, True, 9 * eff
+        return sp
+
+    def att(src):
+        rot = RotarySpec(dims=64, base=500000.0, factor=4.0, original=8192, half=True)
+        return routed(LayerSpec(mixer="diff_attention", heads=H, kv_heads=max(1, H // 4), dim=64, vdim=128, scale=64 ** -0.5, window=1024,
+                                rot=rot, qk_norm="none", v_norm=False, proj_bias=True, conv=4, diff=0.4, kv_from=src))
+
+    def mamba():
+        return routed(LayerSpec(mixer="mamba2", heads=width // 32, kv_heads=1, dim=128, vdim=64, conv=4, norm_groups=1))
+
+    def ret():
+        return routed(LayerSpec(mixer="retention", heads=H, kv_heads=H, dim=128, vdim=128, rot=RotarySpec(dims=128, base=10000.0, half=True),
+                                decay=tuple(1.0 - 2.0 ** (-5.0 - 6.0 * i / max(1, H - 1)) for i in range(H))))
+
+    specs = (att(-1), mamba(), ret(), att(0), mamba(), ret())
+    return ModelConfig(name=f"mini-nipudra-{width}", family="nipudra", vocab_size=vocab, hidden_size=width, n_layers=len(specs), n_heads=H,
+                       n_kv_heads=max(1, H // 4), head_dim=128, ffn_size=9 * eff, max_position=1 << 30, norm="ln", norm_eps=1e-5,
+                       act="relu_sq", glu=False, rope_theta=0.0, tie_embeddings=True, embed_scale=width ** 0.5, final_softcap=30.0,
+                       logit_scale=0.5, layer_specs=specs, block_layout="sandwich", token_side=128)
+
+
 def llama_sized(width: int, layer_params: int, n_layers: int = 4, vocab: int = 32000) -> ModelConfig:
     """Llama layers (GQA 4:1, SwiGLU) whose matrices hold about ``layer_params`` parameters in ``n_layers`` layers"""
     H = width // 128
@@ -312,7 +346,7 @@ def cost(name: str, a, hint: Dict):
     if name == "poly_norm":
         return 0.0, T * a[4] * (4 + a[3].element_size()), False
     if name == "short_conv":
-        return 0.0, 2 * T * a[2].shape[0] * 4, False
+        return 0.0, T * a[2].shape[0] * (4 + a[4].element_size()), False
     if name == "mlstm_gates":
         H, dk = a[17], a[18]
         return 4.0 * T * H * dk, T * H * (2 * dk + 6) * 4 + 2 * S * H * dk * 4, False
@@ -341,6 +375,33 @@ def cost(name: str, a, hint: Dict):
         Tn, H, V, C = a[5], a[6], a[7], a[8]
         elt = a[0].element_size()
         return 2.0 * Tn * H * V * C, Tn * H * C * elt + H * V * C * elt + Tn * H * V * ((4 if a[2] is not None else 0) + elt), False
+    if name == "sandwich_join":
+        W, rows, gathered = a[0].shape[-1], a[2], a[1] is not None
+        return 0.0, rows * W * 4 * ((2 if a[3] is not None and not gathered else 1) + (1 if a[3] is not None else 0)) + \
+            (rows * W * a[11].element_size() if a[11] is not None else 0), False
+    if name == "rot_table":
+        return 0.0, T * a[4].shape[-1] * 4, False
+    if name == "conv_rot_prep":
+        Hq, Gk, Gv, D, V = a[16], a[17], a[18], a[19], a[20]
+        C, tail = (Hq + Gk) * D + Gv * V, 2 * S * (a[2].shape[1] - 1) * a[2].shape[0] * 4
+        return 0.0, T * C * 4 + T * Hq * D * a[7].element_size() + (T * (Gk * D + Gv * V) * a[8].element_size() if Gk else 0) + tail, False
+    if name == "diff_attention":
+        H, G, D, V = a[10], a[11], a[12], a[13]
+        keys, span = visible_keys(hint, a[14], 0)
+        return 4.0 * H * (D + V) * keys, S * span * G * (2 * D + V) * 2 + T * H * (2 * D + V) * 2, q >= 16
+    if name == "diff_combine":
+        H, V = a[5], a[7]
+        return 0.0, T * H * V * (8 + a[3].element_size()), False
+    if name == "rot_cast":
+        return 0.0, T * (a[9] * a[10] + a[7].shape[1]) * 6, False
+    if name == "lin_chunk":
+        H, G, dk, dv = a[19], a[20], a[21], a[22]
+        return 6.0 * T * H * dk * dv, 2 * S * H * dk * dv * 4 + T * (2 * G * dk * 2 + H * dv * (2 + 4)), True
+    if name == "ssd_post":
+        H, V = a[9], a[10]
+        return 0.0, T * H * V * (4 + a[1].element_size() + 4 + a[7].element_size()), False
+    if name == "side_gate":
+        return 0.0, T * a[5] * (4 + a[2].element_size() + a[4].element_size()), False
     if name in ("rmsnorm", "layernorm", "add"):
         return 0.0, 3 * _nb(a[0]), False
     if name == "embed":
@@ -470,7 +531,9 @@ def run(widths, prompt_len=2048, batch=32, steps=32, warmup=3, ctx=512, device="
     out = []
     for w in widths:
         kep = kepovik_sized(w)
-        if family == "kazolorn":
+        if family == "nipudra":
+            pair = (nipudra_sized(w), lonulix_sized(w))
+        elif family == "kazolorn":
             pair = (kazolorn_sized(w), fisopel_sized(w))
         elif family == "fisopel":
             pair = (fisopel_sized(w), lonulix_sized(w))

@@ -649,10 +649,10 @@ void short_conv(const Tensor& x, int64_t off, const Tensor& w, const Tensor& tai
   c10::cuda::CUDAGuard guard(x.device());
   TORCH_CHECK(!(bias.has_value() && bias->defined()) || bias->numel() == w.size(0), "short_conv: one bias per channel");
   check(b2b::launch_short_conv(fp(x), static_cast<int>(x.stride(0)), static_cast<int>(off), fp(w),
-                               const_cast<float*>(fp(tail)), const_cast<float*>(fp(y)), static_cast<int>(y.stride(0)),
+                               const_cast<float*>(fp(tail)), y.data_ptr(), static_cast<int>(y.stride(0)),
                                ip(q_start), ip(q_len), ip(kv_len), ip(seq_slot), static_cast<int>(n_seqs),
                                static_cast<int>(max_q), static_cast<int>(w.size(0)), static_cast<int>(w.size(1)),
-                               fp_or_null(bias), static_cast<int>(act), cur_stream()),
+                               fp_or_null(bias), static_cast<int>(act), is_f32(y), cur_stream()),
         "short_conv");
 }
 
@@ -888,11 +888,50 @@ void ssd_post(const Tensor& o, const Tensor& x, int64_t off_x, const Tensor& z, 
               const Tensor& out, int64_t T, int64_t H, int64_t V, int64_t parts, double eps) {
   c10::cuda::CUDAGuard guard(o.device());
   TORCH_CHECK(skip.numel() == H && w.numel() == H * V && out.size(-1) >= H * V, "ssd_post: sizes");
-  check(b2b::launch_ssd_post(fp(o), static_cast<int>(o.stride(0)), fp(x) + off_x, static_cast<int>(x.stride(0)), fp(z) + off_z,
+  const void* xp = is_f32(x) ? static_cast<const void*>(fp(x) + off_x) : static_cast<const void*>(static_cast<const char*>(x.data_ptr()) + 2 * off_x);
+  check(b2b::launch_ssd_post(fp(o), static_cast<int>(o.stride(0)), xp, is_f32(x), static_cast<int>(x.stride(0)), fp(z) + off_z,
                              static_cast<int>(z.stride(0)), fp(skip), fp(w), out.data_ptr(), static_cast<int>(out.stride(0)),
                              static_cast<int>(T), static_cast<int>(H), static_cast<int>(V), static_cast<int>(parts),
                              static_cast<float>(eps), is_f32(out), cur_stream()),
         "ssd_post");
+}
+
+// proj columns off ..: H2 heads of D channels (queries, then keys), off_v ..: nv columns; qk [T, H2 * D], v [T, nv] bf16
+void rot_cast(const Tensor& proj, int64_t off, int64_t off_v, const OptT& tab, int64_t rdims, const Tensor& slots, const Tensor& qk,
+              const Tensor& v, int64_t T, int64_t H2, int64_t D) {
+  c10::cuda::CUDAGuard guard(proj.device());
+  check_bf16(qk, "qk");
+  check_bf16(v, "v");
+  TORCH_CHECK(qk.is_contiguous() && qk.size(1) == H2 * D && v.is_contiguous() && slots.numel() >= T, "rot_cast: dense rows");
+  TORCH_CHECK(rdims == 0 || (tab.has_value() && tab->defined() && tab->is_contiguous() && tab->size(-1) == rdims), "rot_cast: table");
+  check(b2b::launch_rot_cast(fp(proj), static_cast<int>(proj.stride(0)), static_cast<int>(off), static_cast<int>(off_v), fp_or_null(tab),
+                             static_cast<int>(rdims), ip(slots), qk.data_ptr(), v.data_ptr(), static_cast<int>(T), static_cast<int>(H2),
+                             static_cast<int>(D), static_cast<int>(v.size(1)), cur_stream()),
+        "rot_cast");
+}
+
+// q, k, v: bf16 rows with first columns off_*; mode as in lin_scan (4 state-space, 5 retention)
+void lin_chunk(int64_t mode, const Tensor& q, int64_t off_q, const Tensor& k, int64_t off_k, const Tensor& v, int64_t off_v, const OptT& step,
+               int64_t off_step, const OptT& bias, const Tensor& hparam, double qscale, const Tensor& state, const Tensor& out,
+               const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, const Tensor& seq_slot, int64_t n_seqs, int64_t H,
+               int64_t G, int64_t dk, int64_t dv) {
+  c10::cuda::CUDAGuard guard(q.device());
+  check_bf16(q, "q");
+  check_bf16(k, "k");
+  check_bf16(v, "v");
+  const bool ssd = mode == 4;
+  TORCH_CHECK(mode == 4 || mode == 5, "lin_chunk: one decay per head and token");
+  TORCH_CHECK(!ssd || (fp_or_null(step) != nullptr && fp_or_null(bias) != nullptr), "lin_chunk: step sizes");
+  TORCH_CHECK(hparam.numel() >= H && off_q + (ssd ? G : H) * dk <= q.size(1) && off_k + (ssd ? G : H) * dk <= k.size(1) &&
+                  off_v + H * dv <= v.size(1) && out.size(1) >= H * dv, "lin_chunk: sizes");
+  auto at = [](const Tensor& t, int64_t off) { return static_cast<const void*>(static_cast<const char*>(t.data_ptr()) + 2 * off); };
+  check(b2b::launch_lin_chunk(ssd ? 1 : 0, at(q, off_q), static_cast<int>(q.stride(0)), at(k, off_k), static_cast<int>(k.stride(0)), at(v, off_v),
+                              static_cast<int>(v.stride(0)), ssd ? fp(*step) + off_step : nullptr, ssd ? static_cast<int>(step->stride(0)) : 0,
+                              fp_or_null(bias), fp(hparam), static_cast<float>(qscale), const_cast<float*>(fp(state)),
+                              const_cast<float*>(fp(out)), static_cast<int>(out.stride(0)), ip(q_start), ip(q_len), ip(kv_len), ip(seq_slot),
+                              static_cast<int>(n_seqs), static_cast<int>(H), static_cast<int>(G), static_cast<int>(dk),
+                              static_cast<int>(dv), cur_stream()),
+        "lin_chunk");
 }
 
 void side_gate(const Tensor& z, const Tensor& ids, const Tensor& table, int64_t off, const Tensor& out, int64_t n, int64_t T) {
@@ -978,4 +1017,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("diff_attention_gave_up", &b2b::diff_attention_gave_up);
   m.def("ssd_post", &ssd_post);
   m.def("side_gate", &side_gate);
+  m.def("rot_cast", &rot_cast);
+  m.def("lin_chunk", &lin_chunk);
+  m.def("lin_chunk_supported", &b2b::lin_chunk_supported);
 }

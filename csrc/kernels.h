@@ -117,9 +117,9 @@ int launch_softmax_attention(const float* q, const void* k_cache, const void* v_
                              const int* kv_len, int n_seqs, int max_q, int H, int G, int D, int V, int window,
                              float scale, int ldv, int f32, float softcap, int keep_first, const float* sink, int Gv,
                              const float* slope, int out_f32, cudaStream_t s);
-int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* tail, float* y, int ld_y,
+int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* tail, void* y, int ld_y,
                       const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs,
-                      int max_q, int C, int taps, const float* bias, int act, cudaStream_t s);
+                      int max_q, int C, int taps, const float* bias, int act, int y_f32, cudaStream_t s);
 int launch_short_conv_commit(const float* x, int ld_x, int off, float* tail, const int* q_start, const int* q_len,
                              const int* kv_len, const int* seq_slot, int n_seqs, int C, int taps, cudaStream_t s);
 int launch_mlstm_gates(const float* proj, int ld, int off_q, int off_k, int off_i, int off_f, const float* bi,
@@ -180,7 +180,9 @@ int launch_conv_rot_prep(const float* proj, int ld, int off, const float* w, flo
                          int D, int V, int taps, cudaStream_t s);
 int launch_diff_combine(const float* in, int ld_in, float lambda, float gain, void* out, int ld_out, int T, int H, int G, int V,
                         float eps, int f32, cudaStream_t s);
-int launch_ssd_post(const float* o, int ld_o, const float* x, int ld_x, const float* z, int ld_z, const float* skip, const float* w,
+int launch_rot_cast(const float* proj, int ld, int off, int off_v, const float* tab, int rdims, const int* slots, void* qk, void* v, int T,
+                    int H2, int D, int nv, cudaStream_t s);
+int launch_ssd_post(const float* o, int ld_o, const void* x, int x_f32, int ld_x, const float* z, int ld_z, const float* skip, const float* w,
                     void* out, int ld_out, int T, int H, int V, int parts, float eps, int f32, cudaStream_t s);
 int launch_side_gate(const float* z, int ld_z, const int* ids, const void* table, int ld_t, int off, int vocab, void* out, int ld_out,
                      int n, int T, int f32, cudaStream_t s);
@@ -193,6 +195,13 @@ unsigned diff_attention_gave_up();
 int launch_diff_attention(const void* q, int q_rows, const void* k_cache, const void* v_cache, int n_pages, void* out, int ld_out,
                           const int* block_table, int max_pages, const int* q_start, const int* q_len, const int* kv_len, int n_seqs,
                           int max_q, int H, int G, int D, int V, int window, float lambda, float gain, float eps, cudaStream_t s);
+
+// lin_chunk.cu: the recurrences with one decay per head and token (lin_scan modes 4 and 5) over chunks of a span on tensor cores: bf16
+// q / k / v rows (pointers at their first column), fp32 states shared with lin_scan
+bool lin_chunk_supported(int dk, int dv);
+int launch_lin_chunk(int ssd, const void* q, int ld_q, const void* k, int ld_k, const void* v, int ld_v, const float* step, int ld_step,
+                     const float* bias, const float* hparam, float qscale, float* state, float* out, int ld_out, const int* q_start,
+                     const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs, int H, int G, int dk, int dv, cudaStream_t s);
 
 // bounded handoff waits: device abort word + time limit for the waits of each translation unit (0 / null = trap policy)
 int set_wait_policy_gemm(uint32_t* abort_word, unsigned long long limit_ns);

@@ -5,6 +5,7 @@
 //                      plain copy of the residual as the operand of a matrix product
 //   * rot_table        cos and sin of every rotary pair of every token of a step, once per distinct set of frequencies
 //   * conv_rot_prep    short causal convolutions on q, k and v, rotary positions (pairs i, i + half), K / V rows into the cache
+//   * rot_cast         rotary positions (pairs 2i, 2i + 1) on q and k of a recurrence, bf16 rows of q, k and v
 //   * diff_combine     differential attention: a_1 - lambda a_2 of a head's two maps, divided by its root mean square
 //   * ssd_post         (recurrence output + D x) * silu(z), RMS norm in equal parts, weight -> operand
 //   * side_gate        gelu(z) * the token's own channels for this layer -> operand
@@ -319,6 +320,31 @@ __global__ void __launch_bounds__(128)
   }
 }
 
+// ------------------------------------------------------------------------------------------- rotated bf16 rows of a recurrence
+// columns off .. of proj: H2 heads of D channels (queries, then keys) whose first rdims channels turn in adjacent pairs (2i, 2i + 1) by
+// tab [T, rdims] -> qk [T, H2 * D]; columns off_v .. off_v + nv -> v [T, nv].  Four columns per thread (D and nv multiples of 4).
+__global__ void __launch_bounds__(256)
+    rot_cast_kernel(const float* __restrict__ proj, int ld, int off, int off_v, const float* __restrict__ tab, int rdims,
+                    const int* __restrict__ slots, bf16* __restrict__ qk, bf16* __restrict__ v, int H2, int D, int nv) {
+  pdl_begin();
+  const size_t t = blockIdx.y;
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4, nqk = H2 * D;
+  if (c >= nqk + nv || slots[t] < 0) return;
+  if (c >= nqk) {
+    st4(v + t * nv + (c - nqk), *reinterpret_cast<const float4*>(proj + t * ld + off_v + (c - nqk)));
+    return;
+  }
+  float4 x = *reinterpret_cast<const float4*>(proj + t * ld + off + c);
+  const int d = c % D;
+  if (d < rdims) {
+    const float2 a = *reinterpret_cast<const float2*>(tab + t * rdims + d);
+    float2 b = make_float2(1.f, 0.f);
+    if (d + 2 < rdims) b = *reinterpret_cast<const float2*>(tab + t * rdims + d + 2);
+    x = make_float4(x.x * a.x - x.y * a.y, x.y * a.x + x.x * a.y, x.z * b.x - x.w * b.y, x.w * b.x + x.z * b.y);
+  }
+  st4(qk + t * nqk + c, x);
+}
+
 // ------------------------------------------------------------------------------------------- differential attention: the two maps
 // in [T, 2 H V] fp32: map outputs in the order (key/value head, map, head of its group); out[t, h, :] = d / rms(d) * gain with
 // d = a_1 - lambda a_2.  One warp per (token, head).
@@ -346,9 +372,15 @@ __global__ void __launch_bounds__(128)
 // ------------------------------------------------------------------------------------------- state-space output
 // out[t, c] = v / rms(part of c) * w[c] with v = (o[t, c] + skip[c / V] x[t, c]) * silu(z[t, c]), c < n = heads * V, the root mean
 // square taken over `parts` equal consecutive parts.  One block per (token, part); the part is kept in shared memory.
-template <typename OT, bool VEC>
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename OT, typename XT, bool VEC>
 __global__ void __launch_bounds__(256)
-    ssd_post_kernel(const float* __restrict__ o, int ld_o, const float* __restrict__ x, int ld_x, const float* __restrict__ z, int ld_z,
+    ssd_post_kernel(const float* __restrict__ o, int ld_o, const XT* __restrict__ x, int ld_x, const float* __restrict__ z, int ld_z,
                     const float* __restrict__ skip, const float* __restrict__ w, OT* __restrict__ out, int ld_out, int n, int V,
                     int parts, float eps) {
   pdl_begin();
@@ -357,12 +389,12 @@ __global__ void __launch_bounds__(256)
   const size_t t = blockIdx.x;
   const int np = n / parts, c0 = blockIdx.y * np;
   const float* orow = o + t * ld_o + c0;
-  const float* xrow = x + t * ld_x + c0;
+  const XT* xrow = x + t * ld_x + c0;
   const float* zrow = z + t * ld_z + c0;
   float ss = 0.f;
   if constexpr (VEC) {
     for (int c = 4 * threadIdx.x; c < np; c += 4 * blockDim.x) {
-      const float4 ov = *reinterpret_cast<const float4*>(orow + c), xv = *reinterpret_cast<const float4*>(xrow + c),
+      const float4 ov = *reinterpret_cast<const float4*>(orow + c), xv = ld4(xrow + c),
                    zv = *reinterpret_cast<const float4*>(zrow + c);
       const float D = skip[(c0 + c) / V];
       const float4 v = make_float4((ov.x + D * xv.x) * silu_(zv.x), (ov.y + D * xv.y) * silu_(zv.y), (ov.z + D * xv.z) * silu_(zv.z),
@@ -372,7 +404,7 @@ __global__ void __launch_bounds__(256)
     }
   } else {
     for (int c = threadIdx.x; c < np; c += blockDim.x) {
-      const float v = (orow[c] + skip[(c0 + c) / V] * xrow[c]) * silu_(zrow[c]);
+      const float v = (orow[c] + skip[(c0 + c) / V] * ldf(xrow, c)) * silu_(zrow[c]);
       ss += v * v;
       row[c] = v;
     }
@@ -492,6 +524,16 @@ int launch_conv_rot_prep(const float* proj, int ld, int off, const float* w, flo
   return last_error();
 }
 
+int launch_rot_cast(const float* proj, int ld, int off, int off_v, const float* tab, int rdims, const int* slots, void* qk, void* v, int T,
+                    int H2, int D, int nv, cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (D % 4 != 0 || nv % 4 != 0 || ld % 4 != 0 || off % 4 != 0 || off_v % 4 != 0 || !al16(proj) || rdims % 2 != 0 || rdims > D || T > 65535) return -2;
+  const int cols = H2 * D + nv;
+  launch_kernel(rot_cast_kernel, dim3((cols / 4 + 255) / 256, T), dim3(256), 0, s, 1u, proj, ld, off, off_v, tab, rdims, slots,
+                static_cast<bf16*>(qk), static_cast<bf16*>(v), H2, D, nv);
+  return last_error();
+}
+
 int launch_diff_combine(const float* in, int ld_in, float lambda, float gain, void* out, int ld_out, int T, int H, int G, int V,
                         float eps, int f32, cudaStream_t s) {
   const long long warps = static_cast<long long>(T) * H;
@@ -507,7 +549,7 @@ int launch_diff_combine(const float* in, int ld_in, float lambda, float gain, vo
   return last_error();
 }
 
-int launch_ssd_post(const float* o, int ld_o, const float* x, int ld_x, const float* z, int ld_z, const float* skip, const float* w,
+int launch_ssd_post(const float* o, int ld_o, const void* x, int x_f32, int ld_x, const float* z, int ld_z, const float* skip, const float* w,
                     void* out, int ld_out, int T, int H, int V, int parts, float eps, int f32, cudaStream_t s) {
   const int n = H * V;
   if (T <= 0 || n <= 0) return 0;
@@ -519,19 +561,23 @@ int launch_ssd_post(const float* o, int ld_o, const float* x, int ld_x, const fl
                    al16(z) && al16(w) && al16(out);
   int threads = ((vec ? np / 4 : np) + 31) / 32 * 32;
   if (threads > 256) threads = 256;
-#define B2B_SP(OT, VEC)                                                                                                  \
+  if (f32 && !x_f32) return -2;
+#define B2B_SP(OT, XT, VEC)                                                                                              \
   do {                                                                                                                   \
     if (smem > 48 * 1024)                                                                                                \
-      cudaFuncSetAttribute(ssd_post_kernel<OT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)); \
-    launch_kernel(ssd_post_kernel<OT, VEC>, dim3(T, parts), dim3(threads), smem, s, 1u, o, ld_o, x, ld_x, z, ld_z, skip, w, \
-                  static_cast<OT*>(out), ld_out, n, V, parts, eps);                                                      \
+      cudaFuncSetAttribute(ssd_post_kernel<OT, XT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)); \
+    launch_kernel(ssd_post_kernel<OT, XT, VEC>, dim3(T, parts), dim3(threads), smem, s, 1u, o, ld_o, static_cast<const XT*>(x), ld_x, z, \
+                  ld_z, skip, w, static_cast<OT*>(out), ld_out, n, V, parts, eps);                                       \
   } while (0)
   if (f32) {
-    if (vec) B2B_SP(float, true);
-    else B2B_SP(float, false);
+    if (vec) B2B_SP(float, float, true);
+    else B2B_SP(float, float, false);
+  } else if (x_f32) {
+    if (vec) B2B_SP(bf16, float, true);
+    else B2B_SP(bf16, float, false);
   } else {
-    if (vec) B2B_SP(bf16, true);
-    else B2B_SP(bf16, false);
+    if (vec) B2B_SP(bf16, bf16, true);
+    else B2B_SP(bf16, bf16, false);
   }
 #undef B2B_SP
   return last_error();

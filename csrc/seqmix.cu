@@ -789,10 +789,10 @@ __global__ void __launch_bounds__(32 * SMX_MMA_WARPS, 3)
 // grid (channel blocks, token groups, sequences); a thread walks `tpt` tokens of one channel with the window in registers.
 constexpr int CONV_MAX_TAPS = 32;      // (MT: taps the registers of an instance hold)
 
-template <int MT>
+template <int MT, typename YT>
 __global__ void __launch_bounds__(128)
     short_conv_kernel(const float* __restrict__ x, int ld_x, int off, const float* __restrict__ w,
-                      const float* __restrict__ tail, float* __restrict__ y, int ld_y, const int* __restrict__ q_start,
+                      const float* __restrict__ tail, YT* __restrict__ y, int ld_y, const int* __restrict__ q_start,
                       const int* __restrict__ q_len, const int* __restrict__ kv_len, const int* __restrict__ seq_slot,
                       int C, int taps, int tpt, const float* __restrict__ bias, int act) {
   pdl_begin();
@@ -827,7 +827,7 @@ __global__ void __launch_bounds__(128)
         acc += wr[j] * cur;
       }
     }
-    y[static_cast<size_t>(t0 + i) * ld_y + c] = act ? silu_(acc) : acc;
+    stf(y, static_cast<size_t>(t0 + i) * ld_y + c, act ? silu_(acc) : acc);
   }
 }
 
@@ -1537,19 +1537,24 @@ int launch_short_conv_commit(const float* x, int ld_x, int off, float* tail, con
   return last_error();
 }
 
-int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* tail, float* y, int ld_y,
+int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* tail, void* y, int ld_y,
                       const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs,
-                      int max_q, int C, int taps, const float* bias, int act, cudaStream_t s) {
+                      int max_q, int C, int taps, const float* bias, int act, int y_f32, cudaStream_t s) {
   if (n_seqs <= 0 || max_q <= 0 || C <= 0) return 0;
   if (taps < 1 || taps > CONV_MAX_TAPS) return -2;
   const int tpt = 16;
   dim3 grid((C + 127) / 128, (max_q + tpt - 1) / tpt, n_seqs);
-  if (taps <= 8)
-    launch_kernel(short_conv_kernel<8>, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail), y, ld_y,
-                  q_start, q_len, kv_len, seq_slot, C, taps, tpt, bias, act);
-  else
-    launch_kernel(short_conv_kernel<CONV_MAX_TAPS>, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail), y,
-                  ld_y, q_start, q_len, kv_len, seq_slot, C, taps, tpt, bias, act);
+#define B2B_SC(MT, YT)                                                                                                   \
+  launch_kernel(short_conv_kernel<MT, YT>, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail),  \
+                static_cast<YT*>(y), ld_y, q_start, q_len, kv_len, seq_slot, C, taps, tpt, bias, act)
+  if (y_f32) {
+    if (taps <= 8) B2B_SC(8, float);
+    else B2B_SC(CONV_MAX_TAPS, float);
+  } else {
+    if (taps <= 8) B2B_SC(8, bf16);
+    else B2B_SC(CONV_MAX_TAPS, bf16);
+  }
+#undef B2B_SC
   const int e = last_error();
   return e ? e : launch_short_conv_commit(x, ld_x, off, tail, q_start, q_len, kv_len, seq_slot, n_seqs, C, taps, s);
 }

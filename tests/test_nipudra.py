@@ -153,7 +153,7 @@ def rel_err(got, want):
     return np.sqrt((d ** 2).mean(-1)) / want.std()
 
 
-TOL = {torch.float32: 1e-4, torch.bfloat16: 6e-2}
+TOL = {torch.float32: 1e-4, torch.bfloat16: 8e-2}         # (bf16: a_1 - lambda a_2 is a small difference at some positions, and then normed)
 
 
 def routed(cfg):
@@ -521,8 +521,10 @@ def test_short_convolution_with_bias(taps):
     for silu in (True, False):
         tail, got, at = torch.full((2, max(1, taps - 1), C), 5.0, device=dev), [], 0
         for n in (3, 1, 25, 2, 1, 28):
-            y = torch.zeros(n, 40, device=dev)
-            ops.short_conv(x[at:at + n].to(dev).contiguous(), 0, w.to(dev), tail, y, *_spans((n,), (at,), (1,)), 1, n, bias=b.to(dev), silu=silu)
+            y, yb = torch.zeros(n, 40, device=dev), torch.zeros(n, 40, device=dev, dtype=torch.bfloat16)
+            for t, o in ((tail.clone(), yb), (tail, y)):
+                ops.short_conv(x[at:at + n].to(dev).contiguous(), 0, w.to(dev), t, o, *_spans((n,), (at,), (1,)), 1, n, bias=b.to(dev), silu=silu)
+            assert torch.equal(yb, y.bfloat16())
             got.append(y[:, :C].cpu().double())
             at += n
         assert torch.allclose(torch.cat(got), O.silu(want) if silu else want, atol=2e-5)
@@ -591,6 +593,86 @@ def test_retention_scan(H, D, V, rot):
     got = torch.cat(got)
     assert torch.allclose(got, want, atol=2e-4, rtol=1e-4), float((got - want).abs().max())
     assert bool((state[0] == 9.0).all())
+
+
+@gpu
+@pytest.mark.parametrize("H,G,N,V", [(4, 2, 16, 24), (3, 3, 64, 32), (8, 1, 48, 64), (2, 1, 128, 72), (5, 5, 200, 16), (2, 2, 256, 8)])
+@pytest.mark.parametrize("ssd", [True, False])
+def test_chunked_recurrences_keep_fp32_precision(H, G, N, V, ssd):
+    """spans of many lengths (whole chunks, ragged ones, two tokens) of one sequence beside an idle and a short one, single tokens in
+    between through the token-by-token kernel on the same states.  q, k and v are bf16 numbers here, so the result must be as exact as
+    in fp32: weighted scores, weighted keys and the state keep their low parts.  Strong and weak decays side by side."""
+    from bee2bee_b200 import ops
+
+    dev = "cuda"
+    g = torch.Generator().manual_seed(N + V + ssd)
+    if not ssd:
+        G = H
+    T, T2 = 330, 70
+    rows, want = {}, {}
+    alog, bias = torch.linspace(-6.0, 1.5, H), torch.randn(H, generator=g) - 1
+    decay = [0.5 + 0.4999 * h / max(1, H - 1) for h in range(H)]
+    qs = 1.0 if ssd else N ** -0.5
+    for s, m in ((0, T), (2, T2)):
+        q, k, v = ((torch.randn(m, n, f, generator=g) * sc).bfloat16().float() for n, f, sc in ((G, N, N ** -0.25), (G, N, 1.0 + N ** -0.25), (H, V, 1.0)))
+        dt = torch.randn(m, H + 1, generator=g)
+        step = torch.nn.functional.softplus((dt[:, 1:] + bias).double())
+        rows[s] = (q, k, v, dt)
+        want[s] = torch.cat([O.ssd_walk(v[:, h].double(), k[:, h // (H // G)].double(), q[:, h // (H // G)].double(), step[:, h],
+                                        torch.exp(alog[h].double()), 0.0) if ssd else
+                             O.decayed_walk(q[:, h].double(), k[:, h].double(), v[:, h].double(), decay[h]) * qs for h in range(H)], -1)
+    hp = (alog if ssd else torch.tensor(decay)).to(dev)
+    state, at, got = torch.full((4, H, N, V), 9.0, device=dev), {0: 0, 2: 0}, {0: [], 2: []}
+    for lens in ((64, 0, 2), (1, 0, 1), (100, 0, 33), (2, 0, 1), (1, 0, 1), (128, 0, 32), (34, 0, 0)):
+        parts = [[x[at[s]:at[s] + n] for x in rows[s]] for s, n in ((0, lens[0]), (2, lens[2]))]
+        q, k, v, dt = (torch.cat([a, b]).flatten(1).to(dev) for a, b in zip(*parts))
+        sp = _spans(lens, (at[0], 0, at[2]), (3, 0, 1))
+        o = torch.zeros(sum(lens), H * V, device=dev)
+        src = torch.cat([q, k, v], 1)
+        if max(lens) > 1:
+            b = torch.cat([torch.zeros(src.shape[0], 8, device=dev), src], 1).bfloat16()
+            b = torch.cat([b, torch.zeros(b.shape[0], (-b.shape[1]) % 8, device=dev, dtype=b.dtype)], 1).contiguous()
+            ops.lin_chunk(ops.SCAN_SSD if ssd else ops.SCAN_RETENTION, b, 8, b, 8 + G * N, b, 8 + 2 * G * N, state, o, *sp, 3, H, G, N, V,
+                          step=dt if ssd else None, off_step=1, bias=bias.to(dev) if ssd else None, hparam=hp, qscale=qs)
+        else:
+            ops.lin_scan(ops.SCAN_SSD if ssd else ops.SCAN_RETENTION, src, 0, G * N, src, 2 * G * N, state, o, *sp, 3, max(lens), H, G, N, V,
+                         zbias=bias.to(dev) if ssd else None, hparam=hp, beta=dt if ssd else None, off_b=1, qscale=qs)
+        for s, n, off in ((0, lens[0], 0), (2, lens[2], lens[0])):
+            got[s].append(o[off:off + n].cpu().double())
+            at[s] += n
+    assert at == {0: T, 2: T2}
+    for s in (0, 2):
+        y = torch.cat(got[s])
+        err = float((y - want[s]).abs().max() / want[s].abs().max())
+        assert err < 3e-5, err
+    assert bool((state[[0, 2]] == 9.0).all())
+
+
+@gpu
+@pytest.mark.parametrize("H,D,V,rot", [(3, 16, 24, 16), (2, 48, 40, 22), (4, 128, 64, 128), (1, 8, 16, 0)])
+def test_rotated_bf16_rows(H, D, V, rot):
+    from bee2bee_b200 import ops
+
+    dev, T = "cuda", 37
+    g = torch.Generator().manual_seed(D)
+    q = torch.randn(T, 2 * H, D, generator=g)
+    v = torch.randn(T, H * V, generator=g)
+    perm = torch.arange(D)
+    if rot:
+        perm[:rot] = torch.arange(rot).view(2, rot // 2).t().reshape(-1)
+    proj = torch.cat([torch.zeros(T, 4), q[..., perm].reshape(T, -1), v], 1).to(dev)
+    r = {"dims": rot, "base": 50.0} if rot else None
+    want = O.rotate(q.double(), r)[..., perm].reshape(T, -1)
+    hi, lo = ops.split_frequencies(O.frequencies(r)[0] if rot else [0.0], dev)
+    tab = torch.zeros(T, max(2, rot), device=dev)
+    ops.rot_table(torch.arange(T, dtype=torch.int32, device=dev), hi, lo, 1.0, tab, T)
+    slots = torch.zeros(T, dtype=torch.int32, device=dev)
+    slots[5] = -1
+    qk, vo = torch.zeros(T, 2 * H * D, device=dev, dtype=torch.bfloat16), torch.zeros(T, H * V, device=dev, dtype=torch.bfloat16)
+    ops.rot_cast(proj, 4, 4 + 2 * H * D, tab if rot else None, rot, slots, qk, vo, T, 2 * H, D)
+    ok = [i for i in range(T) if i != 5]
+    assert torch.allclose(qk.cpu().double()[ok], want[ok], atol=3e-2, rtol=1e-2) and torch.equal(vo.cpu()[ok], v.bfloat16()[ok])
+    assert float(qk[5].abs().max()) == 0.0 and float(vo[5].abs().max()) == 0.0
 
 
 @gpu
@@ -935,7 +1017,7 @@ def test_trace_run_command_line(tmp_path):
     ]
     root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
     out = tmp_path / "out"
-    for dtype, tol in (("float32", 1e-4), ("bfloat16", 6e-2)):
+    for dtype, tol in (("float32", 1e-4), ("bfloat16", 8e-2)):
         res = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", path, "--dtype", dtype,
                               "--out", str(out), "--max-tokens", "192", "--slots", "2"],
                              input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
