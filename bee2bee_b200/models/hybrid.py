@@ -282,10 +282,10 @@ class HybridPiece:
 
     def n_launches(self) -> int:
         if self.sandwich:
-            per = {"diff_attention": 2, "mamba2": 4, "retention": 2}         # between the fused and the output projection (decode)
-            n = 3 + len(self.rot_tabs) + (1 if self.caps_logits else 0)      # embedding, first norm, (table, soft cap), commit
+            per = {"diff_attention": 2, "mamba2": 3, "retention": 2}         # between the fused and the output projection (decode)
+            n = 2 + len(self.rot_tabs) + (1 if self.caps_logits else 0)      # embedding, first norm, (table, soft cap)
             for L in self.L.values():
-                n += 3 + per[L.spec.mixer] + (5 if L.spec.ff else 0) + (4 if self.cfg.token_side else 0)
+                n += 3 + per[L.spec.mixer] + (4 if L.spec.ff else 0) + (3 if self.cfg.token_side else 0)
             return n
         if self.post_norm:
             n = 3                                        # embedding, its operand copy, final norm (head GEMM: the runner)
@@ -807,12 +807,16 @@ class HybridPiece:
         one GEMM over the down-projections side by side"""
         sp, o, f32 = L.spec, L.ff_off, torch.float32
         p2 = ops.linear(L.w_up, h, self._buf("proj2", f32, L.w_up.shape[0])[:T], bias=L.b_up)
+        hid = self._buf("ff", self.dtype, L.w_down.shape[1])[:T]
+        if not sp.expert_gated and sp.experts <= 256:    # squared relu times the expert's weight, the shared expert's gate in front
+            ops.route_cols(p2, sp.experts, sp.top, o["up"], sp.expert_ff, sp.shared_ff, ops.GATE_RELU_SQ, hid, T, off_gate=o["sg"],
+                           sigmoid=sp.route_kind == "sigmoid_topk")
+            return ops.linear(L.w_down, hid, self._buf("yff", f32, L.w_down.shape[0])[:T])
         wt = self._buf("route", f32, max(1, sp.experts))[:T]
         idw = self._buf("keep", f32, 1)[:T]
         ops.moe_route(p2, o["router"], None, sp.experts, 1, 1, sp.top, 1.0, wt, idw, T, sigmoid=sp.route_kind == "sigmoid_topk",
                       off_gate=o.get("sg", -1))
-        hid = self._buf("ff", self.dtype, L.w_down.shape[1])[:T]
-        if not sp.expert_gated:          # squared relu times the expert's weight, the shared expert's gate in front
+        if not sp.expert_gated:
             ops.gated_cols(p2, o["up"], 0, hid, o["hidden"], ops.GATE_RELU_SQ, T, wt=wt, per=sp.expert_ff, lead=sp.shared_ff,
                            lead_w=idw if sp.shared_gate else None)
             return ops.linear(L.w_down, hid, self._buf("yff", f32, L.w_down.shape[0])[:T])
@@ -1032,7 +1036,7 @@ class HybridPiece:
         if sp.ff:
             self._build_routed_ff(L, p, tensors)
         if self.cfg.token_side:
-            L.w_side, L.w_side_out = mat(p + "side.gate"), mat(p + "side.proj")
+            L.w_side, L.w_side_out = mat(p + "side.gate"), mat(p + "side.proj", k_mult=128)      # K of the second = padded rows of the first
             L.f["side"] = vec(p + "side.norm")
         return L
 
@@ -1065,9 +1069,12 @@ class HybridPiece:
                 pend = dict(y=self._ff_routed(L, h, T), norm_y=(f["norm2b"], f["norm2b.b"]))
             if c.token_side:
                 join()                   # h: the residual itself as the operand
-                z = ops.linear(L.w_side, h, self._buf("side", f32, L.w_side.shape[0])[:T])
-                g = self._buf(f"sideg{c.token_side}", self.dtype, L.w_side_out.shape[1])[:T]
-                ops.side_gate(z, m.ids, self.side_embed, l * c.token_side, g, c.token_side, T)
+                g = self._buf("sideg", self.dtype, L.w_side_out.shape[1])[:T]
+                if self.dtype == torch.bfloat16:
+                    ops.side_linear(L.w_side, h, g, self.side_embed, l * c.token_side, c.token_side, m.ids)
+                else:
+                    z = ops.linear(L.w_side, h, self._buf("side", f32, L.w_side.shape[0])[:T])
+                    ops.side_gate(z, m.ids, self.side_embed, l * c.token_side, g, c.token_side, T)
                 y = ops.linear(L.w_side_out, g, self._buf("yside", f32, L.w_side_out.shape[0])[:T])
                 pend = dict(y=y, norm_y=(f["side"], None), kind_y=ops.NORM_RMS)
             if self.debug_layers is not None:

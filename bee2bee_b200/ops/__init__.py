@@ -15,7 +15,7 @@ from typing import Optional
 import torch
 
 EPI_PLAIN, EPI_RESIDUAL, EPI_GLU, EPI_QKV_ROPE, EPI_GELU = 0, 1, 2, 3, 4
-ACT_SILU, ACT_GELU, ACT_RELU_SQ, ACT_XIELU = 0, 1, 2, 3   # ``act_gelu`` of ``gemm``: GLU gate activation / EPI_GELU activation
+ACT_SILU, ACT_GELU, ACT_RELU_SQ, ACT_XIELU, ACT_GELU_GATHER = 0, 1, 2, 3, 4   # ``act_gelu`` of ``gemm``: GLU gate activation / EPI_GELU activation
 COLS_COPY, COLS_TANH, COLS_RELU_SQ, COLS_XIELU, COLS_SOFTCAP = 0, 1, 2, 3, 4     # ``act`` of ``act_cols``
 SCAN_GLA, SCAN_DELTA, SCAN_MLSTM, SCAN_HGRN2, SCAN_SSD, SCAN_RETENTION = 0, 1, 2, 3, 4, 5     # ``mode`` of ``lin_scan``
 POST_SIGMOID, POST_SILU, POST_NONE = 0, 1, 2     # ``act`` of ``scan_post``: the output gate
@@ -38,7 +38,7 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
                         "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention", "sandwich_join", "rot_table",
                         "conv_rot_prep", "diff_combine", "diff_attention", "ssd_post", "side_gate", "rot_cast",
-                        "lin_chunk")
+                        "lin_chunk", "route_cols")
 
 
 class _CountedModule:
@@ -226,7 +226,8 @@ def gemm(w: torch.Tensor, x: torch.Tensor, out: Optional[torch.Tensor] = None, *
          fq_out: Optional[torch.Tensor] = None, fq_sf: Optional[torch.Tensor] = None, fq_bn: int = 0,
          sumsq_out: Optional[torch.Tensor] = None, zero_buf: Optional[torch.Tensor] = None,
          sumsq: Optional[torch.Tensor] = None, no_out: bool = False, act_p0: float = 0.0,
-         act_p1: float = 0.0) -> Optional[torch.Tensor]:
+         act_p1: float = 0.0, gather_ids: Optional[torch.Tensor] = None, gather_n: int = 0,
+         gather_rows: int = 0) -> Optional[torch.Tensor]:
     """out[t, n] = epilogue(sum_k x[t, k] * w[n, k]) on the tcgen05 swap-AB kernel."""
     m_tok, k = x.shape
     n_out = w.shape[0]
@@ -274,7 +275,7 @@ def gemm(w: torch.Tensor, x: torch.Tensor, out: Optional[torch.Tensor] = None, *
                   ack_flag, dbg, w_scale, sfa, sfb, GEMM_MC if mc < 0 else mc,
                   L2_PREFETCH if pf < 0 else pf, stages, free_lag, out2_ptr,
                   _ptr(fq_out), _ptr(fq_sf), fq_out.shape[1] if fq_out is not None else 0, fq_bn, _ptr(sumsq_out), _ptr(zero_buf),
-                  _ptr(sumsq))
+                  _ptr(sumsq), gather_ids, gather_n, gather_rows)
     return out
 
 
@@ -578,7 +579,7 @@ def short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max
     holds the inputs before the span and receives the last ones (a second kernel, after the first has read them); ``y`` float32
     or bf16"""
     native().short_conv(x, off, w, tail, y, q_start, q_len, kv_len, seq_slot, n_seqs, max_q, bias, int(bool(silu)))
-    if w.shape[1] > 1:
+    if w.shape[1] > 1 and not (max_q == 1 and w.shape[0] % 4 == 0 and w.shape[1] <= 4):       # (single tokens: one kernel does both)
         LAUNCHES[0] += 1
 
 
@@ -696,6 +697,13 @@ def gated_cols(x, off_a, off_b, out, n, act, T, wt=None, per=0, both=False, lead
     native().gated_cols(x, off_a, off_b, wt, per, out, n, act, T, 2 if scale_input else int(bool(both)), int(lead), lead_w)
 
 
+def route_cols(p, E, top, off, per, lead, act, out, T, off_gate=-1, sigmoid=False):
+    """Router and expert columns in one kernel (experts without a gate, ``E`` <= 256): the ``top`` largest of the logits in columns 0 ..
+    E of ``p``, weighted by the softmax over them (``sigmoid``: their sigmoids), scale ``act`` of the columns from ``off`` on -- ``lead``
+    of a shared expert (weight: sigmoid of column ``off_gate``, or 1), then ``per`` of every expert; what was not chosen becomes zeros"""
+    native().route_cols(p, int(E), int(top), int(bool(sigmoid)), int(off_gate), int(off), int(per), int(lead), int(act), out, T)
+
+
 def head_up_gate(a, U, out, T, H, V, C, gate=None, off_g=0):
     """``out[t, h V + v] = sigmoid(gate[t, off_g + h V + v]) * sum_c U[h, v, c] a[t, h C + c]`` (no gate: the plain product)"""
     native().head_up_gate(a, U, gate, off_g, out, T, H, V, C)
@@ -754,6 +762,14 @@ def diff_attention(q, k_cache, v_cache, out, block_table, q_start, q_len, kv_len
 def ssd_post(o, x, off_x, z, off_z, skip, w, out, T, H, V, parts, eps):
     """``out = groupnorm((o + skip_h x) * silu(z)) * w`` with the RMS norm over ``parts`` equal parts of the ``H * V`` channels"""
     native().ssd_post(o, x, off_x, z, off_z, skip, w, out, T, H, V, parts, float(eps))
+
+
+def side_linear(w, x, out, table, off, n, ids):
+    """bf16: ``out[t, c] = gelu_tanh((x w^T)[t, c]) * table[ids[t], off + c]`` for c < n, zero behind, as the epilogue of the product"""
+    assert out.shape[1] >= w.shape[0] and off + n <= table.shape[1]
+    gemm(w, x, out=out, epi=EPI_GELU, act_gelu=ACT_GELU_GATHER, residual=table[:, off:], gather_ids=ids, gather_n=n,
+         gather_rows=table.shape[0])
+    return out
 
 
 def side_gate(z, ids, table, off, out, n, T):

@@ -400,6 +400,9 @@ def cost(name: str, a, hint: Dict):
     if name == "ssd_post":
         H, V = a[9], a[10]
         return 0.0, T * H * V * (4 + a[1].element_size() + 4 + a[7].element_size()), False
+    if name == "route_cols":
+        E, top, per, lead = a[1], a[2], a[6], a[7]
+        return 0.0, T * ((lead + top * per + E + 1) * 4 + (lead + E * per) * a[9].element_size()), False
     if name == "side_gate":
         return 0.0, T * a[5] * (4 + a[2].element_size() + a[4].element_size()), False
     if name in ("rmsnorm", "layernorm", "add"):

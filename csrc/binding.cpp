@@ -48,7 +48,8 @@ void gemm(const Tensor& w, const Tensor& x, int64_t out_ptr, int64_t ld_out, int
           int64_t free_flag, int64_t bump_epoch, int64_t ack_flag, int64_t dbg, const OptT& w_scale,
           const OptT& sfa, const OptT& sfb, int64_t mc, int64_t pf_tiles, int64_t stages, int64_t free_lag, int64_t out2_ptr,
           // fused MX quantisation of the output / RMSNorm statistics (raw addresses, 0 = off)
-          int64_t q_out8, int64_t q_sf, int64_t ld_q, int64_t q_bn, int64_t sumsq_out, int64_t zero_buf, int64_t sumsq) {
+          int64_t q_out8, int64_t q_sf, int64_t ld_q, int64_t q_bn, int64_t sumsq_out, int64_t zero_buf, int64_t sumsq,
+          const OptT& gather_ids, int64_t gather_n, int64_t gather_rows) {
   const bool fp8 = w.scalar_type() == at::kFloat8_e4m3fn;
   if (fp8) {
     TORCH_CHECK(x.scalar_type() == at::kFloat8_e4m3fn && w.is_cuda() && x.is_cuda() && w.is_contiguous() &&
@@ -131,6 +132,11 @@ void gemm(const Tensor& w, const Tensor& x, int64_t out_ptr, int64_t ld_out, int
                 "q/kv widths must be multiples of 128");
     TORCH_CHECK(p.n_out == (p.n_q_heads + 2 * p.n_kv_heads) * p.head_dim, "qkv rows mismatch");
   }
+  p.gather_ids = ptr_or_null<const int>(gather_ids);
+  p.gather_n = static_cast<int>(gather_n);
+  p.gather_rows = static_cast<int>(gather_rows);
+  TORCH_CHECK(p.epi != b2b::EPI_GELU || p.act_gelu != 4 || (p.gather_ids && p.residual && p.gather_n <= p.n_out && p.gather_rows > 0 &&
+                                                            gather_ids->numel() >= p.m_tok), "gathered epilogue needs ids and a table");
   if (p.epi == b2b::EPI_RESIDUAL) TORCH_CHECK(p.residual != nullptr, "residual epilogue needs residual");
   if (p.epi == b2b::EPI_GLU) TORCH_CHECK(p.out != nullptr || (p.q_out8 != nullptr && p.sfa != nullptr), "GLU epilogue needs an output");
   if (p.signal_flag || p.bump_epoch) TORCH_CHECK(p.done_counter != nullptr, "handoff needs done_counter");
@@ -910,6 +916,18 @@ void rot_cast(const Tensor& proj, int64_t off, int64_t off_v, const OptT& tab, i
         "rot_cast");
 }
 
+// router over columns 0 .. E (biases already added), expert columns off ..: the shared expert's `lead`, then `per` of every expert
+void route_cols(const Tensor& p, int64_t E, int64_t top, int64_t sigmoid, int64_t off_gate, int64_t off, int64_t per, int64_t lead,
+                int64_t act, const Tensor& out, int64_t T) {
+  c10::cuda::CUDAGuard guard(p.device());
+  TORCH_CHECK(off + lead + E * per <= p.size(1) && out.size(1) >= lead + E * per, "route_cols: columns");
+  check(b2b::launch_route_cols(fp(p), static_cast<int>(p.stride(0)), static_cast<int>(E), static_cast<int>(top), static_cast<int>(sigmoid),
+                               static_cast<int>(off_gate), static_cast<int>(off), static_cast<int>(per), static_cast<int>(lead),
+                               static_cast<int>(act), out.data_ptr(), static_cast<int>(out.stride(0)), static_cast<int>(T), is_f32(out),
+                               cur_stream()),
+        "route_cols");
+}
+
 // q, k, v: bf16 rows with first columns off_*; mode as in lin_scan (4 state-space, 5 retention)
 void lin_chunk(int64_t mode, const Tensor& q, int64_t off_q, const Tensor& k, int64_t off_k, const Tensor& v, int64_t off_v, const OptT& step,
                int64_t off_step, const OptT& bias, const Tensor& hparam, double qscale, const Tensor& state, const Tensor& out,
@@ -1019,5 +1037,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("side_gate", &side_gate);
   m.def("rot_cast", &rot_cast);
   m.def("lin_chunk", &lin_chunk);
+  m.def("route_cols", &route_cols);
   m.def("lin_chunk_supported", &b2b::lin_chunk_supported);
 }

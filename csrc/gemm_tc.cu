@@ -526,6 +526,17 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
           resid[i] = (i < n && tok < p.m_tok) ? p.residual[static_cast<size_t>(tok) * p.ld_res + n_glob] : __float2bfloat16_rn(0.f);
         }
       }
+      if constexpr (EPI == EPI_GELU) {
+        if (p.act_gelu == 4) {                   // the tokens' own channels, again all loads of the chunk in flight
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int tok = tok0 + col0 + c + i;
+            resid[i] = __float2bfloat16_rn(0.f);
+            if (i < n && tok < p.m_tok && n_glob < p.gather_n)
+              resid[i] = p.residual[static_cast<size_t>(min(max(p.gather_ids[tok], 0), p.gather_rows - 1)) * p.ld_res + n_glob];
+          }
+        }
+      }
       float v[16];
       load_acc(c, n, v);
       float qv[16];                              // outputs of this chunk for the fused quantiser
@@ -543,7 +554,8 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
           else reinterpret_cast<__nv_bfloat16*>(p.out)[static_cast<size_t>(tok) * p.ld_out + n_glob] = __float2bfloat16_rn(a);
         } else if constexpr (EPI == EPI_GELU) {
           reinterpret_cast<__nv_bfloat16*>(p.out)[static_cast<size_t>(tok) * p.ld_out + n_glob] =
-              __float2bfloat16_rn(p.act_gelu == 2 ? relu_sq(a) : (p.act_gelu == 3 ? xielu(a, p.rope_theta, p.q_scale) : gelu_tanh(a)));
+              __float2bfloat16_rn(p.act_gelu == 2 ? relu_sq(a) : (p.act_gelu == 3 ? xielu(a, p.rope_theta, p.q_scale)
+                                                                                 : (p.act_gelu == 4 ? gelu_tanh(a) * __bfloat162float(resid[i]) : gelu_tanh(a))));
         } else if constexpr (EPI == EPI_RESIDUAL) {
           const float rv = a + __bfloat162float(resid[i]);
           const __nv_bfloat16 r16 = __float2bfloat16_rn(rv);

@@ -22,7 +22,7 @@ struct GemmParams {
   int8_t splitk;         // cluster size along grid.z (1..8)
   int8_t epi;
   int8_t out_fp32;       // EPI_PLAIN only: write fp32 (logits)
-  int8_t act_gelu;       // EPI_GLU: 0 = SiLU (SwiGLU), 1 = tanh-GELU (GeGLU); EPI_GELU: 2 = squared relu, 3 = xIELU (its two slopes ride in rope_theta / q_scale), else tanh-GELU
+  int8_t act_gelu;       // EPI_GLU: 0 = SiLU (SwiGLU), 1 = tanh-GELU (GeGLU); EPI_GELU: 2 = squared relu, 3 = xIELU (its two slopes ride in rope_theta / q_scale), 4 = tanh-GELU times a gathered row (below), else tanh-GELU
   int8_t fp8;            // operands are e4m3 (W8A8): W [N,K] and X [T,K] one byte per element
   int8_t stages;         // shared-memory ring depth (0 = the token tile's default)
   int8_t mc;             // EXPERIMENTAL (0/1 = off): cluster of `mc` CTAs along the weight-tile axis shares the token tile by TMA multicast
@@ -38,6 +38,9 @@ struct GemmParams {
   void* out2;         // EPI_RESIDUAL: optional second destination with the same layout (e.g. the peer's staging slot), or null
   const __nv_bfloat16* residual;  // [m_tok, ld_res]
   int ld_res;
+  // EPI_GELU with act_gelu 4: out[t, n] = gelu(a) * residual[gather_ids[t], n] for n < gather_n (zero behind), rows clamped to gather_rows
+  const int* gather_ids;
+  int gather_n, gather_rows;
   const float* bias;              // [n_out] or null
 
   // fused RMSNorm of the input: gamma is pre-folded into W, so only the per-token

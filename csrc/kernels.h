@@ -158,6 +158,10 @@ int launch_rot_heads(const float* src, int ld, int off, float* dst, int H, int D
 int launch_moe_route(const float* proj, int ld, int off, const float* corr, int E, int n_real, int count, int keep,
                      int top, float scale, float* wt, int ld_wt, float* idw, int* sel_idx, float* sel_w, int T,
                      int sigmoid, int off_gate, cudaStream_t s);
+// the router and the expert columns in one kernel (E <= 256, the largest logits chosen): columns of experts that were not chosen are
+// written as zeros without being read
+int launch_route_cols(const float* p, int ld, int E, int top, int sigmoid, int off_gate, int off, int per, int lead, int act, void* out,
+                      int ld_out, int T, int f32, cudaStream_t s);
 int launch_poly_norm(const float* in, int ld_in, int off, const float* w, void* out, int ld_out, int n, float eps, int T,
                      int f32, cudaStream_t s);
 int launch_gated_cols(const float* in, int ld_in, int off_a, int off_b, const float* wt, int ld_wt, int per, void* out,

@@ -11,6 +11,7 @@
 //   * moe_route        softmax router with a selection-only correction, group-limited top-k and identity experts; top-k sigmoid scores
 //   * gated_cols       out = act(a) * b for two column blocks, or act(a) * per-expert weight (routed experts run as one
 //                      stacked up-projection whose hidden columns are scaled by the token's weight for their expert), or both
+//   * route_cols       router and expert columns of experts without a gate in one kernel; only chosen experts' columns are read
 //   * head_up_gate     a [V, C] matrix per head applied to per-head latent rows, times a sigmoid output gate
 // Norms, gates, router, angles and the residual are fp32 in every mode; OT / CT (operand / cache type) is bf16 or float.
 // This translation unit is compiled WITHOUT --use_fast_math (exact expf / erff / division / sqrt / sincos).
@@ -500,6 +501,73 @@ __global__ void __launch_bounds__(256)
   st4(out + t * ld_out + c, make_float4(act_(a.x, act) * b.x, act_(a.y, act) * b.y, act_(a.z, act) * b.z, act_(a.w, act) * b.w));
 }
 
+// ------------------------------------------------------------------------------------------- router + expert columns
+// One block per (token, slice of columns): warp 0 chooses the `top` largest of the E logits in columns 0 .. E (ties: the lower index)
+// and weights them by the softmax over the chosen ones (sigmoid != 0: by their sigmoids); then out[t, c] = act(x[t, off + c]) * weight,
+// where columns c < lead have the weight sigmoid(x[t, off_gate]) (1 when off_gate < 0) and column c >= lead that of expert
+// (c - lead) / per.  Columns of experts that were not chosen are not read.  VEC: four columns per access (per, lead multiples of four).
+constexpr int RC_THREADS = 256, RC_MAX_E = 256;
+template <typename OT, bool VEC>
+__global__ void __launch_bounds__(RC_THREADS)
+    route_cols_kernel(const float* __restrict__ p, int ld, int E, int top, int sigmoid, int off_gate, int off, int per, int lead, int act,
+                      OT* __restrict__ out, int ld_out, int n) {
+  pdl_begin();
+  __shared__ float wts[RC_MAX_E + 1];                  // [E] and the leading columns' weight
+  const float* row = p + static_cast<size_t>(blockIdx.x) * ld;
+  const int tid = threadIdx.x;
+  if (tid < 32) {
+    const float ninf = -__int_as_float(0x7f800000);
+    float z[RC_MAX_E / 32], first = 0.f, tot = 0.f;
+    unsigned chosen = 0u;                              // bit k: expert lane + 32 k
+#pragma unroll
+    for (int k = 0; k < RC_MAX_E / 32; ++k) z[k] = tid + 32 * k < E ? row[tid + 32 * k] : ninf;
+    const float gate = off_gate >= 0 ? sigmoid_(row[off_gate]) : 1.f;
+    for (int s = 0; s < top; ++s) {
+      float bv = ninf;
+      int bi = 0x7fffffff;
+#pragma unroll
+      for (int k = 0; k < RC_MAX_E / 32; ++k)
+        if (!(chosen >> k & 1u) && z[k] > bv) {
+          bv = z[k];
+          bi = tid + 32 * k;
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > bv || (ov == bv && oi < bi)) {
+          bv = ov;
+          bi = oi;
+        }
+      }
+      if (bi == 0x7fffffff) break;
+      if ((bi & 31) == tid) chosen |= 1u << (bi >> 5);
+      if (s == 0) first = bv;
+      tot += expf(bv - first);
+    }
+#pragma unroll
+    for (int k = 0; k < RC_MAX_E / 32; ++k)
+      if (tid + 32 * k < E) wts[tid + 32 * k] = !(chosen >> k & 1u) ? 0.f : (sigmoid ? sigmoid_(z[k]) : expf(z[k] - first) / tot);
+    if (tid == 0) wts[E] = gate;
+  }
+  __syncthreads();
+  constexpr int S = VEC ? 4 : 1;
+  OT* dst = out + static_cast<size_t>(blockIdx.x) * ld_out;
+  for (int c = S * (blockIdx.y * RC_THREADS + tid); c < n; c += S * RC_THREADS * gridDim.y) {
+    const float w = c < lead ? wts[E] : wts[(c - lead) / per];
+    if constexpr (VEC) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (w != 0.f) {
+        v = *reinterpret_cast<const float4*>(row + off + c);
+        v = make_float4(act_(v.x, act) * w, act_(v.y, act) * w, act_(v.z, act) * w, act_(v.w, act) * w);
+      }
+      st4(dst + c, v);
+    } else {
+      stf(dst, c, w != 0.f ? act_(row[off + c], act) * w : 0.f);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------- per-head up-projection
 // out[t, h * V + v] = gate(t, h * V + v) * sum_c a[t, h * C + c] * U[h, v, c]: every head has its own [V, C] matrix (the
 // value up-projection of latent attention, applied to the attention output taken over the latents), so this is a batch
@@ -763,6 +831,31 @@ int launch_moe_route(const float* proj, int ld, int off, const float* corr, int 
   if (smem > 48 * 1024) return -2;
   launch_kernel(moe_route_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, s, 1u, proj, ld, off, corr, E,
                 n_real, count, keep, top, scale, wt, ld_wt, idw, sel_idx, sel_w, T, sigmoid, off_gate);
+  return last_error();
+}
+
+int launch_route_cols(const float* p, int ld, int E, int top, int sigmoid, int off_gate, int off, int per, int lead, int act, void* out,
+                      int ld_out, int T, int f32, cudaStream_t s) {
+  const int n = lead + E * per;
+  if (T <= 0 || n <= 0) return 0;
+  if (E <= 0 || E > RC_MAX_E || top <= 0 || top > E || per <= 0) return -2;
+  const bool vec = per % 4 == 0 && lead % 4 == 0 && off % 4 == 0 && ld % 4 == 0 && ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(p) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(out) % 16 == 0;
+  const int most = (n + RC_THREADS * (vec ? 4 : 1) - 1) / (RC_THREADS * (vec ? 4 : 1));
+  int slices = T >= 592 ? 1 : (592 + T - 1) / T;       // few tokens: several blocks per token (the choice is made in each of them)
+  if (slices > most) slices = most;
+  const dim3 grid(T, slices);
+#define B2B_RC(OT, VEC)                                                                                                  \
+  launch_kernel(route_cols_kernel<OT, VEC>, grid, dim3(RC_THREADS), 0, s, 1u, p, ld, E, top, sigmoid, off_gate, off, per, lead, act, \
+                static_cast<OT*>(out), ld_out, n)
+  if (f32) {
+    if (vec) B2B_RC(float, true);
+    else B2B_RC(float, false);
+  } else {
+    if (vec) B2B_RC(bf16, true);
+    else B2B_RC(bf16, false);
+  }
+#undef B2B_RC
   return last_error();
 }
 

@@ -831,6 +831,60 @@ __global__ void __launch_bounds__(128)
   }
 }
 
+// four adjacent channels per thread with 16-byte accesses (C, ld and off multiples of four; taps <= MT).  DEC: every span is one token,
+// and the thread that owns a channel shifts its tail itself.
+template <int MT, typename YT, bool DEC>
+__global__ void __launch_bounds__(128)
+    short_conv4_kernel(const float* __restrict__ x, int ld_x, int off, const float* __restrict__ w, float* __restrict__ tail,
+                       YT* __restrict__ y, int ld_y, const int* __restrict__ q_start, const int* __restrict__ q_len,
+                       const int* __restrict__ kv_len, const int* __restrict__ seq_slot, int C, int taps, int tpt,
+                       const float* __restrict__ bias, int act) {
+  pdl_begin();
+  const int s = blockIdx.z, n = q_len[s], i0 = blockIdx.y * tpt;
+  const int c = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+  if (i0 >= n || c >= C) return;
+  const int t0 = q_start[s], pos0 = kv_len[s] - n;
+  float* tl = tail + static_cast<size_t>(seq_slot[s]) * (taps - 1) * C + c;
+  const float* xc = x + off + c;
+  float wr[MT][4];
+  float4 win[MT];
+#pragma unroll
+  for (int j = 0; j < MT; ++j) {
+    win[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) wr[j][e] = j < taps ? w[static_cast<size_t>(c + e) * taps + j] : 0.f;
+    if (j < taps - 1) {
+      const int i = i0 - (taps - 1) + j;
+      if (i >= 0) win[j] = *reinterpret_cast<const float4*>(xc + static_cast<size_t>(t0 + i) * ld_x);
+      else if (pos0 > 0) win[j] = *reinterpret_cast<const float4*>(tl + static_cast<size_t>(taps - 1 + i) * C);
+    }
+  }
+  const float4 b = bias != nullptr ? *reinterpret_cast<const float4*>(bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  const int i1 = min(n, i0 + tpt);
+  for (int i = i0; i < i1; ++i) {
+    const float4 cur = *reinterpret_cast<const float4*>(xc + static_cast<size_t>(t0 + i) * ld_x);
+    float4 acc = b;
+#pragma unroll
+    for (int j = 0; j < MT; ++j) {
+      if (j < taps) {
+        const float4 v = j < taps - 1 ? win[j] : cur;
+        acc.x += wr[j][0] * v.x;
+        acc.y += wr[j][1] * v.y;
+        acc.z += wr[j][2] * v.z;
+        acc.w += wr[j][3] * v.w;
+        if (j < taps - 1) win[j] = (j + 1 < MT && j + 1 < taps - 1) ? win[j + 1 < MT ? j + 1 : j] : cur;
+      }
+    }
+    if (act) acc = make_float4(silu_(acc.x), silu_(acc.y), silu_(acc.z), silu_(acc.w));
+    st_operand(y + static_cast<size_t>(t0 + i) * ld_y, c >> 2, acc, true);
+  }
+  if (DEC) {
+#pragma unroll
+    for (int j = 0; j < MT; ++j)
+      if (j < taps - 1) *reinterpret_cast<float4*>(tl + static_cast<size_t>(j) * C) = win[j];
+  }
+}
+
 // the last taps-1 inputs of every sequence -> tail (runs after the convolution of the step has read the old tail)
 template <int MT>
 __global__ void short_conv_commit_kernel(const float* __restrict__ x, int ld_x, int off, float* __restrict__ tail,
@@ -1308,7 +1362,7 @@ __global__ void __launch_bounds__(LN* CB / ls_cols(DEC) + (DEC ? 0 : ls_stage_th
 // o [T, H*dv] fp32 -> per head: (o / den) / sqrt(mean(.^2) + eps) * weight * act(gate) -> OT.  den (aux given, mLSTM):
 // max(|n.q|, exp(-mx)) + 1e-6.  weight: [dv] shared by the heads (wshared) or [H*dv].  act: 0 sigmoid, 1 silu, 2 no gate.
 // One warp per (token, head).
-template <typename OT>
+template <typename OT, bool VEC>
 __global__ void scan_post_kernel(const float* __restrict__ o, int ld_o, const float* __restrict__ gate, int ld_g,
                                  int off_g, const float* __restrict__ weight, int wshared, int act,
                                  const float* __restrict__ aux, OT* __restrict__ out, int ld_out, int T, int H, int dv,
@@ -1326,6 +1380,23 @@ __global__ void scan_post_kernel(const float* __restrict__ o, int ld_o, const fl
     inv = 1.f / (fmaxf(fabsf(g.w), g.z) + 1e-6f);
   }
   float ss = 0.f;
+  if constexpr (VEC) {                                   // dv <= 128 and every row offset a multiple of four: one access per lane
+    const int d = 4 * lane;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f), g = make_float4(1.f, 1.f, 1.f, 1.f), w = v;
+    if (d < dv) {
+      v = *reinterpret_cast<const float4*>(src + d);
+      if (act != 2) g = *reinterpret_cast<const float4*>(grow + d);
+      w = *reinterpret_cast<const float4*>(weight + (wshared ? d : hd * dv + d));
+    }
+    v = make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv);
+    const float r = 1.f / sqrtf(warp_sum_(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / static_cast<float>(dv) + eps);
+    if (d >= dv) return;
+    if (act == 1) g = make_float4(silu_(g.x), silu_(g.y), silu_(g.z), silu_(g.w));
+    if (act == 0) g = make_float4(sigmoid_(g.x), sigmoid_(g.y), sigmoid_(g.z), sigmoid_(g.w));
+    st_operand(out + static_cast<size_t>(t) * ld_out + hd * dv, lane, make_float4(v.x * r * w.x * g.x, v.y * r * w.y * g.y, v.z * r * w.z * g.z,
+                                                                               v.w * r * w.w * g.w), true);
+    return;
+  }
   for (int d = lane; d < dv; d += 32) {
     const float v = src[d] * inv;
     ss += v * v;
@@ -1544,6 +1615,24 @@ int launch_short_conv(const float* x, int ld_x, int off, const float* w, float* 
   if (taps < 1 || taps > CONV_MAX_TAPS) return -2;
   const int tpt = 16;
   dim3 grid((C + 127) / 128, (max_q + tpt - 1) / tpt, n_seqs);
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (C % 4 == 0 && ld_x % 4 == 0 && off % 4 == 0 && ld_y % 4 == 0 && taps <= 4 && al16(x) && al16(y) && al16(tail) && al16(bias)) {
+    const bool dec = max_q == 1;
+    const dim3 vgrid((C / 4 + 127) / 128, (max_q + tpt - 1) / tpt, n_seqs);
+#define B2B_SC4(YT, DEC)                                                                                                 \
+  launch_kernel(short_conv4_kernel<4, YT, DEC>, vgrid, dim3(128), 0, s, 1u, x, ld_x, off, w, tail, static_cast<YT*>(y), ld_y, q_start, \
+                q_len, kv_len, seq_slot, C, taps, tpt, bias, act)
+    if (y_f32) {
+      if (dec) B2B_SC4(float, true);
+      else B2B_SC4(float, false);
+    } else {
+      if (dec) B2B_SC4(bf16, true);
+      else B2B_SC4(bf16, false);
+    }
+#undef B2B_SC4
+    const int e = last_error();
+    return e || dec ? e : launch_short_conv_commit(x, ld_x, off, tail, q_start, q_len, kv_len, seq_slot, n_seqs, C, taps, s);
+  }
 #define B2B_SC(MT, YT)                                                                                                   \
   launch_kernel(short_conv_kernel<MT, YT>, grid, dim3(128), 0, s, 1u, x, ld_x, off, w, static_cast<const float*>(tail),  \
                 static_cast<YT*>(y), ld_y, q_start, q_len, kv_len, seq_slot, C, taps, tpt, bias, act)
@@ -1634,12 +1723,20 @@ int launch_scan_post(const float* o, int ld_o, const float* gate, int ld_g, int 
   const long long warps = static_cast<long long>(T) * H;
   if (warps <= 0) return 0;
   const int blocks = static_cast<int>((warps + 3) / 4);
-  if (f32)
-    launch_kernel(scan_post_kernel<float>, dim3(blocks), dim3(128), 0, s, 1u, o, ld_o, gate, ld_g, off_g, weight, wshared,
-                  act, aux, static_cast<float*>(out), ld_out, T, H, dv, eps);
-  else
-    launch_kernel(scan_post_kernel<bf16>, dim3(blocks), dim3(128), 0, s, 1u, o, ld_o, gate, ld_g, off_g, weight, wshared,
-                  act, aux, static_cast<bf16*>(out), ld_out, T, H, dv, eps);
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool vec = dv % 4 == 0 && dv <= 128 && ld_o % 4 == 0 && ld_g % 4 == 0 && off_g % 4 == 0 && ld_out % 4 == 0 && al16(o) && al16(gate) &&
+                   al16(weight) && al16(out);
+#define B2B_POST(OT, VEC)                                                                                                \
+  launch_kernel(scan_post_kernel<OT, VEC>, dim3(blocks), dim3(128), 0, s, 1u, o, ld_o, gate, ld_g, off_g, weight, wshared, act, aux, \
+                static_cast<OT*>(out), ld_out, T, H, dv, eps)
+  if (f32) {
+    if (vec) B2B_POST(float, true);
+    else B2B_POST(float, false);
+  } else {
+    if (vec) B2B_POST(bf16, true);
+    else B2B_POST(bf16, false);
+  }
+#undef B2B_POST
   return last_error();
 }
 

@@ -734,6 +734,52 @@ def test_router_with_shared_gate_and_squared_relu_columns(E, top, shared, per):
         out = torch.zeros(T, (n + 63) // 64 * 64, device=dev, dtype=dt)
         ops.gated_cols(p.to(dev), off, 0, out, n, ops.GATE_RELU_SQ, T, wt=wt, per=per, lead=shared, lead_w=idw)
         assert torch.allclose(out[:, :n].float().cpu().double(), want, atol=tol, rtol=1e-2)
+        both = torch.full((T, (n + 63) // 64 * 64), 5.0, device=dev, dtype=dt)                # one kernel for both steps
+        q = p.clone()
+        q[:, off:off + n][cw == 0] = float("nan")                                           # (what was not chosen is not read)
+        ops.route_cols(q.to(dev), E, top, off, per, shared, ops.GATE_RELU_SQ, both, T, off_gate=E)
+        assert torch.allclose(both[:, :n].float().cpu().double(), want, atol=tol, rtol=1e-2)
+        assert bool((both[:, n:] == 5.0).all())
+
+
+@gpu
+@pytest.mark.parametrize("E,top,T", [(40, 6, 3), (100, 9, 700), (256, 5, 2), (1, 1, 5)])
+def test_router_and_columns_of_many_experts(E, top, T):
+    """more experts than lanes; equal logits go to the lower index; no shared expert; sigmoid weights"""
+    from bee2bee_b200 import ops
+
+    dev, per, off = "cuda", 8, (E + 3) // 4 * 4
+    g = torch.Generator().manual_seed(E)
+    p = torch.randn(T, off + E * per, generator=g)
+    p[:, :E] = torch.round(p[:, :E] * 4) / 4                                               # many ties
+    idx, w = O.choose(p[:, :E].double(), top)
+    for sig in (False, True):
+        dense = torch.zeros(T, E, dtype=torch.float64)
+        for t in range(T):
+            for j, v in zip(idx[t], w[t]):
+                dense[t, j] = torch.sigmoid(p[t, j].double()) if sig else v
+        want = O.relu_sq(p[:, off:].double()) * dense.repeat_interleave(per, 1)
+        out = torch.full((T, E * per), 5.0, device=dev)
+        ops.route_cols(p.to(dev), E, top, off, per, 0, ops.GATE_RELU_SQ, out, T, sigmoid=sig)
+        assert torch.allclose(out.cpu().double(), want, atol=1e-5)
+
+
+@gpu
+@pytest.mark.parametrize("T", [1, 33, 300])
+@pytest.mark.parametrize("n", [12, 128, 200])
+def test_token_channels_in_the_product_epilogue(T, n):
+    from bee2bee_b200 import ops
+
+    dev, K, vocab = "cuda", 192, 40
+    g = torch.Generator().manual_seed(T + n)
+    w, x, table = ((torch.randn(*s, generator=g) * k).bfloat16() for s, k in (((n, K), K ** -0.5), ((T, K), 1.0), ((vocab, 3 * n), 1.0)))
+    ids = torch.randint(0, vocab, (T,), generator=g)
+    want = O.gelu_tanh(x.double() @ w.double().T) * table[ids][:, n:2 * n].double()
+    wp = ops.pad_weight(w, 128, 64).to(dev)
+    out = torch.full((T, wp.shape[0]), 5.0, device=dev, dtype=torch.bfloat16)
+    ops.side_linear(wp, x.to(dev), out, table.to(dev), n, n, ids.int().to(dev))
+    assert torch.allclose(out[:, :n].cpu().double(), want, atol=2e-2, rtol=2e-2)
+    assert wp.shape[0] == n or float(out[:, n:].float().abs().max()) == 0.0
 
 
 # ---------------------------------------------------------------------------------------- every mechanism alone
