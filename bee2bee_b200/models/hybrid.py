@@ -1135,6 +1135,9 @@ class HybridPiece:
         if chunked:
             ops.lin_chunk(ops.SCAN_SSD, xbc, inner + G * N, xbc, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len,
                           m.seq_slot, m.n_seqs, H, G, N, V, step=proj, off_step=mx.off["dt"], bias=mx.f["dt_bias"], hparam=mx.f["A_log"])
+        elif m.max_q == 1 and ops.lin_step_supported(m.n_seqs, H, N, V):
+            ops.lin_step(ops.SCAN_SSD, xbc, inner + G * N, xbc, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len,
+                         m.seq_slot, m.n_seqs, H, G, N, V, step=proj, off_step=mx.off["dt"], bias=mx.f["dt_bias"], hparam=mx.f["A_log"])
         else:
             ops.lin_scan(ops.SCAN_SSD, xbc, inner + G * N, inner, xbc, 0, self.state[key], o, m.q_start, m.q_len, m.kv_len,
                          m.seq_slot, m.n_seqs, m.max_q, H, G, N, V, zbias=mx.f["dt_bias"], hparam=mx.f["A_log"], beta=proj,
@@ -1159,6 +1162,9 @@ class HybridPiece:
             ops.rot_cast(proj, mx.off["q"], mx.off["v"], tab, rd, m.slots, qk, v, T, 2 * H, D)
             ops.lin_chunk(ops.SCAN_RETENTION, qk, 0, qk, H * D, v, 0, st, o, m.q_start, m.q_len, m.kv_len, m.seq_slot, m.n_seqs, H, H, D,
                           V, hparam=mx.f["decay"], qscale=D ** -0.5)
+        elif m.max_q == 1 and ops.lin_step_supported(m.n_seqs, H, D, V):
+            ops.lin_step(ops.SCAN_RETENTION, proj, mx.off["q"], proj, mx.off["k"], proj, mx.off["v"], st, o, m.q_start, m.q_len, m.kv_len,
+                         m.seq_slot, m.n_seqs, H, H, D, V, hparam=mx.f["decay"], tab=tab, rdims=rd, qscale=D ** -0.5)
         else:
             ops.lin_scan(ops.SCAN_RETENTION, proj, mx.off["q"], mx.off["k"], proj, mx.off["v"], st, o, m.q_start, m.q_len, m.kv_len,
                          m.seq_slot, m.n_seqs, m.max_q, H, H, D, V, z=tab, hparam=mx.f["decay"], qscale=D ** -0.5, rdims=rd)

@@ -38,7 +38,7 @@ _KERNEL_ENTRY_POINTS = ("add", "attention", "decode_advance", "embed", "fetch_wi
                         "short_conv", "mlstm_gates", "lin_scan", "scan_post", "post_norm_join", "latent_prep", "rot_heads",
                         "moe_route", "gated_cols", "head_up_gate", "talk_prep", "poly_norm", "mixed_attention", "sandwich_join", "rot_table",
                         "conv_rot_prep", "diff_combine", "diff_attention", "ssd_post", "side_gate", "rot_cast",
-                        "lin_chunk", "route_cols")
+                        "lin_chunk", "route_cols", "lin_step")
 
 
 class _CountedModule:
@@ -197,13 +197,15 @@ def pick_splitk(n_out: int, m_tok: int, k: int, bn: int, epi: int, stages: int =
         # measured (tools/layer_sweep.py, Llama-3-8B, reduce-scatter split-K epilogue): up to ~2 CTAs per SM pay off
         # (bn=32: qkv 4, o 4, gate/up 1, down 8 -> 100 us/layer; bn=16: 4/4/1/4 -> 92.6 us); >= 16 k-blocks per
         # CTA, and every CTA of the cluster keeps >= 4 token columns (vector DSMEM stores)
+        # narrower models (K < 4096, or few weight tiles; measured at 32 tokens, back to back): 8 k-blocks per CTA are enough, 4 while
+        # the machine is not full (2048 x 2048: 7.4 against 9.4 us, 1024 x 1024: 5.7 against 9.1, 128 x 2048: 5.6 against 9.1)
         tiles = (n_out // 128) * ((m_tok + bn - 1) // bn)
-        limit = 256 if bn >= 32 else 200
+        kb, limit = k // 64, 256 if bn >= 32 else 200
         want = 1
-        while tiles * want * 2 <= limit and want < 8 and bn // (want * 2) >= 4:
-            want *= 2
-        while want > 1 and (k // 64) // want < 16:
-            want //= 2
+        for s in (2, 4, 8):
+            if bn // s >= 4 and ((tiles * s <= limit and kb // s >= 16) or (tiles * s <= 140 and kb // s >= 4)
+                                 or (kb < 64 and tiles * s <= limit + 16 and kb // s >= 8)):
+                want = s
     want = min(want, 8, max(1, (k // 64) // 2))
     cap = native().gemm_max_splitk(bn, epi, stages)
     while want > cap:
@@ -613,6 +615,18 @@ def lin_chunk(mode, q, off_q, k, off_k, v, off_v, state, out, q_start, q_len, kv
                        seq_slot, n_seqs, H, G, dk, dv)
 
 
+def lin_step_supported(n_seqs, H, dk, dv):
+    """whether ``lin_step`` has a kernel for a decode step of these sizes (enough states to fill the machine; else: ``lin_scan``)"""
+    return bool(native().lin_step_supported(int(n_seqs), int(H), int(dk), int(dv)))
+
+
+def lin_step(mode, q, off_q, k, off_k, v, off_v, state, out, q_start, q_len, kv_len, seq_slot, n_seqs, H, G, dk, dv, *, step=None,
+             off_step=0, bias=None, hparam=None, tab=None, rdims=0, qscale=1.0):
+    """SCAN_SSD / SCAN_RETENTION for single tokens of many sequences: bulk copies stream the fp32 states through shared memory"""
+    native().lin_step(mode, q, off_q, k, off_k, v, off_v, step, off_step, bias, hparam, tab, int(rdims), float(qscale), state, out, q_start,
+                      q_len, kv_len, seq_slot, n_seqs, H, G, dk, dv)
+
+
 def rot_cast(proj, off, off_v, tab, rdims, slots, qk, v, T, H2, D):
     """bf16 rows of a recurrence: ``H2`` heads (queries, then keys) of D channels at column ``off`` with rotary positions on the first
     ``rdims`` (pairs 2i, 2i + 1; ``tab`` [T, rdims]) -> ``qk``; the columns from ``off_v`` on -> ``v``"""
@@ -767,8 +781,11 @@ def ssd_post(o, x, off_x, z, off_z, skip, w, out, T, H, V, parts, eps):
 def side_linear(w, x, out, table, off, n, ids):
     """bf16: ``out[t, c] = gelu_tanh((x w^T)[t, c]) * table[ids[t], off + c]`` for c < n, zero behind, as the epilogue of the product"""
     assert out.shape[1] >= w.shape[0] and off + n <= table.shape[1]
+    tile = {}
+    if x.shape[0] > 64 and w.shape[0] <= 512:      # few weight tiles: narrow token tiles, split along K, so that every SM has one
+        tile = dict(bn=32, stages=0, splitk=4 if x.shape[1] >= 2048 else (2 if x.shape[1] >= 512 else 1))
     gemm(w, x, out=out, epi=EPI_GELU, act_gelu=ACT_GELU_GATHER, residual=table[:, off:], gather_ids=ids, gather_n=n,
-         gather_rows=table.shape[0])
+         gather_rows=table.shape[0], **tile)
     return out
 
 

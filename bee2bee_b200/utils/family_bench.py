@@ -397,6 +397,9 @@ def cost(name: str, a, hint: Dict):
     if name == "lin_chunk":
         H, G, dk, dv = a[19], a[20], a[21], a[22]
         return 6.0 * T * H * dk * dv, 2 * S * H * dk * dv * 4 + T * (2 * G * dk * 2 + H * dv * (2 + 4)), True
+    if name == "lin_step":
+        H, G, dk, dv = a[21], a[22], a[23], a[24]
+        return 6.0 * T * H * dk * dv, 2 * S * H * dk * dv * 4 + T * (2 * G * dk + 2 * H * dv) * 4, False
     if name == "ssd_post":
         H, V = a[9], a[10]
         return 0.0, T * H * V * (4 + a[1].element_size() + 4 + a[7].element_size()), False

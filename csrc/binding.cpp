@@ -150,6 +150,7 @@ void set_wait_policy(int64_t abort_word, double limit_ms) {
   check(b2b::set_wait_policy_elementwise(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(elementwise)");
   check(b2b::set_wait_policy_mixed(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(mixed)");
   check(b2b::set_wait_policy_diff(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(diff)");
+  check(b2b::set_wait_policy_step(as_ptr<uint32_t>(abort_word), ns), "set_wait_policy(step)");
 }
 
 void set_pdl(bool on) { b2b::g_pdl_mode = on ? 1 : 0; }
@@ -916,6 +917,27 @@ void rot_cast(const Tensor& proj, int64_t off, int64_t off_v, const OptT& tab, i
         "rot_cast");
 }
 
+// single tokens; q, k, v: fp32 rows with first columns off_*; tab: rotary table (retention)
+void lin_step(int64_t mode, const Tensor& q, int64_t off_q, const Tensor& k, int64_t off_k, const Tensor& v, int64_t off_v, const OptT& step,
+              int64_t off_step, const OptT& bias, const Tensor& hparam, const OptT& tab, int64_t rdims, double qscale, const Tensor& state,
+              const Tensor& out, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, const Tensor& seq_slot, int64_t n_seqs,
+              int64_t H, int64_t G, int64_t dk, int64_t dv) {
+  c10::cuda::CUDAGuard guard(q.device());
+  const bool ssd = mode == 4;
+  TORCH_CHECK(mode == 4 || mode == 5, "lin_step: one decay per head and token");
+  TORCH_CHECK(!ssd || (fp_or_null(step) != nullptr && fp_or_null(bias) != nullptr), "lin_step: step sizes");
+  TORCH_CHECK(rdims == 0 || (fp_or_null(tab) != nullptr && tab->size(-1) == rdims && tab->is_contiguous()), "lin_step: rotary table");
+  TORCH_CHECK(hparam.numel() >= H && off_q + (ssd ? G : H) * dk <= q.size(1) && off_k + (ssd ? G : H) * dk <= k.size(1) &&
+                  off_v + H * dv <= v.size(1) && out.size(1) >= H * dv && state.is_contiguous(), "lin_step: sizes");
+  check(b2b::launch_lin_step(ssd ? 1 : 0, fp(q) + off_q, static_cast<int>(q.stride(0)), fp(k) + off_k, static_cast<int>(k.stride(0)),
+                             fp(v) + off_v, static_cast<int>(v.stride(0)), ssd ? fp(*step) + off_step : nullptr,
+                             ssd ? static_cast<int>(step->stride(0)) : 0, fp_or_null(bias), fp(hparam), fp_or_null(tab),
+                             static_cast<int>(rdims), static_cast<float>(qscale), const_cast<float*>(fp(state)), const_cast<float*>(fp(out)),
+                             static_cast<int>(out.stride(0)), ip(q_start), ip(q_len), ip(kv_len), ip(seq_slot), static_cast<int>(n_seqs),
+                             static_cast<int>(H), static_cast<int>(G), static_cast<int>(dk), static_cast<int>(dv), cur_stream()),
+        "lin_step");
+}
+
 // router over columns 0 .. E (biases already added), expert columns off ..: the shared expert's `lead`, then `per` of every expert
 void route_cols(const Tensor& p, int64_t E, int64_t top, int64_t sigmoid, int64_t off_gate, int64_t off, int64_t per, int64_t lead,
                 int64_t act, const Tensor& out, int64_t T) {
@@ -1038,5 +1060,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rot_cast", &rot_cast);
   m.def("lin_chunk", &lin_chunk);
   m.def("route_cols", &route_cols);
+  m.def("lin_step", &lin_step);
+  m.def("lin_step_supported", &b2b::lin_step_supported);
+  m.def("lin_step_gave_up", &b2b::lin_step_gave_up);
   m.def("lin_chunk_supported", &b2b::lin_chunk_supported);
 }

@@ -242,6 +242,11 @@ __global__ void __launch_bounds__(DA_THREADS, 1)
     auto tile = [&](int n, auto masked) {
       const int kb = (t_lo + n) * DA_BKV;
       if (!all(ma_wait(&s_full[m], static_cast<uint32_t>(n & 1), abort))) return false;
+      if (quarter * 32 >= n_rows) {                                    // (warp-uniform; decode steps: what its rows hold is never read)
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&p_ready[m]);
+        return true;
+      }
       tc_fence_after();
       uint32_t r[DA_BKV];
 #pragma unroll

@@ -207,10 +207,19 @@ int launch_lin_chunk(int ssd, const void* q, int ld_q, const void* k, int ld_k, 
                      const float* bias, const float* hparam, float qscale, float* state, float* out, int ld_out, const int* q_start,
                      const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs, int H, int G, int dk, int dv, cudaStream_t s);
 
+// single tokens (every span is one token), fp32 rows; for sequences x heads >= 148; _gave_up: CTAs whose bounded waits ran out so far
+bool lin_step_supported(int n_seqs, int H, int dk, int dv);
+unsigned lin_step_gave_up();
+int launch_lin_step(int ssd, const float* q, int ld_q, const float* k, int ld_k, const float* v, int ld_v, const float* step, int ld_step,
+                    const float* bias, const float* hparam, const float* tab, int rdims, float qscale, float* state, float* out, int ld_out,
+                    const int* q_start, const int* q_len, const int* kv_len, const int* seq_slot, int n_seqs, int H, int G, int dk, int dv,
+                    cudaStream_t s);
+
 // bounded handoff waits: device abort word + time limit for the waits of each translation unit (0 / null = trap policy)
 int set_wait_policy_gemm(uint32_t* abort_word, unsigned long long limit_ns);
 int set_wait_policy_mixed(uint32_t* abort_word, unsigned long long limit_ns);
 int set_wait_policy_diff(uint32_t* abort_word, unsigned long long limit_ns);
+int set_wait_policy_step(uint32_t* abort_word, unsigned long long limit_ns);
 int set_wait_policy_elementwise(uint32_t* abort_word, unsigned long long limit_ns);
 
 // gemm_tc.cu

@@ -1673,6 +1673,8 @@ static int launch_scan_cb(const ScanArgs& a, int n_seqs, cudaStream_t s) {
 template <int MODE, int R, int LN, bool DEC>
 static int launch_scan_r(const ScanArgs& a, int n_seqs, cudaStream_t s) {
   if constexpr (DEC) {
+    // a stream over the states: whole 128-byte lines per state row when there are enough blocks
+    if (a.dv % 32 == 0 && static_cast<long long>(a.H) * n_seqs * (a.dv / 32) >= 1184) return launch_scan_cb<MODE, R, LN, true, 32>(a, n_seqs, s);
     return launch_scan_cb<MODE, R, LN, true, 16>(a, n_seqs, s);
   } else {
     // the scan of a span is sequential in its tokens: its only parallelism is heads x sequences x column blocks, so

@@ -649,6 +649,63 @@ def test_chunked_recurrences_keep_fp32_precision(H, G, N, V, ssd):
 
 
 @gpu
+@pytest.mark.parametrize("S,H,G,N,V", [(40, 4, 2, 16, 24), (50, 3, 3, 64, 32), (20, 8, 1, 128, 64), (151, 2, 1, 200, 12), (300, 5, 5, 48, 256), (33, 16, 16, 128, 128)])
+@pytest.mark.parametrize("ssd", [True, False])
+def test_decode_steps_stream_the_states(S, H, G, N, V, ssd):
+    """single tokens of many sequences: some idle (their states are left alone), some at their first token (whatever the slot holds,
+    the state starts from zeros); several steps in a row on scattered slots"""
+    from bee2bee_b200 import ops
+
+    dev = "cuda"
+    g = torch.Generator().manual_seed(S + N)
+    if not ssd:
+        G = H
+    rot = 0 if ssd else N // 2 // 2 * 2
+    slots = torch.randperm(S + 3, generator=g)[:S]
+    live = torch.rand(S, generator=g) > 0.2
+    pos = torch.randint(1, 50, (S,), generator=g)
+    pos[live.nonzero()[0]] = 0
+    pos[live.nonzero()[-1]] = 0
+    state = torch.randn(S + 3, H, N, V, generator=g)
+    state[slots[live & (pos == 0)]] = float("nan")
+    ref = torch.where(torch.isnan(state), torch.zeros(()), state).double()
+    sd = state.to(dev)
+    alog, bias, decay = torch.randn(H, generator=g) - 1, torch.randn(H, generator=g) - 1, torch.rand(H, generator=g)
+    hi, lo = ops.split_frequencies([0.3 ** i for i in range(max(1, rot // 2))], dev)
+    for step in range(3):
+        x = torch.randn(S, 2 * G * N + H * V + 5, generator=g)
+        dt = torch.randn(S, H + 2, generator=g)
+        q, k, v = x[:, 5:5 + G * N].double().view(S, G, N), x[:, 5 + G * N:5 + 2 * G * N].double().view(S, G, N), x[:, 5 + 2 * G * N:].double().view(S, H, V)
+        tab = torch.zeros(S, max(2, rot), device=dev)
+        p = (pos + step).int().to(dev)
+        if rot:
+            ops.rot_table(p, hi, lo, 1.0, tab, S)
+            t = tab.double().cpu().view(S, 1, rot // 2, 2)
+            for z in (q, k):
+                a, b = z[..., :rot:2].clone(), z[..., 1:rot:2].clone()
+                z[..., :rot:2], z[..., 1:rot:2] = a * t[..., 0] - b * t[..., 1], b * t[..., 0] + a * t[..., 1]
+        grp = torch.arange(H) // (H // G)
+        b = torch.nn.functional.softplus((dt[:, 2:] + bias).double()) if ssd else torch.ones(S, H, dtype=torch.float64)
+        d = torch.exp(-torch.exp(alog.double()) * b) if ssd else decay.double().expand(S, H)
+        new = d[..., None, None] * ref[slots] + (b[..., None] * k[:, grp])[..., None] * v[:, :, None]
+        want = torch.einsum("shn,shnv->shv", q[:, grp], new) * 0.5
+        ref[slots[live]] = new[live]
+        out = torch.full((S, H * V), 7.0, device=dev)
+        i32 = dict(dtype=torch.int32, device=dev)
+        ops.lin_step(ops.SCAN_SSD if ssd else ops.SCAN_RETENTION, x.to(dev), 5, x.to(dev), 5 + G * N, x.to(dev), 5 + 2 * G * N, sd, out,
+                     torch.arange(S, **i32), live.int().to(dev), p + 1, slots.int().to(dev), S, H, G, N, V, step=dt.to(dev) if ssd else None, off_step=2,
+                     bias=bias.to(dev) if ssd else None, hparam=(alog if ssd else decay).to(dev), tab=tab if rot else None, rdims=rot, qscale=0.5)
+        got = out.double().cpu().view(S, H, V)
+        assert float((got[live] - want[live]).abs().max()) < 3e-5 * float(want.abs().max())
+        assert bool((got[~live] == 7.0).all())
+    used = slots[live]
+    assert torch.allclose(sd.double().cpu()[used], ref[used], atol=1e-4, rtol=1e-5)
+    idle = [i for i in range(S + 3) if i not in set(used.tolist())]
+    assert torch.equal(sd.cpu()[idle], state[idle])
+    assert ops.lin_step_supported(S, H, N, V) and ops.native().lin_step_gave_up() == 0
+
+
+@gpu
 @pytest.mark.parametrize("H,D,V,rot", [(3, 16, 24, 16), (2, 48, 40, 22), (4, 128, 64, 128), (1, 8, 16, 0)])
 def test_rotated_bf16_rows(H, D, V, rot):
     from bee2bee_b200 import ops
