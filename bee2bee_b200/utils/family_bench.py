@@ -318,7 +318,7 @@ def cost(name: str, a, hint: Dict):
         H, dv = a[6], a[7]
         return 0.0, T * H * dv * (4 + 4 + 2), False
     if name == "act_cols":
-        return 0.0, T * a[3] * 6, False
+        return 0.0, a[5] * a[3] * (4 + a[2].element_size()), False
     if name == "ls_join":
         W = a[0].shape[-1]
         rows = a[4] if a[3] is not None else T

@@ -10,7 +10,7 @@
 // so a chunk is four matrix products instead of 64 dependent steps.  q, k and v are bf16 (projections and convolved activations);
 // everything that enters the recurrence besides them keeps fp32 precision: decays, their logarithms and sums, step sizes, the
 // state (fp32 accumulators that stay in registers from chunk to chunk), and where a product of such numbers is an operand (weighted
-// scores, weighted keys, the state in front of q) it is split into a high and a low bf16 part, 16 bits of mantissa together.
+// scores, weighted values, the state in front of q) it is split into a high and a low bf16 part, 16 bits of mantissa together.
 // A block = 32 state columns of one (sequence, head), sixteen warps.  Tokens of the chunk are the M dimension of the output products
 // (four tiles of 16, four warps each that split the keys and the state rows); state rows are the M dimension of the update.
 // The next chunk's rows come in by cp.async meanwhile, and one warp prepares its decays and step sizes.
@@ -70,6 +70,9 @@ constexpr int LC_L = 64, LC_VB = 32, LC_WARPS = 16, LC_THREADS = 32 * LC_WARPS;
 constexpr int LC_VS = LC_VB + 8;                       // row stride of value and state tiles (elements)
 constexpr int LC_OS = LC_VB + 4;                       // row stride of partial outputs (floats)
 
+// partial outputs that go through shared memory: all four of a token tile, or (widest states: no room) three beside one in registers
+__host__ __device__ constexpr int lc_parts(int KT) { return KT > 8 ? 3 : 4; }
+
 struct ChunkArgs {
   const bf16* q; const bf16* k; const bf16* v;         // [T, ld] rows, already at their first column
   int ld_q, ld_k, ld_v;
@@ -89,7 +92,7 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
   pdl_begin();
   constexpr int NP = 16 * KT, RS = NP + 8;             // row stride of q / k tiles
   constexpr int UN = KT > 8 ? KT / 8 : 1;              // state units (16 rows x 16 columns) per warp
-  constexpr int TILE = LC_L * RS, VT = LC_L * LC_VS;
+  constexpr int TILE = LC_L * RS, VT = LC_L * LC_VS, OB = lc_parts(KT);
   constexpr float LOG2E = 1.4426950408889634f;
   extern __shared__ __align__(16) uint8_t smem_[];
   bf16* qs = reinterpret_cast<bf16*>(smem_);           // [2][64][RS]
@@ -97,8 +100,10 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
   bf16* vs = ks + 2 * TILE;                            // [2][64][VS]
   bf16* sh = vs + 2 * VT;                              // [NP][VS] state, high parts
   bf16* sl = sh + NP * LC_VS;
-  float* ox = reinterpret_cast<float*>(sl + NP * LC_VS);      // [4][64][OS] partial outputs of the four warps of a token tile
-  float* scal = ox + 4 * LC_L * LC_OS;                 // [2][3][64]: c_t (in powers of two), b_s, exp(c_L - c_s) b_s
+  bf16* vh = sl + NP * LC_VS;                          // [64][VS] values times their weight in the update, high and low parts
+  bf16* vl = vh + VT;
+  float* ox = reinterpret_cast<float*>(vl + VT);       // [4][64][OS] partial outputs of the four warps of a token tile
+  float* scal = ox + OB * LC_L * LC_OS;                 // [2][3][64]: c_t (in powers of two), b_s, exp(c_L - c_s) b_s
   const int s = blockIdx.z, hd = blockIdx.y, v0 = blockIdx.x * LC_VB;
   const int n = a.q_len[s];
   if (n <= 0) return;                                  // (block-uniform)
@@ -125,23 +130,31 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
         S[u][nt][e] = (owner && pos0 > 0 && r < a.dk && v0 + c < a.dv) ? Sg[static_cast<size_t>(r) * a.dv + c] : 0.f;
       }
 
-  auto stage = [&](int ch) {
-    const int buf = ch & 1, tb = ch * LC_L;
-    const int cols = a.dk / 8;
+  // this thread's pieces of a chunk: q and k rows sr[] (16 bytes at column sc), and (first 256 threads) 8 channels of value row tid / 4
+  constexpr int PC = (LC_L * (NP / 8) + LC_THREADS - 1) / LC_THREADS;
+  const int sr = tid / (NP / 8), scol = tid % (NP / 8) * 8, vr = tid >> 2, vc = (tid & 3) * 8;
+  constexpr int STEP = LC_THREADS / (NP / 8);          // rows between two pieces of a thread
+  const bool s_ok = scol < a.dk, v_ok = tid < 4 * LC_L && v0 + vc < a.dv;
+  const bf16* qp = qg + static_cast<size_t>(t0 + sr) * a.ld_q + scol;
+  const bf16* kp = kg + static_cast<size_t>(t0 + sr) * a.ld_k + scol;
+  const bf16* vp = vg + static_cast<size_t>(t0 + vr) * a.ld_v + vc;
+  const uint32_t qd = sptr(qs + sr * RS + scol), kd = sptr(ks + sr * RS + scol), vd = sptr(vs + vr * LC_VS + vc);
+  auto stage = [&](int ch) {                           // (called once per chunk, in order)
+    const int left = n - ch * LC_L;
+    const uint32_t bq = (ch & 1) * TILE * 2;
 #pragma unroll
-    for (int e0 = 0; e0 < LC_L * (NP / 8); e0 += LC_THREADS) {
-      const int e = e0 + tid, r = e / (NP / 8), c = e % (NP / 8);
-      const bool ok = tb + r < n && c < cols;
-      const size_t t = static_cast<size_t>(t0 + (ok ? tb + r : 0));
-      cp16(sptr(qs + buf * TILE + r * RS + c * 8), qg + t * a.ld_q + (ok ? c * 8 : 0), ok);
-      cp16(sptr(ks + buf * TILE + r * RS + c * 8), kg + t * a.ld_k + (ok ? c * 8 : 0), ok);
+    for (int i = 0; i < PC; ++i) {
+      const bool ok = s_ok && sr + i * STEP < left;
+      cp16(qd + bq + i * STEP * RS * 2, ok ? qp + i * STEP * a.ld_q : a.q, ok);
+      cp16(kd + bq + i * STEP * RS * 2, ok ? kp + i * STEP * a.ld_k : a.k, ok);
     }
     if (tid < 4 * LC_L) {
-      const int r = tid >> 2, c = tid & 3;             // 64 rows x 4 pieces of 8 columns
-      const bool ok = tb + r < n && v0 + c * 8 < a.dv;
-      const size_t t = static_cast<size_t>(t0 + (ok ? tb + r : 0));
-      cp16(sptr(vs + buf * VT + r * LC_VS + c * 8), vg + t * a.ld_v + (ok ? c * 8 : 0), ok);
+      const bool ok = v_ok && vr < left;
+      cp16(vd + (ch & 1) * VT * 2, ok ? vp : a.v, ok);
     }
+    qp += static_cast<size_t>(LC_L) * a.ld_q;
+    kp += static_cast<size_t>(LC_L) * a.ld_k;
+    vp += static_cast<size_t>(LC_L) * a.ld_v;
     asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
   // the scalar part of a chunk, by one warp that has no keys in front of its tokens (two tokens per lane): step sizes, decays, sums
@@ -184,6 +197,7 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
     scalars(0, xs);
     if (nch > 1) load_step(1, xs);
   }
+  __syncthreads();
   const int mt = warp & 3, kh = warp >> 2;             // token tile; which quarter of the keys and of the state rows
   const uint32_t vt_off = (((lane & 7) + ((lane >> 3) & 1) * 8) * LC_VS + (lane >> 4) * 8) * 2;
   for (int ch = 0; ch < nch; ++ch) {
@@ -204,10 +218,22 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
           }
     }
     asm volatile("cp.async.wait_group 1;\n" ::: "memory");
-    __syncthreads();
     const float* cum = scal + buf * 3 * LC_L;
     const float* wst = cum + LC_L;
-    const float* wup = wst + LC_L;
+    if (tid < 4 * LC_L) {                              // the values this thread has copied, weighted for the update
+      const float w = wst[LC_L + vr];
+      const uint4 x = *reinterpret_cast<const uint4*>(vs + buf * VT + vr * LC_VS + vc);
+      const uint32_t xw[4] = {x.x, x.y, x.z, x.w};
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&xw[e]));
+        split2(f.x * w, f.y * w, &hi[e], &lo[e]);
+      }
+      *reinterpret_cast<uint4*>(vh + vr * LC_VS + vc) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(vl + vr * LC_VS + vc) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    __syncthreads();
 
     // ---- outputs of 16 tokens against a quarter of the keys and of the state rows
     float op[4][4], os[4][4];
@@ -282,11 +308,17 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
     }
     {
       const float e0 = ex2(cr0), e1 = ex2(cr1);
-      float* dst = ox + (kh * LC_L + r0) * LC_OS + 2 * tig;
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {
-        *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(op[nt][0] + e0 * os[nt][0], op[nt][1] + e0 * os[nt][1]);
-        *reinterpret_cast<float2*>(dst + 8 * LC_OS + nt * 8) = make_float2(op[nt][2] + e1 * os[nt][2], op[nt][3] + e1 * os[nt][3]);
+      for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) op[nt][e] += (e < 2 ? e0 : e1) * os[nt][e];
+      if (OB == 4 || kh > 0) {
+        float* dst = ox + ((kh - (4 - OB)) * LC_L + r0) * LC_OS + 2 * tig;
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) {
+          *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(op[nt][0], op[nt][1]);
+          *reinterpret_cast<float2*>(dst + 8 * LC_OS + nt * 8) = make_float2(op[nt][2], op[nt][3]);
+        }
       }
     }
     // ---- state behind this chunk: 16 rows x 16 columns per unit, over all tokens
@@ -300,27 +332,42 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
           for (int e = 0; e < 4; ++e) S[u][nt][e] *= dec;
 #pragma unroll
       for (int k2 = 0; k2 < LC_L / 16; ++k2) {
-        const float2 wa = *reinterpret_cast<const float2*>(wup + k2 * 16 + 2 * tig), wb = *reinterpret_cast<const float2*>(wup + k2 * 16 + 2 * tig + 8);
 #pragma unroll
         for (int u = 0; u < UN; ++u) {
           const int unit = warp + LC_WARPS * u;
-          uint32_t kf[4], hi[4], lo[4], b[4];
+          uint32_t kf[4], b[4], d[4];
           ldsm_t(kf, sptr(ks + buf * TILE + (k2 * 16 + (lane & 7) + (lane >> 4) * 8) * RS + unit % KT * 16 + ((lane >> 3) & 1) * 8));
-          ldsm_t(b, sptr(vs + buf * VT + k2 * 16 * LC_VS) + vt_off + unit / KT * 32);
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kf[e]));
-            split2(f.x * (e < 2 ? wa.x : wb.x), f.y * (e < 2 ? wa.y : wb.y), &hi[e], &lo[e]);
-          }
-          mma(S[u][0], hi, b[0], b[1]);
-          mma(S[u][1], hi, b[2], b[3]);
-          mma(S[u][0], lo, b[0], b[1]);
-          mma(S[u][1], lo, b[2], b[3]);
+          ldsm_t(b, sptr(vh + k2 * 16 * LC_VS) + vt_off + unit / KT * 32);
+          ldsm_t(d, sptr(vl + k2 * 16 * LC_VS) + vt_off + unit / KT * 32);
+          mma(S[u][0], kf, b[0], b[1]);
+          mma(S[u][1], kf, b[2], b[3]);
+          mma(S[u][0], kf, d[0], d[1]);
+          mma(S[u][1], kf, d[2], d[3]);
         }
       }
     }
     __syncthreads();                                   // partial outputs are there; tiles and the state operand may be written again
-    {
+    if constexpr (OB == 3) {
+      if (kh == 0) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int r = r0 + e * 8;
+          if (tb + r >= n) continue;
+          float* dst = a.out + static_cast<size_t>(t0 + tb + r) * a.ld_out + static_cast<size_t>(hd) * a.dv + v0;
+#pragma unroll
+          for (int nt = 0; nt < 4; ++nt) {
+            const int c = nt * 8 + 2 * tig;
+            float2 v = make_float2(op[nt][2 * e], op[nt][2 * e + 1]);
+#pragma unroll
+            for (int k = 0; k < OB; ++k) {
+              const float2 o = *reinterpret_cast<const float2*>(ox + (k * LC_L + r) * LC_OS + c);
+              v = make_float2(v.x + o.x, v.y + o.y);
+            }
+            if (v0 + c < a.dv) *reinterpret_cast<float2*>(dst + c) = make_float2(v.x * a.qscale, v.y * a.qscale);
+          }
+        }
+      }
+    } else {
       const int r = tid >> 3, c = (tid & 7) * 4;       // 64 rows x 8 pieces of 4 columns
       if (tb + r < n && v0 + c < a.dv) {
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -348,8 +395,9 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
 template <int KT, bool SSD>
 int launch_kt(const ChunkArgs& a, int n_seqs, cudaStream_t s) {
   constexpr int NP = 16 * KT, RS = NP + 8;
-  constexpr size_t bytes = static_cast<size_t>(4 * LC_L * RS + 2 * LC_L * LC_VS + 2 * NP * LC_VS) * 2 +
-                           static_cast<size_t>(4 * LC_L * LC_OS + 6 * LC_L) * 4;
+  constexpr size_t bytes = static_cast<size_t>(4 * LC_L * RS + 4 * LC_L * LC_VS + 2 * NP * LC_VS) * 2 +
+                           static_cast<size_t>(lc_parts(KT) * LC_L * LC_OS + 6 * LC_L) * 4;
+  static_assert(bytes <= 227 * 1024, "shared memory of a block");
   static bool set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);

@@ -601,7 +601,7 @@ def test_retention_scan(H, D, V, rot):
 def test_chunked_recurrences_keep_fp32_precision(H, G, N, V, ssd):
     """spans of many lengths (whole chunks, ragged ones, two tokens) of one sequence beside an idle and a short one, single tokens in
     between through the token-by-token kernel on the same states.  q, k and v are bf16 numbers here, so the result must be as exact as
-    in fp32: weighted scores, weighted keys and the state keep their low parts.  Strong and weak decays side by side."""
+    in fp32: weighted scores, weighted values and the state keep their low parts.  Strong and weak decays side by side."""
     from bee2bee_b200 import ops
 
     dev = "cuda"
