@@ -283,6 +283,16 @@ __global__ void __launch_bounds__(256) hc_step_kernel(float* streams, const int*
 // ------------------------------------------------------------------------------------------ activations
 // out[t, c] = act(in[t, off + c]) for c < n   (0 = copy, 1 = tanh, 2 = squared relu,
 // 3 = xIELU: z > 0: p0 z^2 + z/2, z <= 0: p1 (e^z - 1 - z) + z/2,  4 = soft cap p0 tanh(z / p0))
+__device__ __forceinline__ float act_col_(float v, int act, float p0, float p1) {
+  if (act == 1) return tanhf(v);
+  if (act == 2) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  if (act == 3) return v > 0.f ? p0 * v * v + 0.5f * v : p1 * (expm1f(v) - v) + 0.5f * v;
+  return act == 4 ? p0 * tanhf(v / p0) : v;
+}
+
 template <typename OT>
 __global__ void act_cols_kernel(const float* __restrict__ in, int ld_in, int off, OT* __restrict__ out, int ld_out,
                                 int n, int act, float p0, float p1, size_t total) {
@@ -291,12 +301,27 @@ __global__ void act_cols_kernel(const float* __restrict__ in, int ld_in, int off
        i += static_cast<size_t>(gridDim.x) * blockDim.x) {
     const size_t t = i / n;
     const int c = static_cast<int>(i % n);
-    float v = in[t * ld_in + off + c];
-    if (act == 1) v = tanhf(v);
-    else if (act == 2) { v = fmaxf(v, 0.f); v = v * v; }
-    else if (act == 3) v = v > 0.f ? p0 * v * v + 0.5f * v : p1 * (expm1f(v) - v) + 0.5f * v;
-    else if (act == 4) v = p0 * tanhf(v / p0);
+    const float v = act_col_(in[t * ld_in + off + c], act, p0, p1);
     stf(out, t * ld_out + c, v);
+  }
+}
+
+// four columns per thread, grid (column chunks, rows): every offset a multiple of four
+template <typename OT>
+__global__ void __launch_bounds__(256)
+    act_cols4_kernel(const float* __restrict__ in, int ld_in, int off, OT* __restrict__ out, int ld_out, int n, int act, float p0, float p1) {
+  pdl_begin();
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (c >= n) return;
+  const size_t t = blockIdx.y;
+  const float4 v = *reinterpret_cast<const float4*>(in + t * ld_in + off + c);
+  const float r[4] = {act_col_(v.x, act, p0, p1), act_col_(v.y, act, p0, p1), act_col_(v.z, act, p0, p1), act_col_(v.w, act, p0, p1)};
+  OT* dst = out + t * ld_out + c;
+  if constexpr (sizeof(OT) == 4) {
+    *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+  } else {
+    __nv_bfloat162 a = __floats2bfloat162_rn(r[0], r[1]), b = __floats2bfloat162_rn(r[2], r[3]);
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<unsigned*>(&a), *reinterpret_cast<unsigned*>(&b));
   }
 }
 
@@ -925,6 +950,13 @@ int launch_act_cols(const float* in, int ld_in, int off, void* out, int ld_out, 
                     int f32, cudaStream_t s) {
   const size_t total = static_cast<size_t>(T) * n;
   if (total == 0) return 0;
+  if (n % 4 == 0 && ld_in % 4 == 0 && off % 4 == 0 && ld_out % 4 == 0 && T <= 65535 && reinterpret_cast<uintptr_t>(in) % 16 == 0 &&
+      reinterpret_cast<uintptr_t>(out) % 16 == 0) {
+    const dim3 grid((n / 4 + 255) / 256, T);
+    if (f32) launch_kernel(act_cols4_kernel<float>, grid, dim3(256), 0, s, 1u, in, ld_in, off, static_cast<float*>(out), ld_out, n, act, p0, p1);
+    else launch_kernel(act_cols4_kernel<bf16>, grid, dim3(256), 0, s, 1u, in, ld_in, off, static_cast<bf16*>(out), ld_out, n, act, p0, p1);
+    return last_error();
+  }
   const int blocks = static_cast<int>(total / 256 + 1 < 148 * 16 ? total / 256 + 1 : 148 * 16);
   if (f32) launch_kernel(act_cols_kernel<float>, dim3(blocks), dim3(256), 0, s, 1u, in, ld_in, off, static_cast<float*>(out), ld_out, n, act, p0, p1, total);
   else launch_kernel(act_cols_kernel<bf16>, dim3(blocks), dim3(256), 0, s, 1u, in, ld_in, off, static_cast<bf16*>(out), ld_out, n, act, p0, p1, total);

@@ -68,7 +68,7 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t* hi, uint32_t*
 
 constexpr int LC_L = 64, LC_VB = 32, LC_WARPS = 16, LC_THREADS = 32 * LC_WARPS;
 constexpr int LC_VS = LC_VB + 8;                       // row stride of value and state tiles (elements)
-constexpr int LC_OS = LC_VB + 4;                       // row stride of partial outputs (floats)
+constexpr int LC_OS = LC_VB + 8;                       // row stride of partial outputs (floats)
 
 // partial outputs that go through shared memory: all four of a token tile, or (widest states: no room) three beside one in registers
 __host__ __device__ constexpr int lc_parts(int KT) { return KT > 8 ? 3 : 4; }
@@ -244,40 +244,42 @@ __global__ void __launch_bounds__(LC_THREADS, 1)
     const int r0 = mt * 16 + gid, r1 = r0 + 8;
     const float cr0 = cum[r0], cr1 = cum[r1];
     const uint32_t qa = sptr(qs + buf * TILE + (mt * 16 + (lane & 15)) * RS + (lane >> 4) * 8);
+    const bool seen = kh <= mt;                        // (keys behind every token of the tile: nothing)
+    float g[4][4];                                     // two key tiles, even and odd steps apart (shorter chains)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) g[i][e] = 0.f;
     {
       const uint32_t ha = sptr(sh) + vt_off, la = sptr(sl) + vt_off;
-#pragma unroll
-      for (int k2 = 0; k2 < KT / 4; ++k2) {
-        const int kk = kh * (KT / 4) + k2;
-        uint32_t af[4];
-        ldsm(af, qa + kk * 32);
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          uint32_t b[4], d[4];
-          ldsm_t(b, ha + kk * 16 * LC_VS * 2 + j * 32);
-          ldsm_t(d, la + kk * 16 * LC_VS * 2 + j * 32);
-          mma(os[2 * j], af, b[0], b[1]);
-          mma(os[2 * j + 1], af, b[2], b[3]);
-          mma(os[2 * j], af, d[0], d[1]);
-          mma(os[2 * j + 1], af, d[2], d[3]);
-        }
-      }
-    }
-    if (kh <= mt) {                                    // (keys behind every token of the tile: nothing)
-      float g[4][4];                                   // two key tiles, even and odd steps apart (shorter chains)
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) g[i][e] = 0.f;
       const uint32_t kb = sptr(ks + buf * TILE + (kh * 16 + (lane & 7) + (lane >> 4) * 8) * RS + ((lane >> 3) & 1) * 8);
 #pragma unroll
       for (int kk = 0; kk < KT; ++kk) {
-        uint32_t af[4], b[4];
+        const bool mine = kk / (KT / 4) == kh;         // this warp's quarter of the state rows
+        if (!seen && !mine) continue;
+        uint32_t af[4];
         ldsm(af, qa + kk * 32);
-        ldsm(b, kb + kk * 32);
-        mma(g[2 * (kk & 1)], af, b[0], b[1]);
-        mma(g[2 * (kk & 1) + 1], af, b[2], b[3]);
+        if (seen) {
+          uint32_t b[4];
+          ldsm(b, kb + kk * 32);
+          mma(g[2 * (kk & 1)], af, b[0], b[1]);
+          mma(g[2 * (kk & 1) + 1], af, b[2], b[3]);
+        }
+        if (mine) {
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            uint32_t b[4], d[4];
+            ldsm_t(b, ha + kk * 16 * LC_VS * 2 + j * 32);
+            ldsm_t(d, la + kk * 16 * LC_VS * 2 + j * 32);
+            mma(os[2 * j], af, b[0], b[1]);
+            mma(os[2 * j + 1], af, b[2], b[3]);
+            mma(os[2 * j], af, d[0], d[1]);
+            mma(os[2 * j + 1], af, d[2], d[3]);
+          }
+        }
       }
+    }
+    if (seen) {
       // weighted scores -> A operand (high, low), times the values
       uint32_t ph[4], pl[4];
 #pragma unroll
